@@ -1,1 +1,1 @@
-from . import llama, puposun, ravapel, rugedra, vofanex  # noqa: F401 (register LlamaForCausalLM, Puposun, Ravapel, Rugedra and Vofanex)
+from . import livitar, llama, puposun, ravapel, rugedra, vofanex  # noqa: F401 (register Livitar, LlamaForCausalLM, Puposun, Ravapel, Rugedra and Vofanex)

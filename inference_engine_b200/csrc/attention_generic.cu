@@ -23,6 +23,10 @@
 // `softcap` > 0: a score s (after the scale) becomes softcap * tanh(s / softcap).  `keep_first` > 0 (with
 // a window): the keys at positions below `keep_first` stay visible to every later query of the request,
 // beside its window; they keep their own positions.
+// A bias by distance n = (query's position - key's position), added to the score after the scale:
+// -log_r1[head] * ln(1 + log_r2[head] * n), and/or a table, bias_table[head * bias_len + min(n, bias_len -
+// 1)].  `gate_elements` 1: `out_gate` holds a number per head and value entry ([token * gate_ld + head *
+// hdv + d]) instead of one per head.
 #include "common.cuh"
 #include <math.h>
 
@@ -69,7 +73,9 @@ paged_attention_generic_kernel(const T* __restrict__ q, const T* __restrict__ k_
                                int nh, int nkv, int hd, int hdv, int v_stride, int page_size, int total_pages,
                                float scale, int window, int chunk, const float* __restrict__ head_bias,
                                const float* __restrict__ sinks, const float* __restrict__ out_gate, int gate_ld,
-                               float softcap, int keep_first, int* err) {
+                               float softcap, int keep_first, int gate_elements, const float* __restrict__ log_r1,
+                               const float* __restrict__ log_r2, const float* __restrict__ bias_table, int bias_len,
+                               int* err) {
     extern __shared__ float q_smem[];  // [WARPS][hd]
     ie_pdl_trigger();
     ie_pdl_wait();
@@ -116,6 +122,8 @@ paged_attention_generic_kernel(const T* __restrict__ q, const T* __restrict__ k_
                 row = ((long long)page * nkv + kvh) * page_size + (kpos % page_size);
                 s = (hd % 8 == 0 ? dot_row(qs, k_cache + row * hd, hd) : dot_row_any(qs, k_cache + row * hd, hd)) * scale;
                 if (softcap > 0.f) s = softcap * tanhf(s * inv_cap);
+                if (log_r1 != nullptr) s -= log_r1[head] * log1pf(log_r2[head] * (float)(pos - kpos));
+                if (bias_table != nullptr) s += bias_table[(size_t)head * bias_len + min(pos - kpos, bias_len - 1)];
             }
         }
         float m_new = m, p;
@@ -145,11 +153,16 @@ paged_attention_generic_kernel(const T* __restrict__ q, const T* __restrict__ k_
     }
     T* orow = out + ((size_t)token * nh + head) * hdv;
     float inv = gated ? 1.0f : (l > 0.f ? 1.0f / l : 0.f);
-    if (out_gate != nullptr) inv *= 1.0f / (1.0f + expf(-out_gate[(size_t)token * gate_ld + head]));
+    if (out_gate != nullptr && !gate_elements) inv *= 1.0f / (1.0f + expf(-out_gate[(size_t)token * gate_ld + head]));
 #pragma unroll
     for (int i = 0; i < MAX_ACC; ++i) {
         int d = lane + 32 * i;
-        if (i < nacc && d < hdv) ie_store(orow + d, acc[i] * inv);
+        if (i < nacc && d < hdv) {
+            float f = inv;
+            if (out_gate != nullptr && gate_elements)
+                f *= 1.0f / (1.0f + expf(-out_gate[(size_t)token * gate_ld + (size_t)head * hdv + d]));
+            ie_store(orow + d, acc[i] * f);
+        }
     }
 }
 }  // namespace
@@ -160,10 +173,14 @@ IE_API int ie_paged_attention_generic(const void* q, const void* k_cache, const 
                                       int num_tokens, int nh, int nkv, int hd, int hdv, int v_stride,
                                       int page_size, int total_pages, float scale, int window, int chunk,
                                       const float* head_bias, const float* sinks, const float* out_gate,
-                                      int gate_ld, float softcap, int keep_first, int* err, void* stream) {
+                                      int gate_ld, float softcap, int keep_first, int gate_elements,
+                                      const float* log_r1, const float* log_r2, const float* bias_table,
+                                      int bias_len, int* err, void* stream) {
     if (num_tokens <= 0) return 0;
     if (hd < 1 || hdv < 1 || hdv > 32 * MAX_ACC || nkv <= 0 || nh % nkv != 0) return (int)cudaErrorInvalidValue;
     if (keep_first < 0 || softcap < 0.f || (keep_first > 0 && chunk > 0)) return (int)cudaErrorInvalidValue;
+    if ((log_r1 == nullptr) != (log_r2 == nullptr) || (bias_table != nullptr && bias_len < 1))
+        return (int)cudaErrorInvalidValue;
     dim3 grid((nh + WARPS - 1) / WARPS, num_tokens);
     size_t smem = (size_t)WARPS * hd * sizeof(float);
     cudaStream_t s = (cudaStream_t)stream;
@@ -171,11 +188,13 @@ IE_API int ie_paged_attention_generic(const void* q, const void* k_cache, const 
         paged_attention_generic_kernel<<<grid, WARPS * 32, smem, s>>>(
             (const __nv_bfloat16*)q, (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache,
             block_tables, table_width, seq_of_token, positions, (__nv_bfloat16*)out,
-            nh, nkv, hd, hdv, v_stride, page_size, total_pages, scale, window, chunk, head_bias, sinks, out_gate, gate_ld, softcap, keep_first, err);
+            nh, nkv, hd, hdv, v_stride, page_size, total_pages, scale, window, chunk, head_bias, sinks, out_gate, gate_ld, softcap, keep_first,
+            gate_elements, log_r1, log_r2, bias_table, bias_len, err);
     else
         paged_attention_generic_kernel<<<grid, WARPS * 32, smem, s>>>(
             (const float*)q, (const float*)k_cache, (const float*)v_cache,
             block_tables, table_width, seq_of_token, positions, (float*)out,
-            nh, nkv, hd, hdv, v_stride, page_size, total_pages, scale, window, chunk, head_bias, sinks, out_gate, gate_ld, softcap, keep_first, err);
+            nh, nkv, hd, hdv, v_stride, page_size, total_pages, scale, window, chunk, head_bias, sinks, out_gate, gate_ld, softcap, keep_first,
+            gate_elements, log_r1, log_r2, bias_table, bias_len, err);
     return IE_LAUNCH_CHECK();
 }

@@ -4,7 +4,9 @@
 // (their weight is null); value heads divided by their root mean square over `vdim` (eps inside the
 // root, no weight) before they are cached (`value_norm`); values that are the keys as projected
 // (with their bias, before norm and rotation: `values_from_keys`; the projection then holds no value
-// columns and vdim = dim); the rotation's pairs (`interleaved` 0: entry i with entry i + rot_dims / 2;
+// columns and vdim = dim); queries and keys divided by their root mean square without a weight
+// (`unit_norm`); query heads multiplied by a number per head (`q_head_scale`) and by
+// 1 + warm_coef * ln(floor((p + 1) / warm_every) + 1) at position p (`warm_every` > 0); the rotation's pairs (`interleaved` 0: entry i with entry i + rot_dims / 2;
 // 1: entry 2i with entry 2i + 1; the table of angles is the same).
 //
 // qk_norm_rope_write: from the fused 32-bit projection [N, ld] = (heads * dim queries, kv_heads *
@@ -27,6 +29,7 @@ qk_norm_rope_write_kernel(const float* __restrict__ proj, int ld, const int* __r
                           const float* __restrict__ table, int rot_dims, int table_positions,
                           const float* __restrict__ bias, int value_norm, int values_from_keys, int interleaved,
                           const float* __restrict__ q_weight, const float* __restrict__ k_weight, float eps,
+                          int unit_norm, const float* __restrict__ q_head_scale, float warm_coef, int warm_every,
                           T* __restrict__ q_out, T* __restrict__ k_cache, T* __restrict__ v_cache,
                           const int* __restrict__ slot_mapping, int heads, int kv_heads, int dim, int vdim,
                           int page_size, int total_pages, int* err) {
@@ -87,6 +90,11 @@ qk_norm_rope_write_kernel(const float* __restrict__ proj, int ld, const int* __r
         for (int d = lane; d < dim; d += 32) y[d] = (y[d] * inv) * weight[d];
     __syncwarp();
     int pos = positions[n];
+    float factor = (unit_norm && weight == nullptr) ? inv : 1.0f;
+    if (is_q) {
+        if (q_head_scale != nullptr) factor *= q_head_scale[unit];
+        if (warm_every > 0) factor *= 1.0f + warm_coef * logf((float)((pos + 1) / warm_every + 1));
+    }
     int half = rot_dims / 2;
     if (half > 0 && (pos < 0 || pos >= table_positions)) {
         if (lane == 0) ie_report(err, IE_ERR_POSITION, pos, n);
@@ -108,7 +116,7 @@ qk_norm_rope_write_kernel(const float* __restrict__ proj, int ld, const int* __r
             float c = table[((size_t)pos * 2) * half + (d - half)], s = table[((size_t)pos * 2 + 1) * half + (d - half)];
             r = y[d] * c + y[d - half] * s;
         }
-        ie_store(dst + d, r);
+        ie_store(dst + d, r * factor);
     }
 }
 }  // namespace
@@ -116,14 +124,14 @@ qk_norm_rope_write_kernel(const float* __restrict__ proj, int ld, const int* __r
 IE_API int ie_qk_norm_rope_write(const float* proj, int ld, const int* positions, const float* table, int rot_dims,
                                  int table_positions, const float* bias, int value_norm, int values_from_keys,
                                  int interleaved, const float* q_weight,
-                                 const float* k_weight, float eps,
-                                 void* q_out, void* k_cache, void* v_cache, int dtype, const int* slot_mapping,
+                                 const float* k_weight, float eps, int unit_norm, const float* q_head_scale,
+                                 float warm_coef, int warm_every, void* q_out, void* k_cache, void* v_cache, int dtype, const int* slot_mapping,
                                  int num_tokens, int heads, int kv_heads, int dim, int vdim, int page_size,
                                  int total_pages, int* err, void* stream) {
     if (num_tokens <= 0) return 0;
     if (rot_dims < 0 || rot_dims % 2 || rot_dims > dim || (rot_dims > 0 && table == nullptr))
         return (int)cudaErrorInvalidValue;
-    if (values_from_keys && vdim != dim) return (int)cudaErrorInvalidValue;
+    if ((values_from_keys && vdim != dim) || warm_every < 0) return (int)cudaErrorInvalidValue;
     size_t smem = (size_t)QW_WARPS * dim * sizeof(float);
     if (smem > 48 * 1024) return (int)cudaErrorInvalidValue;
     int units = heads + 2 * kv_heads;
@@ -131,10 +139,10 @@ IE_API int ie_qk_norm_rope_write(const float* proj, int ld, const int* positions
     cudaStream_t s = (cudaStream_t)stream;
     if (dtype == IE_BF16)
         return ie_launch(qk_norm_rope_write_kernel<__nv_bfloat16>, grid, dim3(QW_WARPS * 32), smem, s, proj, ld,
-                         positions, table, rot_dims, table_positions, bias, value_norm, values_from_keys, interleaved, q_weight, k_weight, eps, (__nv_bfloat16*)q_out,
+                         positions, table, rot_dims, table_positions, bias, value_norm, values_from_keys, interleaved, q_weight, k_weight, eps, unit_norm, q_head_scale, warm_coef, warm_every, (__nv_bfloat16*)q_out,
                          (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, slot_mapping, heads, kv_heads, dim, vdim,
                          page_size, total_pages, err);
     return ie_launch(qk_norm_rope_write_kernel<float>, grid, dim3(QW_WARPS * 32), smem, s, proj, ld, positions, table,
-                     rot_dims, table_positions, bias, value_norm, values_from_keys, interleaved, q_weight, k_weight, eps, (float*)q_out, (float*)k_cache,
+                     rot_dims, table_positions, bias, value_norm, values_from_keys, interleaved, q_weight, k_weight, eps, unit_norm, q_head_scale, warm_coef, warm_every, (float*)q_out, (float*)k_cache,
                      (float*)v_cache, slot_mapping, heads, kv_heads, dim, vdim, page_size, total_pages, err);
 }

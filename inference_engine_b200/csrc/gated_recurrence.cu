@@ -15,7 +15,12 @@
 //    numbers), taken as exp(logsigmoid(z_t) / tau); w_t = k_t, u_t = v_t; the read-out's gate is
 //    silu(.) instead of sigmoid(.).
 //
-// Kernels: lowrank_decay (a block takes sixteen tokens and 128 channels, so that a row of W2 is read
+//  * retention: a_t is one constant per head and the write gate is 1 (the gates' array then holds one
+//    token's numbers for all of them: a token stride of 0), w_t = k_t, u_t = v_t with q and k rotated by
+//    position; the read-out's unit root mean square has no weight.
+//
+// Kernels: rotate_heads (in place in the 32-bit projection: the first rot_dims entries of every head, by
+// pairs (i, i + rot_dims / 2), from the 32-bit table of angles); lowrank_decay (a block takes sixteen tokens and 128 channels, so that a row of W2 is read
 // once per sixteen tokens); short_conv_residual (+ tail update): out = x + causal convolution of x over time per
 // channel, the last taps - 1 inputs kept per request; hgrn2_gates; mlstm_gates (a warp per request
 // and head walks the step's tokens in order); gated_recurrence (columns of S do not interact: a
@@ -105,6 +110,28 @@ __global__ void hgrn2_gates_kernel(float* __restrict__ proj, int ld, const float
         float f = l + (1.0f - l) * sigmoid_f(row[size + c] + bias[c]);
         row[size + c] = f;
         write[idx] = 1.0f - f;
+    }
+}
+
+// grid: (tokens, blocks of pairs).  x: `units` heads of `dim` entries at the start of rows `ld` apart.
+__global__ void __launch_bounds__(128)
+rotate_heads_kernel(float* __restrict__ x, int ld, const int* __restrict__ positions, const float* __restrict__ table,
+                    int rot_dims, int table_positions, int units, int dim, int* err) {
+    ie_pdl_trigger();
+    ie_pdl_wait();
+    int n = blockIdx.x, half = rot_dims / 2;
+    int pos = positions[n];
+    if (pos < 0 || pos >= table_positions) {
+        if (threadIdx.x == 0) ie_report(err, IE_ERR_POSITION, pos, n);
+        return;
+    }
+    const float* cs = table + (size_t)pos * rot_dims;  // cos of the angles, then their sin
+    for (int i = blockIdx.y * 128 + threadIdx.x; i < units * half; i += gridDim.y * 128) {
+        int unit = i / half, j = i - unit * half;
+        float* p = x + (size_t)n * ld + (size_t)unit * dim + j;
+        float u = p[0], v = p[half], c = cs[j], s = cs[half + j];
+        p[0] = u * c - v * s;
+        p[half] = v * c + u * s;
     }
 }
 
@@ -211,15 +238,16 @@ __device__ __forceinline__ void cp_async16(float* dst, const float* src) {
 
 // grid: (column blocks, heads, requests).  Lane `sub` of a column's TPC lanes holds rows sub, sub + TPC,
 // ..., R of them.  q, a, w: element (n, head, d) at [n * ld + head * dim + d]; SCALAR: a and the write
-// gate b come from gates[(n * heads + head) * 3 + {0, 1}] and column `vdim` (if cols > vdim) has the
+// gate b come from gates[n * gate_stride + head * 3 + {0, 1}] and column `vdim` (if cols > vdim) has the
 // value 1.  v: (n, head, c) at [n * v_ld + head * vdim + c].  out: [N, heads, cols], times q_scale.
 template <int R, int TPC, bool SCALAR>
 __global__ void __launch_bounds__(GR_THREADS)
 gated_recurrence_kernel(const float* __restrict__ q, int q_ld, const float* __restrict__ a, int a_ld,
                         const float* __restrict__ w, int w_ld, const float* __restrict__ gates,
-                        const float* __restrict__ v, int v_ld, float* __restrict__ state, long long state_stride,
-                        const int* __restrict__ slots, const int* __restrict__ cu_q, float* __restrict__ out,
-                        int heads, int dim, int vdim, int cols, float q_scale, int num_slots) {
+                        int gate_stride, const float* __restrict__ v, int v_ld, float* __restrict__ state,
+                        long long state_stride, const int* __restrict__ slots, const int* __restrict__ cu_q,
+                        float* __restrict__ out, int heads, int dim, int vdim, int cols, float q_scale,
+                        int num_slots) {
     extern __shared__ __align__(16) float sm[];
     constexpr int COLS = GR_THREADS / TPC, DP = R * TPC;
     constexpr int ROWS = SCALAR ? 2 : 3;  // arrays of DP floats per token: q, w (, a)
@@ -283,7 +311,7 @@ gated_recurrence_kernel(const float* __restrict__ q, int q_ld, const float* __re
             if (c0 + c < vdim) cp_async4(vs + tt * COLS + c, v + (size_t)(start + t0 + tt) * v_ld + head * vdim + c0 + c);
         }
         if (SCALAR && tid < 2 * cnt)
-            cp_async4(gs + tid, gates + ((size_t)(start + t0 + (tid >> 1)) * heads + head) * 3 + (tid & 1));
+            cp_async4(gs + tid, gates + (size_t)(start + t0 + (tid >> 1)) * gate_stride + head * 3 + (tid & 1));
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     // (a step of one chunk waits for its memory once; a prompt's chunks find theirs landed: with one
@@ -348,8 +376,8 @@ gated_recurrence_kernel(const float* __restrict__ q, int q_ld, const float* __re
 }
 
 // One warp per (token, head).  o: [rows, cols]; with `gates` the column `vdim` is n . q and the
-// row is first divided by max(|n . q|, exp(-m)) + 1e-6.  weight: [vdim] shared by the heads, or
-// [heads * vdim].  gate_pre (optional): element (n, head, d) at [n * gate_ld + head * vdim + d]; the
+// row is first divided by max(|n . q|, exp(-m)) + 1e-6.  weight: [vdim] shared by the heads,
+// [heads * vdim], or null.  gate_pre (optional): element (n, head, d) at [n * gate_ld + head * vdim + d]; the
 // row is multiplied by sigmoid(gate_pre), or by silu(gate_pre) with gate_silu.
 template <typename T>
 __global__ void __launch_bounds__(128)
@@ -374,9 +402,10 @@ recurrence_readout_kernel(const float* __restrict__ o, int cols, const float* __
     }
     ss = warp_sum(ss);
     float inv = 1.0f / sqrtf(ss / (float)vdim + eps);
-    const float* wrow = weight + (weight_per_head ? (size_t)head * vdim : 0);
+    const float* wrow = weight != nullptr && weight_per_head ? weight + (size_t)head * vdim : weight;
     for (int d = lane; d < vdim; d += 32) {
-        float y = (src[d] / den) * inv * wrow[d];
+        float y = (src[d] / den) * inv;
+        if (weight != nullptr) y *= wrow[d];
         if (gate_pre != nullptr) {
             float gp = gate_pre[n * gate_ld + (size_t)head * vdim + d];
             y *= gate_silu ? silu_f(gp) : sigmoid_f(gp);
@@ -392,8 +421,8 @@ inline int grid_for(size_t total, int threads) {
 
 template <int R, int TPC, bool SCALAR>
 int launch_recurrence(const float* q, int q_ld, const float* a, int a_ld, const float* w, int w_ld,
-                      const float* gates, const float* v, int v_ld, float* state, long long state_stride,
-                      const int* slots, const int* cu_q, float* out, int num_seqs, int heads, int dim, int vdim,
+                      const float* gates, int gate_stride, const float* v, int v_ld, float* state,
+                      long long state_stride, const int* slots, const int* cu_q, float* out, int num_seqs, int heads, int dim, int vdim,
                       int cols, float q_scale, int num_slots, cudaStream_t s) {
     constexpr int COLS = GR_THREADS / TPC;
     size_t smem = (size_t)GR_STAGES * GR_CHUNK * ((SCALAR ? 2 : 3) * R * TPC + COLS + 4) * sizeof(float);
@@ -402,7 +431,7 @@ int launch_recurrence(const float* q, int q_ld, const float* a, int a_ld, const 
     if (e != cudaSuccess) return (int)e;
     dim3 grid((cols + COLS - 1) / COLS, heads, num_seqs);
     return ie_launch(gated_recurrence_kernel<R, TPC, SCALAR>, grid, dim3(GR_THREADS), smem, s, q, q_ld, a, a_ld, w,
-                     w_ld, gates, v, v_ld, state, state_stride, slots, cu_q, out, heads, dim, vdim, cols, q_scale,
+                     w_ld, gates, gate_stride, v, v_ld, state, state_stride, slots, cu_q, out, heads, dim, vdim, cols, q_scale,
                      num_slots);
 }
 }  // namespace
@@ -435,6 +464,18 @@ IE_API int ie_short_conv_residual(const void* x, int dtype, const float* w, floa
                      state_stride, slots, cu_q, channels, taps, num_slots);
 }
 
+IE_API int ie_rotate_heads(float* x, int ld, const int* positions, const float* table, int rot_dims,
+                           int table_positions, int num_tokens, int units, int dim, int* err, void* stream) {
+    if (num_tokens <= 0 || rot_dims == 0) return 0;
+    if (rot_dims < 0 || rot_dims % 2 || rot_dims > dim || table == nullptr || units < 1 || (long long)units * dim > ld)
+        return (int)cudaErrorInvalidValue;
+    int pairs = units * (rot_dims / 2), per_row = (pairs + 127) / 128;
+    // few tokens: a thread per pair; many: several pairs per thread
+    dim3 grid(num_tokens, num_tokens >= 256 ? (per_row + 3) / 4 : per_row);
+    return ie_launch(rotate_heads_kernel, grid, dim3(128), 0, (cudaStream_t)stream, x, ld, positions, table, rot_dims,
+                     table_positions, units, dim, err);
+}
+
 IE_API int ie_lowrank_decay(const float* y, int y_ld, const float* w2, const float* bias, float inv_tau,
                             float* decay, int num_tokens, int channels, int rank, void* stream) {
     if (num_tokens <= 0 || channels <= 0) return 0;
@@ -460,16 +501,17 @@ IE_API int ie_mlstm_gates(const float* gi, const float* gf, int ld, const float*
                      bias_i, bias_f, cap, state, state_stride, m_offset, slots, cu_q, gates, heads, num_slots);
 }
 
-// gates == nullptr: a and w per head and channel (a, a_ld given); else the gates' scalars.
+// gates == nullptr: a and w per head and channel (a, a_ld given); else the gates' scalars, a token's
+// `gate_stride` numbers apart (0: the same for every token).
 IE_API int ie_gated_recurrence(const float* q, int q_ld, const float* a, int a_ld, const float* w, int w_ld,
-                               const float* gates, const float* v, int v_ld, float* state, long long state_stride,
-                               const int* slots, const int* cu_q, float* out, int num_seqs, int heads, int dim,
+                               const float* gates, int gate_stride, const float* v, int v_ld, float* state,
+                               long long state_stride, const int* slots, const int* cu_q, float* out, int num_seqs, int heads, int dim,
                                int vdim, int cols, float q_scale, int num_slots, void* stream) {
     if (num_seqs <= 0) return 0;
     if (cols < vdim || cols > vdim + 1 || (gates == nullptr && (a == nullptr || cols != vdim)))
         return (int)cudaErrorInvalidValue;
     cudaStream_t s = (cudaStream_t)stream;
-#define IE_GR_ARGS q, q_ld, a, a_ld, w, w_ld, gates, v, v_ld, state, state_stride, slots, cu_q, out, num_seqs, heads, dim, vdim, cols, q_scale, num_slots, s
+#define IE_GR_ARGS q, q_ld, a, a_ld, w, w_ld, gates, gate_stride, v, v_ld, state, state_stride, slots, cu_q, out, num_seqs, heads, dim, vdim, cols, q_scale, num_slots, s
 #define IE_GR_PICK(SC)                                                        \
     if (dim <= 8) return launch_recurrence<8, 1, SC>(IE_GR_ARGS);             \
     if (dim <= 16) return launch_recurrence<8, 2, SC>(IE_GR_ARGS);            \

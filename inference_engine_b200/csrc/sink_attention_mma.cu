@@ -28,6 +28,14 @@
 // query of the request beside its window, at their own positions.  A block then walks the tiles that
 // hold kept keys and lie wholly before its window's first tile, then the window's tiles; with key
 // ranges cut among blocks the first `kept_splits` ranges are the kept tiles'.
+//
+// Variants chosen at build time, SK_BIAS: a bias by distance n = (query's position - key's position) is
+// added to a score after the scale.  1: -log_r1[head] * ln(1 + log_r2[head] * n).  2: a table,
+// bias_table[head * bias_len + min(n, bias_len - 1)]; a tile whose keys all lie at least bias_len - 1
+// before the block's first query takes the table's last entry without looking.  These variants also
+// leave the mask out in tiles that every row of the block sees whole.
+// `gate_elements` 1: the gate is a number per head and value entry, out_gate[token * gate_ld + head * SK_DV
+// + c], instead of one per head.
 #include "common.cuh"
 #include <math.h>
 
@@ -37,12 +45,16 @@
 #ifndef SK_DV
 #define SK_DV 64
 #endif
+#ifndef SK_BIAS
+#define SK_BIAS 0
+#endif
 
 namespace {
-constexpr int D = SK_D, DV = SK_DV;
+constexpr int D = SK_D, DV = SK_DV, BIAS = SK_BIAS;
 constexpr int ROWS = 64, KEYS = 64, WARPS = 4, THREADS = WARPS * 32;
 static_assert(THREADS == 2 * KEYS, "two threads bring a key's rows");
 constexpr int LDK = D + 8, LDV = DV + 8;  // rows 16 bytes longer: ldmatrix rows fall on different banks
+static_assert(BIAS >= 0 && BIAS <= 2, "no bias, the logarithm of the distance, a table");
 static_assert(D % 16 == 0 && DV % 16 == 0 && D <= 256 && DV <= 256, "sizes");
 constexpr float LOG2E = 1.4426950408889634f;
 
@@ -75,6 +87,12 @@ __device__ __forceinline__ float tanh_fast(float x) {
     x = fminf(fmaxf(x, -15.f), 15.f);
     return 1.f - __fdividef(2.f, __expf(2.f * x) + 1.f);
 }
+__device__ __forceinline__ float log2_fast(float x) {
+    float y;
+    asm("lg2.approx.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+__device__ __forceinline__ float sigmoid_of(float z) { return 1.0f / (1.0f + expf(-z)); }
 __device__ __forceinline__ float quad_max(float x) {
     x = fmaxf(x, __shfl_xor_sync(0xffffffffu, x, 1));
     return fmaxf(x, __shfl_xor_sync(0xffffffffu, x, 2));
@@ -93,7 +111,8 @@ sink_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat
                           int total_pages, float scale, int window, const float* __restrict__ sinks,
                           const float* __restrict__ out_gate, int gate_ld, float* __restrict__ partial,
                           int splits, int tiles_per_split, float softcap, int keep_first, int kept_splits,
-                          int* err) {
+                          int gate_elements, const float* __restrict__ log_r1, const float* __restrict__ log_r2,
+                          const float* __restrict__ bias_table, int bias_len, int* err) {
     extern __shared__ __align__(16) unsigned char raw[];
     __nv_bfloat16* qs = reinterpret_cast<__nv_bfloat16*>(raw);  // [ROWS][LDK]
     __nv_bfloat16* ks = qs + ROWS * LDK;                        // [2][KEYS][LDK]
@@ -199,6 +218,22 @@ sink_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat
     // sink's term of the sum is counted by the first thread of the four that share a row
     const float sl2 = scale * LOG2E;
     const float cap_in = softcap > 0.f ? scale / softcap : 0.f, cap_out = softcap * LOG2E;
+    // BIAS: the two rows' numbers.  1: r1 (in units of log2 e of ln: the factor of log2) and r2; 2: the
+    // table row and its last entry (in units of log2 e).
+    float r1_a = 0.f, r1_b = 0.f, r2_a = 0.f, r2_b = 0.f;
+    const float *tab_a = nullptr, *tab_b = nullptr;
+    if constexpr (BIAS != 0) {
+        int h_a = r_a < rows_here ? row_head(r_a) : 0, h_b = r_b < rows_here ? row_head(r_b) : 0;
+        if constexpr (BIAS == 1) {
+            r1_a = log_r1[h_a]; r1_b = log_r1[h_b];
+            r2_a = log_r2[h_a]; r2_b = log_r2[h_b];
+        } else {
+            tab_a = bias_table + (size_t)h_a * bias_len;
+            tab_b = bias_table + (size_t)h_b * bias_len;
+            r1_a = tab_a[bias_len - 1] * LOG2E;
+            r1_b = tab_b[bias_len - 1] * LOG2E;
+        }
+    }
     const bool with_sink = sinks != nullptr && !split_mode;  // (split: the merge adds the sink's term)
     float sink2 = with_sink ? sinks[head] * LOG2E : -INFINITY;
     float m_a = sink2, m_b = sink2;
@@ -228,19 +263,53 @@ sink_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat
         }
         // scores in units of log2 e, -inf where the key is not visible; the rows' new maxima
         float mx_a = m_a, mx_b = m_b;
+        if constexpr (BIAS == 0) {
 #pragma unroll
-        for (int nt = 0; nt < KEYS / 8; ++nt) {
-            int kp = t * KEYS + nt * 8 + t4 * 2;
+            for (int nt = 0; nt < KEYS / 8; ++nt) {
+                int kp = t * KEYS + nt * 8 + t4 * 2;
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                int key_pos = kp + (e & 1);
-                int pos = e < 2 ? pos_a : pos_b, lo = e < 2 ? lo_a : lo_b;
-                bool visible = key_pos <= pos && (key_pos >= lo || key_pos < keep_first);
-                float sc = softcap > 0.f ? cap_out * tanh_fast(s[nt][e] * cap_in) : s[nt][e] * sl2;
-                s[nt][e] = visible ? sc : -INFINITY;
+                for (int e = 0; e < 4; ++e) {
+                    int key_pos = kp + (e & 1);
+                    int pos = e < 2 ? pos_a : pos_b, lo = e < 2 ? lo_a : lo_b;
+                    bool visible = key_pos <= pos && (key_pos >= lo || key_pos < keep_first);
+                    float sc = softcap > 0.f ? cap_out * tanh_fast(s[nt][e] * cap_in) : s[nt][e] * sl2;
+                    s[nt][e] = visible ? sc : -INFINITY;
+                }
+                mx_a = fmaxf(mx_a, fmaxf(s[nt][0], s[nt][1]));
+                mx_b = fmaxf(mx_b, fmaxf(s[nt][2], s[nt][3]));
             }
-            mx_a = fmaxf(mx_a, fmaxf(s[nt][0], s[nt][1]));
-            mx_b = fmaxf(mx_b, fmaxf(s[nt][2], s[nt][3]));
+        } else {
+            // (the first query of the block is the one nearest to the tile)
+            const bool whole = window == 0 && t * KEYS + KEYS - 1 <= first_pos;
+            const bool all_far = BIAS == 2 && first_pos - (t * KEYS + KEYS - 1) >= bias_len - 1;
+#pragma unroll
+            for (int nt = 0; nt < KEYS / 8; ++nt) {
+                int kp = t * KEYS + nt * 8 + t4 * 2;
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    int key_pos = kp + (e & 1);
+                    int dist = (e < 2 ? pos_a : pos_b) - key_pos;
+                    float sc = s[nt][e] * sl2;
+                    if (softcap > 0.f) sc = cap_out * tanh_fast(s[nt][e] * cap_in);
+                    if constexpr (BIAS == 1) {
+                        // -r1 ln(1 + r2 n) in units of log2 e is -r1 log2(1 + r2 n)
+                        float n = (float)max(dist, 0);
+                        sc = fmaf(-(e < 2 ? r1_a : r1_b), log2_fast(fmaf(e < 2 ? r2_a : r2_b, n, 1.0f)), sc);
+                    } else if (all_far) {
+                        sc += e < 2 ? r1_a : r1_b;
+                    } else {
+                        sc = fmaf(__ldg((e < 2 ? tab_a : tab_b) + min(max(dist, 0), bias_len - 1)), LOG2E, sc);
+                    }
+                    if (!whole) {
+                        int lo = e < 2 ? lo_a : lo_b;
+                        bool visible = dist >= 0 && (key_pos >= lo || key_pos < keep_first);
+                        sc = visible ? sc : -INFINITY;
+                    }
+                    s[nt][e] = sc;
+                }
+                mx_a = fmaxf(mx_a, fmaxf(s[nt][0], s[nt][1]));
+                mx_b = fmaxf(mx_b, fmaxf(s[nt][2], s[nt][3]));
+            }
         }
         mx_a = quad_max(mx_a);
         mx_b = quad_max(mx_b);
@@ -305,7 +374,7 @@ sink_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat
         return;
     }
     float f_a = l_a > 0.f ? 1.0f / l_a : 0.f, f_b = l_b > 0.f ? 1.0f / l_b : 0.f;
-    if (out_gate != nullptr) {
+    if (out_gate != nullptr && !gate_elements) {
         if (pos_a >= 0) f_a *= 1.0f / (1.0f + expf(-out_gate[(size_t)(q0 + row0 + r_a) * gate_ld + head]));
         if (pos_b >= 0) f_b *= 1.0f / (1.0f + expf(-out_gate[(size_t)(q0 + row0 + r_b) * gate_ld + head]));
     }
@@ -314,6 +383,18 @@ sink_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat
 #pragma unroll
     for (int nt = 0; nt < DV / 8; ++nt) {
         int c = nt * 8 + t4 * 2;
+        if (out_gate != nullptr && gate_elements) {
+            if (pos_a >= 0) {
+                const float* gr = out_gate + (size_t)(q0 + row0 + r_a) * gate_ld + (size_t)head * DV + c;
+                o[nt][0] *= sigmoid_of(gr[0]);
+                o[nt][1] *= sigmoid_of(gr[1]);
+            }
+            if (pos_b >= 0) {
+                const float* gr = out_gate + (size_t)(q0 + row0 + r_b) * gate_ld + (size_t)head * DV + c;
+                o[nt][2] *= sigmoid_of(gr[0]);
+                o[nt][3] *= sigmoid_of(gr[1]);
+            }
+        }
         if (pos_a >= 0) *reinterpret_cast<unsigned*>(out_a + c) = pack_bf16(o[nt][0] * f_a, o[nt][1] * f_a);
         if (pos_b >= 0) *reinterpret_cast<unsigned*>(out_b + c) = pack_bf16(o[nt][2] * f_b, o[nt][3] * f_b);
     }
@@ -325,7 +406,8 @@ constexpr int MERGE_MAX_SPLITS = 1024;
 __global__ void __launch_bounds__(128)
 sink_attention_merge_kernel(const float* __restrict__ partial, const int* __restrict__ cu_q, int num_seqs,
                             __nv_bfloat16* __restrict__ out, int heads, int splits,
-                            const float* __restrict__ sinks, const float* __restrict__ out_gate, int gate_ld) {
+                            const float* __restrict__ sinks, const float* __restrict__ out_gate, int gate_ld,
+                            int gate_elements) {
     ie_pdl_trigger();
     ie_pdl_wait();
     int token = blockIdx.x / heads, head = blockIdx.x - token * heads;
@@ -360,11 +442,15 @@ sink_attention_merge_kernel(const float* __restrict__ partial, const int* __rest
         }
     }
     float f = l > 0.f ? 1.0f / l : 0.f;
-    if (out_gate != nullptr) f *= 1.0f / (1.0f + expf(-out_gate[(size_t)token * gate_ld + head]));
+    if (out_gate != nullptr && !gate_elements) f *= 1.0f / (1.0f + expf(-out_gate[(size_t)token * gate_ld + head]));
 #pragma unroll
     for (int i = 0; i < (DV + 127) / 128; ++i) {
         int c = i * 128 + threadIdx.x;
-        if (c < DV) out[((size_t)token * heads + head) * DV + c] = __float2bfloat16_rn(acc[i] * f);
+        if (c >= DV) continue;
+        float v = acc[i] * f;
+        if (out_gate != nullptr && gate_elements)
+            v *= sigmoid_of(out_gate[(size_t)token * gate_ld + (size_t)head * DV + c]);
+        out[((size_t)token * heads + head) * DV + c] = __float2bfloat16_rn(v);
     }
 }
 }  // namespace
@@ -372,7 +458,7 @@ sink_attention_merge_kernel(const float* __restrict__ partial, const int* __rest
 IE_API int ie_sink_attention_dims(int* d, int* dv) {
     *d = D;
     *dv = DV;
-    return 0;
+    return BIAS;
 }
 
 IE_API int ie_sink_attention_mma(const void* q, const void* k_cache, const void* v_cache, const int* block_tables,
@@ -380,12 +466,17 @@ IE_API int ie_sink_attention_mma(const void* q, const void* k_cache, const void*
                                  int max_q_len, int heads, int kv_heads, int page_size, int total_pages,
                                  float scale, int window, const float* sinks, const float* out_gate, int gate_ld,
                                  float* partial, int splits, int tiles_per_split, int num_tokens, float softcap,
-                                 int keep_first, int kept_splits, int* err, void* stream) {
+                                 int keep_first, int kept_splits, int gate_elements, const float* log_r1,
+                                 const float* log_r2, const float* bias_table, int bias_len, int* err,
+                                 void* stream) {
     if (num_seqs <= 0 || max_q_len <= 0) return 0;
     if (kv_heads <= 0 || heads % kv_heads != 0 || page_size < 1 || (page_size & (page_size - 1)) || window < 0)
         return (int)cudaErrorInvalidValue;
     if (softcap < 0.f || keep_first < 0 || kept_splits < 0 || (window == 0 && keep_first > 0))
         return (int)cudaErrorInvalidValue;
+    if ((BIAS == 1) != (log_r1 != nullptr && log_r2 != nullptr) || (BIAS == 2) != (bias_table != nullptr) ||
+        (BIAS == 2 && bias_len < 1))
+        return (int)cudaErrorInvalidValue;  // (the library was built for another kind of bias)
     size_t smem = (size_t)(ROWS * LDK + 2 * KEYS * LDK + 2 * KEYS * LDV) * sizeof(__nv_bfloat16);
     static IePerDevice allowed;
     cudaError_t e = ie_allow_smem(allowed, sink_attention_mma_kernel, smem);
@@ -400,15 +491,17 @@ IE_API int ie_sink_attention_mma(const void* q, const void* k_cache, const void*
                            (cudaStream_t)stream, (const __nv_bfloat16*)q, (const __nv_bfloat16*)k_cache,
                            (const __nv_bfloat16*)v_cache, block_tables, table_width, cu_q, ctx_lens, (__nv_bfloat16*)out,
                            heads, kv_heads, page_size, total_pages, scale, window, sinks, out_gate, gate_ld, partial,
-                           splits, tiles_per_split, softcap, keep_first, kept_splits, err);
+                           splits, tiles_per_split, softcap, keep_first, kept_splits, gate_elements, log_r1, log_r2,
+                           bias_table, bias_len, err);
         if (rc != 0) return rc;
         return ie_launch(sink_attention_merge_kernel, dim3(num_tokens * heads), dim3(128), 0, (cudaStream_t)stream,
                          (const float*)partial, cu_q, num_seqs, (__nv_bfloat16*)out, heads, splits, sinks, out_gate,
-                         gate_ld);
+                         gate_ld, gate_elements);
     }
     dim3 grid((max_q_len + ROWS - 1) / ROWS, heads, num_seqs);
     return ie_launch(sink_attention_mma_kernel, grid, dim3(THREADS), smem, (cudaStream_t)stream,
                      (const __nv_bfloat16*)q, (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache, block_tables,
                      table_width, cu_q, ctx_lens, (__nv_bfloat16*)out, heads, kv_heads, page_size, total_pages, scale,
-                     window, sinks, out_gate, gate_ld, (float*)nullptr, 1, 0, softcap, keep_first, 0, err);
+                     window, sinks, out_gate, gate_ld, (float*)nullptr, 1, 0, softcap, keep_first, 0,
+                     gate_elements, log_r1, log_r2, bias_table, bias_len, err);
 }

@@ -161,14 +161,18 @@ def build_sigmoid_attention(dim: int, vdim: int) -> Path:
                          [f"-DSA_D={dim}", f"-DSA_DV={vdim}"])
 
 
-def build_sink_attention(dim: int, vdim: int) -> Path:
-    """The tensor-core softmax attention with a sink, a window and head gates for one pair of key and
-    value sizes (compiled on first use for the sizes the loaded model has)."""
+DISTANCE_BIAS = {"none": 0, "log": 1, "table": 2}  # what the softmax attention adds to a score by distance
+
+
+def build_sink_attention(dim: int, vdim: int, bias: str = "none") -> Path:
+    """The tensor-core softmax attention with a sink, a window, output gates and a bias by distance of
+    one kind for one pair of key and value sizes (compiled on first use for what the loaded model has)."""
     if dim % 16 or vdim % 16 or not 16 <= dim <= 256 or not 16 <= vdim <= 256:
         raise BuildError(f"the tensor-core sink attention takes sizes that are multiples of 16 up to 256, "
                          f"not {dim} and {vdim}")
-    return build_library(f"ie_b200_sinkattn_d{dim}_v{vdim}", ["sink_attention_mma.cu"],
-                         [f"-DSK_D={dim}", f"-DSK_DV={vdim}"])
+    kind = DISTANCE_BIAS[bias]
+    return build_library(f"ie_b200_sinkattn_d{dim}_v{vdim}" + (f"_b{kind}" if kind else ""), ["sink_attention_mma.cu"],
+                         [f"-DSK_D={dim}", f"-DSK_DV={vdim}"] + ([f"-DSK_BIAS={kind}"] if kind else []))
 
 
 # Kernels only some mixers and feed-forwards need, each a library of its own that is built the
@@ -183,6 +187,8 @@ PART_LIBRARIES = {
     "recurrent": ["gated_recurrence.cu"],
     # attention with normalised queries and keys and sigmoid weights: the input stage
     "gated_attn": ["gated_attention.cu"],
+    # several residual streams mixed and read by every sublayer, and the norm without statistics
+    "streams": ["residual_streams.cu"],
 }
 
 
@@ -199,7 +205,8 @@ def build_all(prune: bool = True) -> list[Path]:
     with ThreadPoolExecutor(max_workers=os.cpu_count() or 2) as pool:
         libs += list(pool.map(build_attention, ATTENTION_HEAD_DIMS))
         libs += list(pool.map(build_part_library, PART_LIBRARIES))
-        libs += [build_sigmoid_attention(64, 64), build_sink_attention(64, 64)]
+        libs += [build_sigmoid_attention(64, 64), build_sink_attention(64, 64),
+                 build_sink_attention(64, 64, "log"), build_sink_attention(64, 64, "table")]
     if prune:
         keep = {lib.name for lib in libs}
         for old in build_dir().glob("libie_b200_*.so"):

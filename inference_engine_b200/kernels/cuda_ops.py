@@ -86,7 +86,7 @@ def _kind(name):
                     timer.end(span)
                 if nvtx:
                     self.torch.cuda.nvtx.range_pop()
-        call.__name__, call.__doc__ = method.__name__, method.__doc__
+        call.__name__, call.__doc__, call.__wrapped__ = method.__name__, method.__doc__, method
         return call
     return decorate
 
@@ -99,6 +99,18 @@ def _dtype_code(t) -> int:
     if t.dtype == torch.bfloat16:
         return 1
     raise KernelError(f"kernels take float32 or bfloat16 tensors, not {t.dtype}")
+
+
+class _BufferEnd:
+    """A workspace as a matrix product sees it that hands out the rows behind the first ``before`` ones of
+    the buffer asked for; ``whole`` is the buffer with them."""
+
+    def __init__(self, ws, before: int) -> None:
+        self.ws, self.before, self.whole = ws, before, None
+
+    def buffer(self, name, rows, cols, dtype, rows_cap=0):
+        self.whole = self.ws.buffer(name, self.before + rows, cols, dtype, rows_cap)
+        return self.whole[self.before:]
 
 
 class CudaOps:
@@ -125,7 +137,7 @@ class CudaOps:
         self._attn_libs: dict[int, object] = {}
         self._part_libs: dict[str, object] = {}
         self._sigattn_libs: dict[tuple[int, int], object] = {}
-        self._sinkattn_libs: dict[tuple[int, int], object] = {}
+        self._sinkattn_libs: dict[tuple[int, int, str], object] = {}
         self.sink_mma = os.environ.get("IE_B200_SINK_MMA", "1") != "0"  # tensor-core sink attention
         # residual gates' products as partial sums: faster by themselves, slower inside a captured step
         self.gate_split = os.environ.get("IE_B200_GATE_SPLIT", "0") == "1"
@@ -203,7 +215,7 @@ class CudaOps:
     def _declare(self) -> None:
         P, I, F, L = c_void_p, c_int, c_float, ctypes.c_longlong
         sigs = {
-            "ie_embedding": [P, I, P, P, I, I, I, F, P, P],
+            "ie_embedding": [P, I, P, P, I, I, I, F, I, P, P],
             "ie_rmsnorm": [P, P, I, L, F, P, F, P, I, P, I, I, P],
             "ie_layernorm": [P, P, I, L, F, P, F, P, I, P, I, I, P],
             "ie_add_position_rows": [P, P, I, P, I, I, I, P, P],
@@ -217,7 +229,7 @@ class CudaOps:
             "ie_gemm_tma_bf16": [P, P, P, I, I, I, I, I, I, P, P],
             "ie_gemm_tc5_bf16": [P, P, P, I, I, I, I, I, I, P, P],
             "ie_gemm_tc5_ok": [I, I, I],
-            "ie_paged_attention_generic": [P, P, P, I, P, I, P, P, P, I, I, I, I, I, I, I, I, F, I, I, P, P, P, I, F, I, P, P],
+            "ie_paged_attention_generic": [P, P, P, I, P, I, P, P, P, I, I, I, I, I, I, I, I, F, I, I, P, P, P, I, F, I, I, P, P, P, I, P, P],
             "ie_sample": [P, I, I, P, P, P, P, P, P, I, P, P, P, P, P],
             "ie_bigram_embedding": [P, P, I, P, P, P, P, P, P, L, I, P, I, I, I, I, L, L, P, P],
             "ie_sandwich_norm": [P, P, I, L, P, I, L, P, P, P, F, P, F, P, I, P, I, I, P],
@@ -305,11 +317,11 @@ class CudaOps:
     # --- kernels ----------------------------------------------------------------------------
 
     @_kind("embedding")
-    def embedding(self, table, ids, out, scale: float = 1.0) -> None:
-        """``out[n] = table[ids[n]] * scale`` as 32-bit rows."""
+    def embedding(self, table, ids, out, scale: float = 1.0, copies: int = 1) -> None:
+        """``out[n] = table[ids[n]] * scale`` as 32-bit rows (``copies`` of it next to each other)."""
         self._check(self._embedding(table.data_ptr(), _dtype_code(table), ids.data_ptr(),
                                     out.data_ptr(), ids.shape[0], table.shape[1], table.shape[0],
-                                    float(scale), self._err_ptr, self._stream()), "embedding")
+                                    float(scale), int(copies), self._err_ptr, self._stream()), "embedding")
 
     @staticmethod
     def _partials(t) -> tuple[int, int]:
@@ -405,10 +417,14 @@ class CudaOps:
         return parts
 
     @_kind(lambda kwargs: "linear:" + kwargs.get("tag", "linear"))
-    def linear(self, x, w, out=None, *, ws=None, tag="linear", out_dtype=None, allow_split=False):
+    def linear(self, x, w, out=None, *, ws=None, tag="linear", out_dtype=None, allow_split=False, slices_before=0):
         """``x[M, K] @ w[N, K]^T``.  With ``out`` given the product is written there; otherwise a
         buffer named ``tag`` is taken from ``ws``.  With ``allow_split`` the result may come back
-        as ``[S, M, N]`` partial sums (32-bit) that the consumer adds in order."""
+        as ``[S, M, N]`` partial sums (32-bit) that the consumer adds in order.  With ``slices_before``
+        the result is ``[slices_before + S, M, N]`` and the product's parts are its last S slices: the
+        others are the caller's to write (another sublayer's parts that are added with these)."""
+        if slices_before:
+            return self._linear_behind(x, w, ws, tag, slices_before)
         torch = self.torch
         m, k = x.shape
         n = w.shape[0]
@@ -477,6 +493,13 @@ class CudaOps:
         else:
             torch.mm(x, w.t(), out_dtype=out.dtype, out=out)
         return out
+
+    def _linear_behind(self, x, w, ws, tag, before: int):
+        """A 32-bit product whose parts follow ``before`` free slices of one buffer."""
+        m, n = x.shape[0], w.shape[0]
+        end = _BufferEnd(ws, before * m)
+        CudaOps.linear.__wrapped__(self, x, w, ws=end, tag=tag, out_dtype=self.torch.float32, allow_split=True)
+        return end.whole.view(-1, m, n)
 
     @_kind("rotary+cache")
     def rope_kv_write(self, qkv, positions, table, rotary_dim, q_out, k_cache, v_cache,
@@ -870,6 +893,8 @@ class CudaOps:
             ctx.num_seqs, tiles, nh, nkv, page_size, total_pages, scale, window,
             self._err_ptr, stream), "attention_prefill")
 
+    _NO_BIAS = (0, None, None, None, 0)  # (one gate per head, no bias by distance: the general kernel's last parameters)
+
     @_kind("attention.general")
     def paged_attention_general(self, q, k_cache, v_cache, block_tables, ctx, nh, nkv, hd,
                                 page_size, scale, window, out) -> None:
@@ -877,7 +902,8 @@ class CudaOps:
             q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), _dtype_code(q),
             block_tables.data_ptr(), block_tables.shape[1], ctx.seq_of_token.data_ptr(),
             ctx.positions.data_ptr(), out.data_ptr(), ctx.num_tokens, nh, nkv, hd, hd, hd, page_size,
-            k_cache.shape[0], scale, window, 0, None, None, None, 0, 0.0, 0, self._err_ptr, self._stream()), "paged_attention")
+            k_cache.shape[0], scale, window, 0, None, None, None, 0, 0.0, 0, *self._NO_BIAS, self._err_ptr,
+            self._stream()), "paged_attention")
 
     @_kind("attention.latent")
     def latent_paged_attention(self, q, k_cache, v_cache, block_tables, ctx, nh, nkv, hd, value_dim,
@@ -913,7 +939,7 @@ class CudaOps:
             block_tables.data_ptr(), block_tables.shape[1], ctx.seq_of_token.data_ptr(),
             ctx.positions.data_ptr(), out.data_ptr(), ctx.num_tokens, nh, nkv, hd, value_dim,
             v_cache.shape[-1], page_size, k_cache.shape[0], scale, window, 0, None, None, None, 0, 0.0, 0,
-            self._err_ptr, self._stream()), "paged_attention_latent")
+            *self._NO_BIAS, self._err_ptr, self._stream()), "paged_attention_latent")
 
     # --- kernels of single mixers and feed-forwards (libraries built on first use) -------------
 
@@ -942,12 +968,16 @@ class CudaOps:
             "ie_short_conv_residual": "P I P P L P P P P I I I I I P P",
             "ie_hgrn2_gates": "P I P P P I I P",
             "ie_mlstm_gates": "P P I P P F P L L P P P I I I P",
-            "ie_gated_recurrence": "P I P I P I P P I P L P P P I I I I I F I P",
+            "ie_gated_recurrence": "P I P I P I P I P I P L P P P I I I I I F I P",
+            "ie_rotate_heads": "P I P P I I I I I P P",
             "ie_recurrence_readout": "P I P P I F P I I P I L I I P",
             "ie_lowrank_decay": "P I P P F P I I I P",
         },
         "gated_attn": {
-            "ie_qk_norm_rope_write": "P I P P I I P I I I P P F P P P I P I I I I I I I P P",
+            "ie_qk_norm_rope_write": "P I P P I I P I I I P P F I P F I P P P I P I I I I I I I P P",
+        },
+        "streams": {
+            "ie_stream_mix_norm": "P I P I L P P P P P P F P I P I I P",
         },
     }
 
@@ -1060,9 +1090,10 @@ class CudaOps:
             ids.shape[1], groups, keep, 1 if scoring == "sigmoid" else 0, self._ptr(correction), int(group_top),
             float(weight_scale), ids.data_ptr(), weights.data_ptr(), self._stream()), "route_topk")
 
-    def routed_experts(self, x, ids, weights, w_gate_up, w_down, *, limit, alpha, up_offset, ws, tag="moe"):
+    def routed_experts(self, x, ids, weights, w_gate_up, w_down, *, limit, alpha, up_offset, ws, tag="moe", out=None):
         """The chosen experts' weighted outputs as ``[top, N, hidden]`` 32-bit slices (to be added in
-        order).  ``w_gate_up``: ``[experts, 2, ff, hidden]``, ``w_down``: ``[experts, hidden, ff]``."""
+        order).  ``w_gate_up``: ``[experts, 2, ff, hidden]``, ``w_down``: ``[experts, hidden, ff]``; ``out``: where
+        the slices go (contiguous), else a buffer from ``ws``."""
         torch = self.torch
         lib = self._part_lib("routed")
         n, top = ids.shape
@@ -1073,7 +1104,8 @@ class CudaOps:
         index = ws.buffer(tag + ".index", 1, rows + max_tiles + 4, torch.int32, rows_cap=None)[0]
         sorted_pairs, tile_expert, meta = index[:rows], index[rows: rows + max_tiles], index[rows + max_tiles:]
         y = ws.buffer(tag + ".act", pairs, ff, x.dtype)
-        out = ws.buffer(tag + ".delta", pairs, hidden, torch.float32).view(top, n, hidden)
+        if out is None:
+            out = ws.buffer(tag + ".delta", pairs, hidden, torch.float32).view(top, n, hidden)
         self._routed_align(lib, ids, pairs, experts, sorted_pairs, tile_expert, meta, max_tiles)
         self._routed_gate_up(lib, x, w_gate_up, y, sorted_pairs, tile_expert, meta, max_tiles, top, hidden, ff,
                              limit, alpha, up_offset)
@@ -1159,6 +1191,27 @@ class CudaOps:
                                        self._stream()), "weighted_sum")
 
     @_kind("norm")
+    def stream_mix_norm(self, h, streams, delta, mix, out_coef, read, weight, bias, alpha, eps, out, rows=None) -> None:
+        """``h``: ``[N, streams * width]``.  With a ``delta`` (``[N, width]``, or parts of it ``[S, N, width]``)
+        stream ``t`` becomes ``sum_s mix[s, t] x_s + out_coef[t] * delta``, all at once (not with ``rows``, which
+        selects rows and leaves ``h``); ``u = sum_t read[t] x_t`` of the new streams; ``out = tanh(alpha * u) *
+        weight + bias`` with an ``alpha`` (a one-element tensor), else ``rms(u) * weight``; ``out`` None: only
+        the streams are brought up to date.  ``mix`` None: the streams keep their values; ``out_coef`` or
+        ``read`` None: ones."""
+        width = h.shape[1] // streams
+        if h.shape[1] != streams * width or h.dtype != self.torch.float32 or not h.is_contiguous():
+            raise KernelError("stream_mix_norm: the streams are contiguous 32-bit rows")
+        if delta is not None and (delta.dtype != self.torch.float32 or tuple(delta.shape[-2:]) != (h.shape[0], width)
+                                  or not delta.is_contiguous()):
+            raise KernelError("stream_mix_norm: the sublayer's output must be 32-bit rows of one stream's width")
+        n = h.shape[0] if rows is None else rows.shape[0]
+        parts, stride = self._partials(delta)
+        self._check(self._part_lib("streams").ie_stream_mix_norm(
+            h.data_ptr(), streams, self._ptr(delta), parts, stride, self._ptr(mix), self._ptr(out_coef), self._ptr(read),
+            self._ptr(weight), self._ptr(bias), self._ptr(alpha), eps, self._ptr(out),
+            _dtype_code(out) if out is not None else 0, self._ptr(rows), n, width, self._stream()), "stream_mix_norm")
+
+    @_kind("norm")
     def gated_add_norm(self, h, delta, gate_pre, gate_bias, weight, eps, out, rows=None) -> None:
         """``h += sigmoid(gate_pre + gate_bias) * delta`` element by element (not with ``rows``, which
         selects rows and leaves ``h``); ``out = rms(h) * weight`` unless ``out`` is None.  ``delta`` may be
@@ -1227,29 +1280,41 @@ class CudaOps:
         """``S <- diag(a) S + w u^T; o = S^T q`` per head over every request's tokens of the step, from
         and to its slot (``[heads, cols, dim]``).  ``q``, ``a``, ``w``: views ``[N, heads * dim]``;
         ``v``: view ``[N, heads * vdim]``; with ``gates`` (``[N, heads, 3]``) ``a`` is the gates' decay,
-        ``u = gate * v``, and column ``vdim`` (if ``cols = vdim + 1``) carries the value 1."""
+        ``u = gate * v``, and column ``vdim`` (if ``cols = vdim + 1``) carries the value 1.  Gates of shape
+        ``[1, heads, 3]`` are every token's (a decay that is a constant per head)."""
         if dim > 512:
             raise KernelError(f"the recurrence kernel takes key sizes up to 512, not {dim}")
         self._check(self._part_lib("recurrent").ie_gated_recurrence(
             q.data_ptr(), q.stride(0), self._ptr(a), 0 if a is None else a.stride(0), w.data_ptr(), w.stride(0),
-            self._ptr(gates), v.data_ptr(), v.stride(0), state.data_ptr(), state.stride(0), slots.data_ptr(),
-            ctx.cu_q.data_ptr(), out.data_ptr(), ctx.num_seqs, heads, dim, vdim, cols, float(q_scale),
+            self._ptr(gates), 0 if gates is None or (gates.dim() == 3 and gates.shape[0] == 1) else 3 * heads,
+            v.data_ptr(), v.stride(0), state.data_ptr(), state.stride(0), slots.data_ptr(), ctx.cu_q.data_ptr(), out.data_ptr(), ctx.num_seqs, heads, dim, vdim, cols, float(q_scale),
             state.shape[0], self._stream()), "gated_recurrence")
 
     @_kind("recurrent.out")
     def recurrence_readout(self, o, gates, weight, eps, gate_pre, out, heads, vdim, cols, gate_act="sigmoid") -> None:
         """Per (token, head): with ``gates`` divide by ``max(|o[vdim]|, exp(-m)) + 1e-6``; divide by the
-        root mean square over ``vdim``; times ``weight`` (``[vdim]`` or ``[heads * vdim]``) and
+        root mean square over ``vdim``; times ``weight`` (``[vdim]``, ``[heads * vdim]`` or None) and
         ``sigmoid(gate_pre)`` (``gate_act="silu"``: ``silu(gate_pre)``; a view ``[N, heads * vdim]``) if given."""
         if gate_act not in ("sigmoid", "silu"):
             raise KernelError(f"recurrence_readout: no gate activation {gate_act!r}")
-        per_head = 1 if weight.numel() == heads * vdim and heads > 1 else 0
-        if weight.numel() not in (vdim, heads * vdim):
+        per_head = 1 if weight is not None and weight.numel() == heads * vdim and heads > 1 else 0
+        if weight is not None and weight.numel() not in (vdim, heads * vdim):
             raise KernelError("recurrence_readout: the weight fits neither a head nor all heads")
         self._check(self._part_lib("recurrent").ie_recurrence_readout(
-            o.data_ptr(), cols, self._ptr(gates), weight.data_ptr(), per_head, eps, self._ptr(gate_pre),
+            o.data_ptr(), cols, self._ptr(gates), self._ptr(weight), per_head, eps, self._ptr(gate_pre),
             0 if gate_pre is None else gate_pre.stride(0), 1 if gate_act == "silu" else 0, out.data_ptr(),
             _dtype_code(out), o.shape[0] * heads, heads, vdim, self._stream()), "recurrence_readout")
+
+    @_kind("recurrent.rotate")
+    def rotate_heads(self, x, positions, table, rot_dims, units, dim) -> None:
+        """The first ``rot_dims`` entries of each of the ``units`` heads of ``dim`` entries at the start of
+        ``x``'s rows (a 32-bit projection) are rotated in place by the token's position, by pairs
+        ``(i, i + rot_dims / 2)``."""
+        if x.dtype != self.torch.float32 or x.stride(1) != 1 or x.shape[1] < units * dim or table.shape[2] * 2 != rot_dims:
+            raise KernelError("rotate_heads: the heads or the table do not fit the 32-bit rows")
+        self._check(self._part_lib("recurrent").ie_rotate_heads(
+            x.data_ptr(), x.stride(0), positions.data_ptr(), table.data_ptr(), rot_dims, table.shape[0], x.shape[0],
+            units, dim, self._err_ptr, self._stream()), "rotate_heads")
 
     @_kind("recurrent.gates")
     def lowrank_decay(self, y, w2, bias, tau: float, decay) -> None:
@@ -1267,14 +1332,22 @@ class CudaOps:
     def qk_norm_rope_write(self, proj, positions, table, rot_dims, q_weight, k_weight, eps, q_out, k_cache,
                            v_cache, slot_mapping, heads, kv_heads, dim, vdim, page_size, bias=None,
                            value_norm: bool = False, values_from_keys: bool = False,
-                           interleaved: bool = False) -> None:
+                           interleaved: bool = False, unit_norm: bool = False, q_head_scale=None,
+                           warm_coef: float = 0.0, warm_every: int = 0) -> None:
         """The input stage of an attention with per-head norms (see ``csrc/gated_attention.cu``).
         ``q_weight`` / ``k_weight`` None: queries and keys are not normalised; ``bias``: one row laid
         out like the projection's first columns, added first; ``value_norm``: value heads are divided
         by their root mean square.  ``proj`` may hold more columns behind the values.
         ``values_from_keys``: the projection holds queries and keys only, and the cached values are
         the keys as projected (with their bias, before any norm or rotation).  ``interleaved``: the
-        rotation pairs entry ``2i`` with ``2i + 1`` instead of ``i`` with ``i + rot_dims / 2``."""
+        rotation pairs entry ``2i`` with ``2i + 1`` instead of ``i`` with ``i + rot_dims / 2``.
+        ``unit_norm`` (without weights): queries and keys are divided by their root mean square.
+        ``q_head_scale`` (32-bit, one per head) multiplies the query heads; with ``warm_every`` > 0 the
+        queries at position ``p`` are multiplied by ``1 + warm_coef * ln(floor((p + 1) / warm_every) + 1)``."""
+        if unit_norm and q_weight is not None:
+            raise KernelError("qk_norm_rope_write: a norm with weights or one without, not both")
+        if q_head_scale is not None and (q_head_scale.dtype != self.torch.float32 or q_head_scale.numel() != heads):
+            raise KernelError("qk_norm_rope_write: the queries' scale is one 32-bit number per head")
         if table is not None and table.shape[2] * 2 != rot_dims:
             raise KernelError("rotary table does not match the rotated dims")
         if values_from_keys and vdim != dim:
@@ -1288,7 +1361,8 @@ class CudaOps:
             proj.data_ptr(), proj.stride(0), positions.data_ptr(), self._ptr(table), rot_dims,
             0 if table is None else table.shape[0], self._ptr(bias), 1 if value_norm else 0,
             1 if values_from_keys else 0, 1 if interleaved else 0,
-            self._ptr(q_weight), self._ptr(k_weight), eps, q_out.data_ptr(),
+            self._ptr(q_weight), self._ptr(k_weight), eps, 1 if unit_norm else 0, self._ptr(q_head_scale),
+            float(warm_coef), int(warm_every), q_out.data_ptr(),
             k_cache.data_ptr(), v_cache.data_ptr(), _dtype_code(q_out), self._ptr(slot_mapping), proj.shape[0],
             heads, kv_heads, dim, vdim, page_size, k_cache.shape[0], self._err_ptr, self._stream()),
             "qk_norm_rope_write")
@@ -1332,22 +1406,22 @@ class CudaOps:
             q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), _dtype_code(q),
             block_tables.data_ptr(), block_tables.shape[1], ctx.seq_of_token.data_ptr(),
             ctx.positions.data_ptr(), out.data_ptr(), ctx.num_tokens, nh, nkv, hd, vdim, vdim, page_size,
-            k_cache.shape[0], scale, 0, int(chunk or 0), head_bias.data_ptr(), None, None, 0, 0.0, 0, self._err_ptr,
-            self._stream()), "sigmoid_attention")
+            k_cache.shape[0], scale, 0, int(chunk or 0), head_bias.data_ptr(), None, None, 0, 0.0, 0, *self._NO_BIAS,
+            self._err_ptr, self._stream()), "sigmoid_attention")
 
-    def _sink_attention_lib(self, hd: int, vdim: int):
-        lib = self._sinkattn_libs.get((hd, vdim))
+    def _sink_attention_lib(self, hd: int, vdim: int, bias: str = "none"):
+        lib = self._sinkattn_libs.get((hd, vdim, bias))
         if lib is None:
-            path = build_sink_attention(hd, vdim)
+            path = build_sink_attention(hd, vdim, bias)
             try:
                 lib = ctypes.CDLL(str(path))
             except OSError as exc:
                 raise KernelError(f"the kernel library {path} could not be loaded: {exc}") from exc
             P, I, F = c_void_p, c_int, c_float
             lib.ie_sink_attention_mma.argtypes = [P, P, P, P, I, P, P, P, I, I, I, I, I, I, F, I, P, P, I, P, I, I, I,
-                                                  F, I, I, P, P]
+                                                  F, I, I, I, P, P, P, I, P, P]
             lib.ie_sink_attention_mma.restype = c_int
-            self._sinkattn_libs[(hd, vdim)] = lib
+            self._sinkattn_libs[(hd, vdim, bias)] = lib
         return lib
 
     # requests that bring at most so many tokens have their window's keys cut among blocks, each of
@@ -1357,7 +1431,8 @@ class CudaOps:
 
     @_kind("attention.sink")
     def sink_attention(self, q, k_cache, v_cache, block_tables, ctx, nh, nkv, hd, vdim, page_size, scale,
-                       window, sinks, gate, out, softcap: float | None = None, keep_first: int = 0) -> None:
+                       window, sinks, gate, out, softcap: float | None = None, keep_first: int = 0,
+                       log_bias=None, bias_table=None) -> None:
         """Softmax attention over the paged cache whose denominator also holds ``exp(sinks[head])`` (a
         term without key or value; ``sinks`` None: a plain softmax), over the latest ``window``
         positions (None or 0: all), with value rows of ``vdim`` entries; ``gate`` (a 32-bit view
@@ -1371,7 +1446,21 @@ class CudaOps:
         a prompt portion); 32-bit and other sizes the general kernel, whose order of operations
         does not depend on the batch.  ``softcap``: a score ``s`` becomes ``softcap * tanh(s / softcap)``
         before the softmax.  ``keep_first`` (with a window): the keys at positions below it stay visible
-        to every later query beside its window, at their own positions."""
+        to every later query beside its window, at their own positions.  ``gate`` may instead be a view
+        ``[N, heads * vdim]``: a sigmoid per head and value entry.  A bias by the distance ``n`` of query
+        and key joins the score: ``log_bias = (r1, r2)`` (a 32-bit number per head each) adds ``-r1 * ln(1 +
+        r2 * n)``, ``bias_table`` (32-bit ``[heads, L]``) adds entry ``min(n, L - 1)`` of the head's row."""
+        if log_bias is not None and bias_table is not None:
+            raise KernelError("sink_attention: one kind of bias by distance at a time")
+        for t in (*(log_bias or ()), *(() if bias_table is None else (bias_table,))):
+            if t.dtype != self.torch.float32 or not t.is_contiguous() or t.shape[0] != nh:
+                raise KernelError("sink_attention: a bias by distance is 32-bit, with an entry or a row per head")
+        kind = "log" if log_bias is not None else "table" if bias_table is not None else "none"
+        if gate is not None and gate.shape[1] not in (nh, nh * vdim):
+            raise KernelError("sink_attention: the gate is a number per head, or per head and value entry")
+        by_distance = (1 if gate is not None and gate.shape[1] != nh else 0,
+                       *((log_bias[0].data_ptr(), log_bias[1].data_ptr()) if log_bias is not None else (None, None)),
+                       self._ptr(bias_table), 0 if bias_table is None else bias_table.shape[1])
         if gate is not None and (gate.dtype != self.torch.float32 or gate.stride(1) != 1):
             raise KernelError("sink_attention: the output gate must be a 32-bit view with unit stride")
         cap = float(softcap or 0.0)
@@ -1380,7 +1469,7 @@ class CudaOps:
             raise KernelError("sink_attention: the cap of the scores and the kept keys cannot be negative")
         if (self.sink_mma and q.dtype == self.torch.bfloat16 and hd % 16 == 0 and vdim % 16 == 0
                 and 16 <= hd <= 256 and 16 <= vdim <= 256 and page_size & (page_size - 1) == 0):
-            lib = self._sink_attention_lib(hd, vdim)
+            lib = self._sink_attention_lib(hd, vdim, kind)
             bounds = getattr(ctx, "bounds", None)
             longest = bounds[0] if bounds is not None else ctx.max_q_len  # (a captured step: its token bound)
             scratch, splits, per_split, kept_splits = None, 1, 0, 0
@@ -1406,7 +1495,8 @@ class CudaOps:
                 block_tables.shape[1], ctx.cu_q.data_ptr(), ctx.ctx_lens.data_ptr(), out.data_ptr(), ctx.num_seqs,
                 longest, nh, nkv, page_size, k_cache.shape[0], scale, int(window or 0), self._ptr(sinks),
                 self._ptr(gate), 0 if gate is None else gate.stride(0), self._ptr(scratch), splits, per_split,
-                ctx.num_tokens, cap, keep, kept_splits if scratch is not None else 0, self._err_ptr, self._stream()),
+                ctx.num_tokens, cap, keep, kept_splits if scratch is not None else 0, *by_distance, self._err_ptr,
+                self._stream()),
                 "sink_attention_mma")
             if scratch is not None:  # (the call launched the merge kernel too)
                 self.launches += 1
@@ -1417,7 +1507,7 @@ class CudaOps:
             block_tables.data_ptr(), block_tables.shape[1], ctx.seq_of_token.data_ptr(),
             ctx.positions.data_ptr(), out.data_ptr(), ctx.num_tokens, nh, nkv, hd, vdim, vdim, page_size,
             k_cache.shape[0], scale, int(window or 0), 0, None, self._ptr(sinks), self._ptr(gate),
-            0 if gate is None else gate.stride(0), cap, keep, self._err_ptr, self._stream()), "sink_attention")
+            0 if gate is None else gate.stride(0), cap, keep, *by_distance, self._err_ptr, self._stream()), "sink_attention")
 
     @_kind("activation")
     def silu_mul(self, gate_up, out, interleave: int = 0) -> None:

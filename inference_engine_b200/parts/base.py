@@ -45,7 +45,8 @@ class WeightDecl:
     ``vector`` (scales and biases; used in 32-bit), ``table`` (rows gathered by index) or
     ``int_table`` (integers, kept as int32).
     ``init`` says how the random-weights mode draws it: ``normal`` is N(0, std),
-    ``ones_plus_normal`` is 1 + N(0, std), ``zeros`` and ``ones`` are constant.
+    ``ones_plus_normal`` is 1 + N(0, std), ``eye_plus_normal`` the unit matrix plus N(0, std), ``zeros`` and
+    ``ones`` are constant.
     """
 
     shape: tuple[int, ...]

@@ -23,6 +23,12 @@ feed-forward that starts with one product over its input carries its gate's rows
 feed_forward(h)`` with ``h = norm(x)``.  The two outputs stay apart (each whole or in the parts of a
 split product) and are added, with the mixer's output bias if it has one, in the kernel of the
 next norm: the mixer's output is the pending delta, the rest travels beside it (``output_post``).
+
+``hyper_residual``: several residual streams (hyper-connections).  A sublayer reads a weighted sum of
+the streams through its norm; then every stream becomes a weighted sum of the old streams plus its own
+multiple of the sublayer's output.  The coefficients are small tensors of each sublayer.  One kernel
+does a sublayer's mixing, the next one's reading and its norm (``StreamMix`` travels with the pending
+delta); at the model's end the final norm reads the streams' plain sum.
 """
 
 from __future__ import annotations
@@ -30,7 +36,7 @@ from __future__ import annotations
 import os
 
 from .base import Block, BuildEnv, CacheBinding, WeightDecl
-from .norm import AddedTerms, PostNorm, ResidualGate
+from .norm import AddedTerms, PostNorm, ResidualGate, StreamMix
 from .registry import build_part, register_part
 
 
@@ -246,3 +252,68 @@ class GatedPreNormResidualBlock(Block):
         out = self.feed_forward.forward(x, ctx)
         self._pending = ResidualGate(self.feed_forward.extra_out, self.gate_bias["feed_forward_gate"])
         return out
+
+
+@register_part("block", "hyper_residual")
+class HyperResidualBlock(Block):
+    """Norms ``pre_mixer`` and, with a feed-forward, ``pre_feed_forward``.  Parameters: ``streams`` and the
+    tensor names ``mixer`` and ``feed_forward``, each a mapping of ``in`` (``[streams]``, what the sublayer
+    reads), ``mix`` (``[streams, streams]``, from and to) and ``out`` (``[streams]``)."""
+
+    MAX_STREAMS = 16
+
+    def __init__(self, mixer, feed_forward, norms: dict, names: dict, streams: int) -> None:
+        _adds_no_output_bias(mixer)
+        if not 1 <= streams <= self.MAX_STREAMS:
+            raise ValueError(f"a model keeps between 1 and {self.MAX_STREAMS} residual streams, not {streams}")
+        self.mixer, self.feed_forward, self.norms = mixer, feed_forward, norms
+        self.names, self.streams = names, int(streams)
+        self.residual_mult = 1.0
+        self.read: dict = {}
+        self.write: dict = {}
+
+    @classmethod
+    def from_spec(cls, params: dict, env: BuildEnv, *, layer, **_):
+        has_ff = layer.feed_forward is not None
+        norms = {"mixer": build_part("norm", layer.norms["pre_mixer"], env)}
+        if has_ff:
+            norms["feed_forward"] = build_part("norm", layer.norms["pre_feed_forward"], env)
+        return cls(build_part("mixer", layer.mixer, env),
+                   build_part("feed_forward", layer.feed_forward, env) if has_ff else None,
+                   norms, {which: dict(params[which]) for which in norms}, params["streams"])
+
+    def parts(self):
+        return [*self.norms.values(), self.mixer] + ([self.feed_forward] if self.feed_forward is not None else [])
+
+    def weights(self) -> dict[str, WeightDecl]:
+        s, out = self.streams, {}
+        for names in self.names.values():
+            out[names["in"]] = WeightDecl((s,), "vector", "ones_plus_normal")
+            out[names["mix"]] = WeightDecl((s, s), "vector", "eye_plus_normal")
+            out[names["out"]] = WeightDecl((s,), "vector", "ones_plus_normal")
+        return out
+
+    def bind(self, tensors, env: BuildEnv) -> None:
+        for which, names in self.names.items():
+            self.read[which] = tensors[names["in"]].float().contiguous()
+            self.write[which] = StreamMix(self.streams, tensors[names["mix"]].float().contiguous(),
+                                          tensors[names["out"]].float().contiguous())
+
+    @property
+    def output_post(self) -> StreamMix:
+        """How this block's returned delta enters the streams."""
+        return self.write["mixer" if self.feed_forward is None else "feed_forward"]
+
+    def forward(self, h, delta, ctx, binding: CacheBinding | None, delta_scale: float = 1.0, delta_post=None):
+        if delta_post is None:
+            delta_post = StreamMix(self.streams)
+        if not isinstance(delta_post, StreamMix) or delta_post.streams != self.streams:
+            raise ValueError("the layers of a model with several residual streams all keep as many of them")
+        x = self.norms["mixer"].add_norm(h, delta, ctx, tag="norm.mixer", delta_scale=delta_scale,
+                                         delta_post=delta_post.reading(self.read["mixer"]))
+        mixed = self.mixer.forward(x, ctx, binding)
+        if self.feed_forward is None:
+            return mixed
+        x = self.norms["feed_forward"].add_norm(h, mixed, ctx, tag="norm.ffn",
+                                                delta_post=self.write["mixer"].reading(self.read["feed_forward"]))
+        return self.feed_forward.forward(x, ctx)

@@ -74,7 +74,9 @@ class SwiGLU(FeedForward):
             self.w_gate_up = torch.cat([gate, up]).contiguous()
         self.w_down = tensors[self.names["down"]].to(self.dtype).contiguous()
 
-    def forward(self, x, ctx):
+    def forward(self, x, ctx, slices_before: int = 0):
+        """``slices_before``: the result is ``[slices_before + parts, N, hidden]``, its first slices free for
+        the outputs of a feed-forward that is added with this one."""
         import torch
 
         if self.bias_gate_up is not None:
@@ -83,6 +85,11 @@ class SwiGLU(FeedForward):
             ctx.ops.silu_mul_bias(gate_up, self.bias_gate_up, act)
         else:
             act = ctx.ops.gated_linear(x, self.w_gate_up, self.interleave, ws=ctx.ws, tag="ffn", out_dtype=self.dtype)
+        if slices_before:
+            if self.output_bias is not None:
+                raise ValueError("a feed-forward beside others has no output bias")
+            return ctx.ops.linear(act, self.w_down, ws=ctx.ws, tag="ffn.delta", out_dtype=torch.float32,
+                                  allow_split=True, slices_before=slices_before)
         return ctx.ops.linear(act, self.w_down, ws=ctx.ws, tag="ffn.delta", out_dtype=torch.float32,
                               allow_split=True)
 

@@ -1,4 +1,5 @@
-"""Root-mean-square norm over the last dimension, with the residual add fused in.
+"""Norms over the last dimension, with the residual add fused in: root mean square, layer norm, dynamic
+tanh; and what may be done to a sublayer's output on its way into the residual stream or streams.
 
 Formula (engine/model/layers.py:41-43): ``normed = x * rsqrt(mean(x^2) + eps)`` in 32-bit,
 then ``weight * normed``.  The residual stream is kept in 32-bit here, so square, mean,
@@ -130,4 +131,62 @@ class LayerNorm(Norm):
         n = h.shape[0] if rows is None else rows.shape[0]
         out = ctx.ws.buffer(tag, n, self.size, self.dtype)
         ctx.ops.layernorm(h, delta, self.weight, self.eps, out, rows, delta_scale=float(delta_scale))
+        return out
+
+
+class StreamMix:
+    """Several residual streams side by side in a row of ``h`` (``[N, streams * width]``).  What a sublayer
+    returned enters all of them at once: ``x_t <- sum_s mix[s, t] x_s + out[t] * delta`` (``mix[from, to]``), and
+    what the next sublayer reads is ``sum_t read[t] x_t`` (no ``read``: the streams' plain sum, as at a
+    model's end).  Carried beside the pending delta to whoever adds it, like :class:`PostNorm`; the
+    mixing, the reading and the next norm are one kernel.  Without coefficients nothing is mixed."""
+
+    def __init__(self, streams: int, mix=None, out=None, read=None) -> None:
+        self.streams, self.mix, self.out, self.read = int(streams), mix, out, read
+
+    def reading(self, read) -> "StreamMix":
+        return StreamMix(self.streams, self.mix, self.out, read)
+
+    def add_norm(self, h, delta, ctx, weight, eps, out, rows, bias=None, alpha=None) -> None:
+        ctx.ops.stream_mix_norm(h, self.streams, delta, self.mix, self.out, self.read, weight, bias, alpha, eps, out,
+                                rows)
+
+    def settle(self, h, delta, ctx) -> None:
+        ctx.ops.stream_mix_norm(h, self.streams, delta, self.mix, self.out, None, None, None, None, 0.0, None)
+
+
+@register_part("norm", "dynamic_tanh")
+class DynamicTanh(Norm):
+    """``tanh(alpha * x) * weight + bias`` entry by entry: no mean, no variance.  ``alpha`` is one stored number.
+    32-bit throughout; the result is rounded once to the compute dtype."""
+
+    def __init__(self, weight: str, bias: str, alpha: str, size: int, dtype) -> None:
+        self.weight_name, self.bias_name, self.alpha_name = weight, bias, alpha
+        self.size, self.dtype = int(size), dtype
+        self.weight = self.bias = self.alpha = None
+
+    @classmethod
+    def from_spec(cls, params: dict, env: BuildEnv, **_):
+        return cls(params["weight"], params["bias"], params["alpha"], params.get("size", env.hidden_size),
+                   env.torch_dtype)
+
+    def weights(self) -> dict[str, WeightDecl]:
+        return {self.weight_name: WeightDecl((self.size,), "vector", "ones_plus_normal"),
+                self.bias_name: WeightDecl((self.size,), "vector"),
+                self.alpha_name: WeightDecl((), "vector", "ones_plus_normal")}
+
+    def bind(self, tensors, env: BuildEnv) -> None:
+        self.weight = tensors[self.weight_name].float().contiguous()
+        self.bias = tensors[self.bias_name].float().contiguous()
+        self.alpha = tensors[self.alpha_name].float().reshape(1).contiguous()
+
+    def add_norm(self, h, delta, ctx, rows=None, tag: str = "norm", delta_scale: float = 1.0, delta_post=None):
+        if delta_scale != 1.0:
+            raise ValueError("the tanh norm's kernel adds a delta without a residual multiplier")
+        post = delta_post if delta_post is not None else StreamMix(1)
+        if not isinstance(post, StreamMix):
+            raise ValueError(f"the tanh norm's kernel cannot treat a delta by {type(post).__name__}")
+        n = h.shape[0] if rows is None else rows.shape[0]
+        out = ctx.ws.buffer(tag, n, self.size, self.dtype)
+        post.add_norm(h, delta, ctx, self.weight, 0.0, out, rows, bias=self.bias, alpha=self.alpha)
         return out

@@ -24,6 +24,11 @@ square over ``vdim`` and multiplied by a weight of size ``vdim`` that the heads 
 together are multiplied by ``silu(W_g h)``; ``W_o``.  Its input product can carry more rows of another
 map of the same input (``accepts_input_rows``).
 
+``retention``: linear attention with one constant decay per head.  ``q = W_q h``, ``k = W_k h`` (both
+rotated by position, if a rotary encoding is named), ``v = W_v h``; ``S <- decay[head] S + k v^T``, ``o = S^T
+q * dim^-1/2``; each head's ``o`` is divided by its root mean square over ``vdim`` (no weight); the heads
+together are multiplied by ``silu(W_g h)``; ``W_o``.
+
 Gates, decays, the state and the read-out are 32-bit in every precision; the projections run in
 the compute dtype with 32-bit sums.  The state lives in the request's state slot: ``S`` column by
 column (``[heads, columns, dim]``; the normaliser is one more column), then the maxima.
@@ -264,3 +269,68 @@ class GatedLinearAttention(Mixer):
         ops.recurrence_readout(o, None, self.out_norm, self.eps, proj[:, at_g: at_a], out, self.heads, self.vdim,
                                self.vdim, gate_act="silu")
         return ops.linear(out, self.w_o, ws=ws, tag="gla.delta", out_dtype=f32, allow_split=self.allow_split)
+
+
+@register_part("mixer", "retention")
+class Retention(Mixer):
+    allow_split = True
+    accepts_input_rows = True
+
+    def __init__(self, *, names: dict, hidden_size: int, heads: int, dim: int, vdim: int, decay, eps: float, position,
+                 dtype) -> None:
+        decay = tuple(float(d) for d in decay)
+        if len(decay) != heads:
+            raise ValueError(f"one decay per head: {len(decay)} for {heads} heads")
+        if position is not None and getattr(position, "layout", "halves") != "halves":
+            raise ValueError("retention rotates pairs half a rotation's width apart")
+        self.names, self.hidden_size = dict(names), hidden_size
+        self.heads, self.dim, self.vdim, self.decay, self.eps = heads, dim, vdim, decay, float(eps)
+        self.position, self.dtype = position, dtype
+        self.qk_size, self.v_size = heads * dim, heads * vdim
+        self.w_in = self.gates = None
+
+    @classmethod
+    def from_spec(cls, params: dict, env: BuildEnv, **_):
+        return cls(names=params["names"], hidden_size=params.get("hidden_size", env.hidden_size),
+                   heads=params["heads"], dim=params["dim"], vdim=params["vdim"], decay=params["decay"],
+                   eps=params["eps"], position=env.positions[params["position"]] if params.get("position") else None,
+                   dtype=env.torch_dtype)
+
+    def weights(self) -> dict[str, WeightDecl]:
+        n, h = self.names, self.hidden_size
+        return {n["q"]: WeightDecl((self.qk_size, h)), n["k"]: WeightDecl((self.qk_size, h)),
+                n["v"]: WeightDecl((self.v_size, h)), n["g"]: WeightDecl((self.v_size, h)),
+                n["o"]: WeightDecl((h, self.v_size))}
+
+    def bind(self, tensors, env: BuildEnv) -> None:
+        import torch
+
+        n = self.names
+        self.w_in, self.extra_at = self._with_extra_rows([tensors[n[k]].to(self.dtype) for k in ("q", "k", "v", "g")])
+        self.w_o = tensors[n["o"]].to(self.dtype).contiguous()
+        # (decay, write gate, unused) per head, the same for every token
+        self.gates = torch.tensor([[[d, 1.0, 1.0] for d in self.decay]], dtype=torch.float32, device=self.w_o.device)
+
+    def cache_request(self) -> StateRequest:
+        return StateRequest((self.heads * self.vdim * self.dim,))
+
+    def forward(self, x, ctx, binding):
+        import torch
+
+        f32, n, qk, vs = torch.float32, x.shape[0], self.qk_size, self.v_size
+        group = ctx.groups[binding.group]
+        ops, ws = ctx.ops, ctx.ws
+        proj = ops.linear(x, self.w_in, ws=ws, tag="retention.in", out_dtype=f32)
+        self.extra_out = self._extra_columns(proj, self.extra_at)
+        at_g = 2 * qk + vs
+        if self.position is not None and self.position.rotary_dim:
+            ops.rotate_heads(proj, ctx.positions, self.position.rotary_table(), self.position.rotary_dim,
+                             2 * self.heads, self.dim)
+        o = ws.buffer("retention.o", n, vs, f32)
+        ops.gated_recurrence(proj[:, :qk], None, proj[:, qk: 2 * qk], self.gates, proj[:, 2 * qk: at_g],
+                             group.state[binding.slot], group.slots, ctx, o, self.heads, self.dim, self.vdim,
+                             self.vdim, self.dim ** -0.5)
+        out = ws.buffer("retention.out", n, vs, self.dtype)
+        ops.recurrence_readout(o, None, None, self.eps, proj[:, at_g: at_g + vs], out, self.heads, self.vdim,
+                               self.vdim, gate_act="silu")
+        return ops.linear(out, self.w_o, ws=ws, tag="retention.delta", out_dtype=f32, allow_split=self.allow_split)

@@ -15,6 +15,10 @@ An expert: ``g = min(gate(x), limit)``, ``u = clamp(up(x), -limit, limit)``,
 ``y = g * sigmoid(alpha * g) * (u + up_offset)``, output ``down(y)``; no biases.  ``limit``,
 ``alpha`` and ``up_offset`` are parameters (``limit=None``: nothing is clamped).
 
+``shared``: a feed-forward of its own (a part description) that every token passes; its output is one
+more slice, or the parts of a split product, behind the chosen experts' slices.  It must return its
+output from one last product that can be told where to go (``forward(x, ctx, slices_before)``).
+
 The experts' matrices are stacked (``[experts, 2, ff, hidden]`` gates then ups, and
 ``[experts, hidden, ff]``), a step's (token, expert) pairs are sorted by expert on the device, and
 two grouped products run over the sorted list; nothing about the routing is read by the host.  The
@@ -24,8 +28,9 @@ choice, and the next norm adds the slices in order, like the parts of a split ma
 
 from __future__ import annotations
 
+from ..config.spec import PartSpec
 from .base import BuildEnv, FeedForward, WeightDecl
-from .registry import register_part
+from .registry import build_part, register_part
 
 
 @register_part("feed_forward", "routed_experts")
@@ -33,7 +38,9 @@ class RoutedExperts(FeedForward):
     def __init__(self, *, router: str, expert_prefix: str, experts: int, top: int, groups: int,
                  keep_groups: int, hidden_size: int, intermediate_size: int, limit: float | None,
                  alpha: float, up_offset: float, dtype, router_bias: str | None = None, scoring: str = "softmax",
-                 correction: str | None = None, group_top: int = 1, weight_scale: float = 1.0) -> None:
+                 correction: str | None = None, group_top: int = 1, weight_scale: float = 1.0,
+                 shared: FeedForward | None = None) -> None:
+        self.shared = shared
         if not 1 <= top <= experts:
             raise ValueError(f"top ({top}) must be between 1 and the number of experts ({experts})")
         if groups < 1 or experts % groups or not 1 <= keep_groups <= groups:
@@ -58,6 +65,9 @@ class RoutedExperts(FeedForward):
 
     @classmethod
     def from_spec(cls, params: dict, env: BuildEnv, **_):
+        shared = params.get("shared")
+        if shared is not None and not isinstance(shared, PartSpec):
+            shared = PartSpec(shared["kind"], dict(shared.get("params", {})))
         return cls(router=params["router"], expert_prefix=params["expert_prefix"],
                    experts=params["experts"], top=params["top"], groups=params.get("groups", 1),
                    keep_groups=params.get("keep_groups", 1),
@@ -66,7 +76,11 @@ class RoutedExperts(FeedForward):
                    alpha=params.get("alpha", 1.702), up_offset=params.get("up_offset", 1.0),
                    dtype=env.torch_dtype, router_bias=params.get("router_bias"),
                    scoring=params.get("scoring", "softmax"), correction=params.get("correction"),
-                   group_top=params.get("group_top", 1), weight_scale=params.get("weight_scale", 1.0))
+                   group_top=params.get("group_top", 1), weight_scale=params.get("weight_scale", 1.0),
+                   shared=build_part("feed_forward", shared, env) if shared is not None else None)
+
+    def parts(self):
+        return [self.shared] if self.shared is not None else []
 
     def _name(self, e: int, which: str) -> str:
         return f"{self.expert_prefix}{e}.{which}"
@@ -114,6 +128,11 @@ class RoutedExperts(FeedForward):
             ctx.ops.route_topk(x, self.w_router, self.groups, self.keep_groups, ids, weights)
         else:
             ctx.ops.route_topk(x, self.w_router, self.groups, self.keep_groups, ids, weights, bias=self.router_bias)
-        return ctx.ops.routed_experts(x, ids, weights, self.w_gate_up, self.w_down,
-                                      limit=self.limit, alpha=self.alpha, up_offset=self.up_offset,
-                                      ws=ctx.ws, tag="moe")
+        if self.shared is None:
+            return ctx.ops.routed_experts(x, ids, weights, self.w_gate_up, self.w_down,
+                                          limit=self.limit, alpha=self.alpha, up_offset=self.up_offset,
+                                          ws=ctx.ws, tag="moe")
+        both = self.shared.forward(x, ctx, slices_before=self.top)  # [top + parts, N, hidden]
+        ctx.ops.routed_experts(x, ids, weights, self.w_gate_up, self.w_down, limit=self.limit, alpha=self.alpha,
+                               up_offset=self.up_offset, ws=ctx.ws, tag="moe", out=both[: self.top])
+        return both

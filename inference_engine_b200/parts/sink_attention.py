@@ -1,4 +1,5 @@
-"""Grouped-query softmax attention over the paged cache with a sink, a window and a gate per head.
+"""Grouped-query softmax attention over the paged cache with a sink, a window, output gates and a bias by
+distance.
 
 ``q = W_q h (+ b_q)``, ``k = W_k h (+ b_k)``, ``v = W_v h (+ b_v)``; value rows may have another size
 than key rows.  With ``value_norm`` each value head is divided by its root mean square over
@@ -20,9 +21,19 @@ every head instead of a learned tensor (0: the denominator's extra term is ``exp
 queries, at their own positions, and their pages are kept.  A rotary encoding of either layout
 (halves or interleaved pairs) on the first ``rotary_dim`` entries of each head.  ``o_bias`` among
 the names: a bias of the output projection, which the part leaves to whoever adds its output to the
-residual stream (``output_bias``).
+residual stream (``output_bias``).  ``unit_qk``: query and key heads are divided by their root mean
+square over ``dim`` (no weight).  ``temp`` among the names: a number per head that multiplies its scores
+(taken into the queries before they are rounded).  ``warmth = (coef, every)``: the queries at position
+``p`` are multiplied by ``1 + coef * ln(floor((p + 1) / every) + 1)``.  ``gate`` among the names, in
+place of a head gate: a sigmoid of a linear map of the input per head and value entry.
 
-Queries, keys, values and the head gates come from one matrix product over the row-concatenated
+A bias by the distance ``n`` of query and key, added to the score after scale and temperature: with
+``r1`` and ``r2`` among the names ``-r1[head] * ln(1 + r2[head] * n)``; with ``rel`` among them ``rel[bucket(n),
+head]`` from ``B`` rows: the distances below ``B / 2`` have a bucket each, the other buckets widen with
+the logarithm of the distance up to ``bias_max`` (:func:`distance_bucket`), and the last one holds
+everything farther.  The kernels read a table of the bias by distance up to where it is constant.
+
+Queries, keys, values and the gates come from one matrix product over the row-concatenated
 weights, which can carry more rows of another map of the same input (``accepts_input_rows``);
 biases, value norm and the cache write are one kernel; the gate is applied where the attention
 kernel writes its result.
@@ -30,8 +41,27 @@ kernel writes its result.
 
 from __future__ import annotations
 
+import math
+
 from .base import BuildEnv, CacheBinding, Mixer, PagedKVRequest, WeightDecl
 from .registry import register_part
+
+
+def distance_bucket(n: int, buckets: int, bias_max: float) -> int:
+    """The bucket of distance ``n``: ``n`` itself below half the buckets, then by the logarithm of the
+    distance, so that ``bias_max`` and everything beyond it fall into the last bucket."""
+    half = buckets // 2
+    if n < half or buckets == 1:
+        return min(n, buckets - 1)
+    return min(buckets - 1, half + math.floor(math.log(n / half) / math.log(bias_max / half) * (buckets - half)))
+
+
+def buckets_by_distance(buckets: int, bias_max: float) -> list[int]:
+    """The bucket of every distance up to the first from which on it stays the last one."""
+    out = [distance_bucket(0, buckets, bias_max)]
+    while out[-1] < buckets - 1:
+        out.append(distance_bucket(len(out), buckets, bias_max))
+    return out
 
 
 @register_part("mixer", "sink_attention")
@@ -42,7 +72,8 @@ class SinkAttention(Mixer):
     def __init__(self, *, names: dict, hidden_size: int, heads: int, kv_heads: int, dim: int, vdim: int,
                  scale: float, window: int | None, value_norm: bool, eps: float, position, dtype,
                  values: str = "projected", softcap: float | None = None, sink_value: float | None = None,
-                 keep_first: int = 0) -> None:
+                 keep_first: int = 0, unit_qk: bool = False, warmth: tuple | None = None,
+                 rel_buckets: int | None = None, bias_max: float | None = None) -> None:
         if heads % kv_heads:
             raise ValueError(f"heads ({heads}) not divisible by kv_heads ({kv_heads})")
         if window is not None and window < 1:
@@ -66,6 +97,22 @@ class SinkAttention(Mixer):
             raise ValueError("the sink is a learned tensor or a constant, not both")
         if keep_first < 0 or (keep_first and window is None):
             raise ValueError("first positions are kept beside a window, and there cannot be fewer than none")
+        if (names.get("r1") is None) != (names.get("r2") is None):
+            raise ValueError("the logarithmic bias needs both of its numbers per head")
+        if names.get("rel"):
+            if names.get("r1"):
+                raise ValueError("one kind of bias by distance at a time")
+            if not rel_buckets or rel_buckets < 1 or bias_max is None or not bias_max > rel_buckets // 2:
+                raise ValueError("the bucketed bias needs its number of buckets and a largest distance beyond half of them")
+        if names.get("gate") and names.get("head_gate"):
+            raise ValueError("a gate per head or one per value entry, not both")
+        if warmth is not None and int(warmth[1]) < 1:
+            raise ValueError("the queries' warmth steps up after at least one position")
+        self.unit_qk = bool(unit_qk)
+        self.warmth = (0.0, 0) if warmth is None else (float(warmth[0]), int(warmth[1]))
+        self.rel_buckets, self.bias_max = rel_buckets, bias_max
+        self.temp = self.log_bias = self.bias_table = None
+        self.gate_size = heads * vdim if names.get("gate") else heads if names.get("head_gate") else 0
         self.names = {k: v for k, v in names.items() if v}
         self.hidden_size, self.heads, self.kv_heads, self.dim, self.vdim = hidden_size, heads, kv_heads, dim, vdim
         self.scale, self.window, self.value_norm, self.eps = float(scale), window, bool(value_norm), float(eps)
@@ -84,7 +131,9 @@ class SinkAttention(Mixer):
                    scale=params["scale"], window=params.get("window"), value_norm=params.get("value_norm", False),
                    eps=params.get("eps", 1e-6), position=position, dtype=env.torch_dtype,
                    values=params.get("values", "projected"), softcap=params.get("softcap"),
-                   sink_value=params.get("sink_value"), keep_first=params.get("keep_first") or 0)
+                   sink_value=params.get("sink_value"), keep_first=params.get("keep_first") or 0,
+                   unit_qk=params.get("unit_qk", False), warmth=params.get("warmth"),
+                   rel_buckets=params.get("rel_buckets"), bias_max=params.get("bias_max"))
 
     def weights(self) -> dict[str, WeightDecl]:
         n, h = self.names, self.hidden_size
@@ -105,6 +154,13 @@ class SinkAttention(Mixer):
             out[n["sink"]] = WeightDecl((self.heads,), "vector")
         if "head_gate" in n:
             out[n["head_gate"]] = WeightDecl((self.heads, h))
+        if "gate" in n:
+            out[n["gate"]] = WeightDecl((self.heads * self.vdim, h))
+        for name in ("temp", "r1", "r2"):
+            if name in n:
+                out[n[name]] = WeightDecl((self.heads,), "vector", "ones_plus_normal")
+        if "rel" in n:
+            out[n["rel"]] = WeightDecl((self.rel_buckets, self.heads), "vector")
         return out
 
     def bind(self, tensors, env: BuildEnv) -> None:
@@ -114,12 +170,22 @@ class SinkAttention(Mixer):
         rows = [tensors[n[k]].to(self.dtype) for k in self.projected]
         if "head_gate" in n:
             rows.append(tensors[n["head_gate"]].to(self.dtype))
+        if "gate" in n:
+            rows.append(tensors[n["gate"]].to(self.dtype))
         self.w_in, self.extra_at = self._with_extra_rows(rows)
         self.w_o = tensors[n["o"]].to(self.dtype).contiguous()
         if "q_bias" in n:
             self.bias = torch.cat([tensors[n[k]].float() for k in self.bias_names]).contiguous()
         if "o_bias" in n:
             self.output_bias = tensors[n["o_bias"]].float().contiguous()
+        if "temp" in n:
+            self.temp = tensors[n["temp"]].float().contiguous()
+        if "r1" in n:
+            self.log_bias = tuple(tensors[n[r]].float().contiguous() for r in ("r1", "r2"))
+        if "rel" in n:
+            rel = tensors[n["rel"]].float()
+            index = torch.tensor(buckets_by_distance(self.rel_buckets, self.bias_max), device=rel.device)
+            self.bias_table = rel[index].t().contiguous()  # [heads, distances]
         if "sink" in n:
             self.sinks = tensors[n["sink"]].float().contiguous()
         elif self.sink_value is not None:
@@ -144,11 +210,14 @@ class SinkAttention(Mixer):
                                group.slot_mapping if binding.writes else None, self.heads, self.kv_heads,
                                self.dim, self.vdim, group.page_size, bias=self.bias, value_norm=self.value_norm,
                                values_from_keys=self.values_from_keys,
-                               interleaved=getattr(self.position, "layout", "halves") == "interleaved")
-        gate = proj[:, self.qkv_size: self.qkv_size + self.heads] if "head_gate" in self.names else None
+                               interleaved=getattr(self.position, "layout", "halves") == "interleaved",
+                               unit_norm=self.unit_qk, q_head_scale=self.temp, warm_coef=self.warmth[0],
+                               warm_every=self.warmth[1])
+        gate = proj[:, self.qkv_size: self.qkv_size + self.gate_size] if self.gate_size else None
         out = ws.buffer("sinkattn.out", n, self.heads * self.vdim, self.dtype)
         ops.sink_attention(q, k_cache, v_cache, group.block_tables, ctx, self.heads, self.kv_heads, self.dim,
                            self.vdim, group.page_size, self.scale, self.window, self.sinks, gate, out,
-                           softcap=self.softcap, keep_first=self.keep_first)
+                           softcap=self.softcap, keep_first=self.keep_first, log_bias=self.log_bias,
+                           bias_table=self.bias_table)
         return ops.linear(out, self.w_o, ws=ws, tag="sinkattn.delta", out_dtype=torch.float32,
                           allow_split=self.allow_split)

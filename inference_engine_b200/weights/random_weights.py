@@ -32,6 +32,8 @@ def random_tensor(name: str, decl: Any, seed: int, std: float, dtype, device="cp
         t = torch.randn(decl.shape, generator=gen, dtype=torch.float32, device=device) * std
         if decl.init == "ones_plus_normal":
             t += 1.0
+        elif decl.init == "eye_plus_normal":
+            t += torch.eye(*decl.shape, device=device)
     if decl.role == "int_table":
         return t.to(torch.int32)
     return t.to(dtype)

@@ -14,8 +14,8 @@ import torch
 class RefOps:
     name = "torch-reference"
 
-    def embedding(self, table, ids, out, scale=1.0):
-        out.copy_(table[ids.long()].float() * scale)
+    def embedding(self, table, ids, out, scale=1.0, copies=1):
+        out.copy_((table[ids.long()].float() * scale).repeat(1, copies))
 
     @staticmethod
     def _added(h, delta, rows, delta_scale):
@@ -174,9 +174,10 @@ class RefOps:
         ids.copy_(chosen.to(ids.dtype))
         weights.copy_(w / (w.sum(-1, keepdim=True) + 1e-20) * weight_scale)
 
-    def routed_experts(self, x, ids, weights, w_gate_up, w_down, *, limit, alpha, up_offset, ws, tag="moe"):
+    def routed_experts(self, x, ids, weights, w_gate_up, w_down, *, limit, alpha, up_offset, ws, tag="moe", out=None):
         n, top = ids.shape
-        out = ws.buffer(tag + ".delta", top * n, w_down.shape[1], torch.float32).view(top, n, -1)
+        if out is None:
+            out = ws.buffer(tag + ".delta", top * n, w_down.shape[1], torch.float32).view(top, n, -1)
         xf = x.float()
         for t in range(n):
             for j in range(top):
@@ -295,12 +296,36 @@ class RefOps:
                 if cols > vdim:
                     u = torch.cat([u, torch.ones(heads, 1)], dim=-1)
                 if gates is not None:
-                    g = gates[t].view(heads, 3)
+                    g = gates[0 if gates.dim() == 3 and gates.shape[0] == 1 else t].view(heads, 3)
                     S = g[:, 0, None, None] * S + wt[:, :, None] * (g[:, 1, None] * u)[:, None, :]
                 else:
                     S = a[t].view(heads, dim)[:, :, None] * S + wt[:, :, None] * u[:, None, :]
                 o[t] = torch.einsum("hdc,hd->hc", S, qt) * q_scale
             state[slot, :matrix] = S.transpose(1, 2).reshape(-1)
+
+    def rotate_heads(self, x, positions, table, rot_dims, units, dim):
+        half = rot_dims // 2
+        heads = x[:, : units * dim].unflatten(1, (units, dim))
+        u, v = heads[..., :half].clone(), heads[..., half:rot_dims].clone()
+        cos, sin = table[positions.long(), 0][:, None, :], table[positions.long(), 1][:, None, :]
+        heads[..., :half], heads[..., half:rot_dims] = u * cos - v * sin, v * cos + u * sin
+
+    def stream_mix_norm(self, h, streams, delta, mix, out_coef, read, weight, bias, alpha, eps, out, rows=None):
+        x = (h if rows is None else h[rows.long()]).unflatten(1, (streams, -1))  # [n, S, width]
+        if delta is not None:
+            y = delta.sum(0) if delta.dim() == 3 else delta
+            y = y if rows is None else y[rows.long()]
+            mixed = x if mix is None else torch.einsum("st,nsw->ntw", mix, x)
+            x = mixed + (1.0 if out_coef is None else out_coef[None, :, None]) * y[:, None, :]
+            if rows is None:
+                h.copy_(x.reshape(h.shape))
+        if out is None:
+            return
+        u = x.sum(1) if read is None else torch.einsum("t,ntw->nw", read, x)
+        if alpha is not None:
+            out.copy_((torch.tanh(alpha * u) * weight + bias).to(out.dtype))
+        else:
+            out.copy_((weight * (u * torch.rsqrt(u.pow(2).mean(-1, keepdim=True) + eps))).to(out.dtype))
 
     def lowrank_decay(self, y, w2, bias, tau, decay):
         z = y.float() @ w2.t()
@@ -315,7 +340,8 @@ class RefOps:
             den = torch.maximum(x[..., vdim].abs(), gates.view(-1, heads, 3)[..., 2]) + 1e-6
             y = y / den[..., None]
         y = y * torch.rsqrt(y.pow(2).mean(-1, keepdim=True) + eps)
-        y = y * (weight.view(heads, vdim) if weight.numel() == heads * vdim else weight)
+        if weight is not None:
+            y = y * (weight.view(heads, vdim) if weight.numel() == heads * vdim else weight)
         if gate_pre is not None:
             g = gate_pre.float().reshape(-1, heads, vdim)
             y = y * (torch.sigmoid(g) if gate_act == "sigmoid" else g * torch.sigmoid(g))
@@ -325,7 +351,8 @@ class RefOps:
 
     def qk_norm_rope_write(self, proj, positions, table, rot_dims, q_weight, k_weight, eps, q_out, k_cache,
                            v_cache, slot_mapping, heads, kv_heads, dim, vdim, page_size, bias=None,
-                           value_norm=False, values_from_keys=False, interleaved=False):
+                           value_norm=False, values_from_keys=False, interleaved=False, unit_norm=False,
+                           q_head_scale=None, warm_coef=0.0, warm_every=0):
         n = proj.shape[0]
         end = (heads + kv_heads) * dim + (0 if values_from_keys else kv_heads * vdim)
         proj = proj[:, :end].float()
@@ -337,6 +364,13 @@ class RefOps:
         if q_weight is not None:
             q = q * torch.rsqrt(q.pow(2).mean(-1, keepdim=True) + eps) * q_weight
             k = k * torch.rsqrt(k.pow(2).mean(-1, keepdim=True) + eps) * k_weight
+        if unit_norm:
+            q = q * torch.rsqrt(q.pow(2).mean(-1, keepdim=True) + eps)
+            k = k * torch.rsqrt(k.pow(2).mean(-1, keepdim=True) + eps)
+        if q_head_scale is not None:
+            q = q * q_head_scale[None, :, None]
+        if warm_every:
+            q = q * (1.0 + warm_coef * torch.log(((positions + 1) // warm_every + 1).float()))[:, None, None]
         if value_norm:
             v = v * torch.rsqrt(v.pow(2).mean(-1, keepdim=True) + eps)
         if table is not None and rot_dims > 0:
@@ -377,7 +411,7 @@ class RefOps:
             out[t] = torch.einsum("hk,khd->hd", weights, v).reshape(nh * vdim).to(out.dtype)
 
     def sink_attention(self, q, k_cache, v_cache, block_tables, ctx, nh, nkv, hd, vdim, page_size, scale,
-                       window, sinks, gate, out, softcap=None, keep_first=0):
+                       window, sinks, gate, out, softcap=None, keep_first=0, log_bias=None, bias_table=None):
         groups = nh // nkv
         tables = block_tables.long().cpu()
         positions = ctx.positions.cpu().tolist()
@@ -394,12 +428,16 @@ class RefOps:
             scores = torch.einsum("hd,khd->hk", q[t].reshape(nh, hd).float(), k) * scale
             if softcap:
                 scores = softcap * torch.tanh(scores / softcap)
+            if log_bias is not None:
+                scores = scores - log_bias[0][:, None] * torch.log1p(log_bias[1][:, None] * (p - keys).float())
+            if bias_table is not None:
+                scores = scores + bias_table[:, (p - keys).clamp(max=bias_table.shape[1] - 1)]
             if sinks is not None:
                 scores = torch.cat([scores, sinks[:, None]], dim=1)
             weights = scores.softmax(-1)[:, : keys.numel()]
             o = torch.einsum("hk,khd->hd", weights, v)
             if gate is not None:
-                o = o * torch.sigmoid(gate[t].float())[:, None]
+                o = o * torch.sigmoid(gate[t].float()).view(nh, -1)  # (per head, or per head and value entry)
             out[t] = o.reshape(nh * vdim).to(out.dtype)
 
     def gated_add_norm(self, h, delta, gate_pre, gate_bias, weight, eps, out, rows=None):
@@ -426,7 +464,12 @@ class RefOps:
 
         out.copy_((a * unit(x) + b * unit(x * x) + c * unit(x * x * x) + e).to(out.dtype))
 
-    def linear(self, x, w, out=None, *, ws=None, tag="linear", out_dtype=None, allow_split=False):
+    def linear(self, x, w, out=None, *, ws=None, tag="linear", out_dtype=None, allow_split=False, slices_before=0):
+        if slices_before:
+            whole = ws.buffer(tag, (slices_before + 1) * x.shape[0], w.shape[0], torch.float32)
+            whole = whole.view(slices_before + 1, x.shape[0], w.shape[0])
+            whole[-1] = x.float() @ w.float().t()
+            return whole
         if out is None:
             out = ws.buffer(tag, x.shape[0], w.shape[0], out_dtype)
         out.copy_((x.float() @ w.float().t()).to(out.dtype))
