@@ -709,6 +709,81 @@ def puposun_rows(size: str, kinds: dict, peaks: dict, tokens: int, batch: int, c
     return rows
 
 
+# --- the Livitar design beside the closest models ------------------------------------------------
+
+LIVITAR_SIZES = {
+    # width, residual streams, (retention: heads, dim, vdim, rotated dims), (both attentions: heads, kv_heads,
+    # dim, vdim), (attention_2: distance buckets, largest distance, queries' warmth: coef, every),
+    # (experts: ff, count, top, shared ff)
+    "w1024": (1024, 4, (8, 128, 128, 128), (16, 4, 64, 64), (32, 800, 0.2, 512), (512, 16, 4, 1024)),
+    "w2048": (2048, 4, (16, 128, 128, 128), (16, 4, 128, 128), (32, 800, 0.2, 512), (1024, 32, 4, 2048)),
+}
+
+
+def livitar_config(size: str) -> dict:
+    width, streams, re, at, by, ex = LIVITAR_SIZES[size]
+    retention = {"heads": re[0], "dim": re[1], "vdim": re[2], "rot": {"dims": re[3], "base": 10000.0},
+                 "decay": [1.0 - 2.0 ** -(4.0 + 6.0 * i / re[0]) for i in range(re[0])]}
+    attention = {"heads": at[0], "kv_heads": at[1], "dim": at[2], "vdim": at[3], "scale": at[2] ** -0.5}
+    bucketed = {**attention, "bias_buckets": by[0], "bias_max": by[1], "q_temp": {"coef": by[2], "every": by[3]}}
+    moe = {"kind": "moe", "expert": {"ff": ex[0]}, "router": {"experts": ex[1], "top": ex[2], "scale": 1.5},
+           "shared": {"ff": ex[3]}}
+    layers = [("retention", retention), ("attention", attention), ("attention_2", bucketed), ("retention", retention)]
+    return {"architecture": "Livitar", "vocab": DESIGN_VOCAB, "width": width, "streams": streams,
+            "max_positions": MAX_CONTEXT, "norm": {"eps": 1e-6},
+            "layers": [{"type": t, "mixer": m, "mlp": moe} for t, m in layers]}
+
+
+def livitar_rows(size: str, kinds: dict, peaks: dict, tokens: int, batch: int, ctx: float, decode: bool) -> dict:
+    """Per kind of kernel of the Livitar model: microseconds per launch and, where the kind has such a
+    figure, what it is of the measured peak: decode launches against the copy rate for the bytes they
+    must read (weights, cached rows, state read and written), prompt launches against the burst bf16
+    rate for their flops (the retention in a prompt: those of its recurrence, four per state entry and
+    token); the norms against the copy rate in both."""
+    width, streams, re, at, by, ex = LIVITAR_SIZES[size]
+    H, G, d, dv = at
+    eff, experts, top, shared = ex
+    used = min(experts, batch * top if decode else experts)
+    weights = {  # elements of the matrix a launch reads
+        "linear:retention.in": width * re[0] * (2 * re[1] + 2 * re[2]), "linear:retention.delta": width * re[0] * re[2],
+        "linear:sinkattn.in": width * ((H + G) * d + G * dv + H * dv), "linear:sinkattn.delta": width * H * dv,
+        "linear:ffn.gate_up": 2 * width * shared, "linear:ffn.delta": width * shared,
+        "linear:head": width * DESIGN_VOCAB,
+        "routed.gate_up": 2 * eff * width * used, "routed.down": eff * width * used,
+    }
+    state = re[0] * re[1] * re[2]  # floats of a layer's state per request
+    flops = {  # per prompt launch
+        "attention.sink": 2.0 * H * (d + dv) * tokens * tokens / 2.0,
+        "recurrent.rule": 4.0 * tokens * state, "recurrent.retention": 4.0 * tokens * state,
+        "routed.gate_up": 2.0 * tokens * top * 2 * eff * width, "routed.down": 2.0 * tokens * top * eff * width,
+    }
+    rows = {}
+    for kind, r in kinds.items():
+        us = r["ms"] / r["launches"] * 1e3
+        out = {"us": round(us, 2), "launches": r["launches"]}
+        nbytes = None
+        if kind == "norm":  # (the final norm, of a row or a batch of rows, is one of the nine)
+            parts = (1 + top + 1) / 2  # the output's parts: one behind a mixer, the experts' and the shared one's behind the rest
+            nbytes = tokens * width * (2 * streams * 4 + parts * 4 + 2) * 8 / 9
+        elif decode:
+            if weights.get(kind):
+                nbytes = 2 * weights[kind]
+            elif kind == "attention.sink":
+                nbytes = batch * ctx * G * (d + dv) * 2
+            elif kind in ("recurrent.rule", "recurrent.retention"):
+                nbytes = batch * state * 4 * 2
+        else:
+            f = flops.get(kind) or (2.0 * tokens * weights[kind] if weights.get(kind) and kind != "linear:head" else None)
+            if f:
+                out.update(tflops=round(f / (us * 1e-6) / 1e12, 1),
+                           frac=round(f / (us * 1e-6) / 1e12 / peaks["bf16_tflops"], 4))
+        if nbytes:
+            out.update(gbs=round(nbytes / (us * 1e-6) / 1e9, 1),
+                       frac=round(nbytes / (us * 1e-6) / 1e9 / peaks["hbm_gbs"], 4))
+        rows[kind] = out
+    return rows
+
+
 def run_design(args) -> dict:
     """`--design rugedra`: prompt and decode throughput of the Rugedra design at layer sizes of a real
     model's (four layers: latent attention + dense, delta rule + experts, latent attention + experts,
@@ -720,7 +795,10 @@ def run_design(args) -> dict:
     attention + experts, windowed sink attention + dense, gated linear attention + experts) beside
     the Ravapel and the Llama model.  `--design puposun`: the Puposun design (attention over every
     earlier position, windowed attention twice in a loop, attention again; every layer with experts
-    beside its mixer) beside the Vofanex and the Llama model."""
+    beside its mixer) beside the Vofanex and the Llama model.  `--design livitar`: the Livitar design
+    (retention, attention with a logarithmic and with a bucketed bias by distance, retention; every
+    layer with experts beside a shared one, four residual streams) beside the Puposun, Vofanex and
+    Llama models."""
     import torch
 
     from inference_engine_b200.engine.llm_engine import LLMEngine
@@ -744,6 +822,11 @@ def run_design(args) -> dict:
         elif args.design == "puposun":
             models = [("puposun", puposun_config(size)), ("vofanex", vofanex_config(size)),
                       ("llama", llama_config_like(size))]
+        elif args.design == "livitar":
+            models = [("livitar", livitar_config(size)), ("puposun", puposun_config(size)),
+                      ("vofanex", vofanex_config(size)), ("llama", llama_config_like(size))]
+        if args.only:
+            models = [m for m in models if m[0] in args.only.split(",")]
         for name, cfg in models:
             engine = LLMEngine.from_random(
                 cfg, seed=0, dtype="bfloat16", device="cuda", max_model_len=MAX_CONTEXT,
@@ -756,7 +839,10 @@ def run_design(args) -> dict:
                    "prefill_tokens_per_s": round(PREFILL_LEN / (prefill_ms / 1e3), 1), "prefill_ms": round(prefill_ms, 3),
                    # (the prompt step is launched eagerly: what its kernels take by themselves, without the host)
                    "prefill_kernels_ms": round(sum(r["ms"] for r in kinds_prefill.values()), 3)}
-            if name == "puposun":
+            if name == "livitar":
+                row["kernels"] = {f"decode_b{batch}": livitar_rows(size, kinds, peaks, batch, batch, ctx, True),
+                                  f"prefill_{PREFILL_LEN}": livitar_rows(size, kinds_prefill, peaks, PREFILL_LEN, 1, PREFILL_LEN, False)}
+            elif name == "puposun":
                 row["kernels"] = {f"decode_b{batch}": puposun_rows(size, kinds, peaks, batch, batch, ctx, True),
                                   f"prefill_{PREFILL_LEN}": puposun_rows(size, kinds_prefill, peaks, PREFILL_LEN, 1, PREFILL_LEN, False)}
             elif name == "vofanex":
@@ -896,9 +982,10 @@ def main() -> int:
     ap.add_argument("--warmup", type=int, default=8)
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--design", default=None, choices=["rugedra", "ravapel", "vofanex", "puposun"],
+    ap.add_argument("--design", default=None, choices=["rugedra", "ravapel", "vofanex", "puposun", "livitar"],
                     help="instead of the default workload: this design at real layer sizes beside the closest "
                          "model the engine had, prompt and decode throughput and every kind of kernel")
+    ap.add_argument("--only", default=None, help="with --design: only these of its models (comma-separated)")
     ap.add_argument("--sizes", default="w1024,w2048", help="with --design: which of " + ",".join(DESIGN_SIZES))
     args = ap.parse_args()
     if args.gpus != 1 or int(os.environ.get("WORLD_SIZE", "1")) != 1:

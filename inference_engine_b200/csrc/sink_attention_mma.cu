@@ -92,6 +92,16 @@ __device__ __forceinline__ float log2_fast(float x) {
     asm("lg2.approx.f32 %0, %1;" : "=f"(y) : "f"(x));
     return y;
 }
+// The bias of a score at distance n, in units of log2 e.  Below zero (a key that is masked anyway) it is the
+// one at distance zero.  BIAS 1: -r1 ln(1 + r2 n) is -r1 log2(1 + r2 n) in these units.
+__device__ __forceinline__ float log_bias_at(float n, float r1, float r2) {
+    return -r1 * log2_fast(fmaf(r2, fmaxf(n, 0.f), 1.0f));
+}
+__device__ __forceinline__ float distance_bias(int n, float r1, float r2, const float* table, int len) {
+    if constexpr (BIAS == 1) return log_bias_at((float)n, r1, r2);
+    if constexpr (BIAS == 2) return __ldg(table + min(max(n, 0), len - 1)) * LOG2E;
+    return 0.f;
+}
 __device__ __forceinline__ float sigmoid_of(float z) { return 1.0f / (1.0f + expf(-z)); }
 __device__ __forceinline__ float quad_max(float x) {
     x = fmaxf(x, __shfl_xor_sync(0xffffffffu, x, 1));
@@ -102,7 +112,8 @@ __device__ __forceinline__ float quad_sum(float x) {
     return x + __shfl_xor_sync(0xffffffffu, x, 2);
 }
 
-// grid: (query tiles, heads, requests).
+// grid: (query tiles, heads, requests); SPLIT: (ranges of key tiles, key/value heads, requests).
+template <bool SPLIT>
 __global__ void __launch_bounds__(THREADS)
 sink_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ k_cache,
                           const __nv_bfloat16* __restrict__ v_cache, const int* __restrict__ block_tables,
@@ -121,7 +132,7 @@ sink_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat
     ie_pdl_wait();
     // (with `partial` the first grid dimension counts ranges of key tiles and the second key/value heads;
     // row r of the block is then token r / group with query head kvh * group + r % group)
-    const bool split_mode = partial != nullptr;
+    constexpr bool split_mode = SPLIT;
     const int group = heads / kv_heads;
     int seq = blockIdx.z, head = blockIdx.y, tile = split_mode ? 0 : gridDim.x - 1 - blockIdx.x;
     int q0 = cu_q[seq], q_len = cu_q[seq + 1] - q0;
@@ -192,6 +203,18 @@ sink_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat
         }
     }
     load_tile(tile_of(t_begin), 0);
+    if constexpr (BIAS == 2) {
+        // (a range of few tiles is a chain of trips to memory: the bias entries it needs set out with the keys)
+        if (split_mode) {
+            int nearest = max(first_pos - (tile_of(t_end) * KEYS + KEYS - 1), 0), farthest = last_pos - tile_of(t_begin) * KEYS;
+            int lines = (min(farthest, bias_len - 1) - min(nearest, bias_len - 1)) / 32 + 2;
+            for (int i = tid; i < group * lines; i += THREADS) {
+                int h = i / lines, at = min(nearest + (i - h * lines) * 32, bias_len - 1);
+                const float* p = bias_table + (size_t)(kvh * group + h) * bias_len + at;
+                asm volatile("prefetch.global.L1 [%0];" ::"l"(p));
+            }
+        }
+    }
     // the block's queries (rows beyond the request's tokens read as zero)
     for (int i = tid; i < ROWS * (D / 8); i += THREADS) {
         int r = i / (D / 8), c = i - r * (D / 8);
@@ -218,9 +241,12 @@ sink_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat
     // sink's term of the sum is counted by the first thread of the four that share a row
     const float sl2 = scale * LOG2E;
     const float cap_in = softcap > 0.f ? scale / softcap : 0.f, cap_out = softcap * LOG2E;
-    // BIAS: the two rows' numbers.  1: r1 (in units of log2 e of ln: the factor of log2) and r2; 2: the
-    // table row and its last entry (in units of log2 e).
+    // BIAS: the two rows' numbers.  1: r1 and r2; 2: the table row and, in r1's place, its last entry (in
+    // units of log2 e).
     float r1_a = 0.f, r1_b = 0.f, r2_a = 0.f, r2_b = 0.f;
+    // (positions for the bias: rows that do not exist follow their block's)
+    const int bpos_a = first_pos + (split_mode ? max(pos_a - first_pos, 0) : r_a);
+    const int bpos_b = first_pos + (split_mode ? max(pos_b - first_pos, 0) : r_b);
     const float *tab_a = nullptr, *tab_b = nullptr;
     if constexpr (BIAS != 0) {
         int h_a = r_a < rows_here ? row_head(r_a) : 0, h_b = r_b < rows_here ? row_head(r_b) : 0;
@@ -282,31 +308,61 @@ sink_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat
             // (the first query of the block is the one nearest to the tile)
             const bool whole = window == 0 && t * KEYS + KEYS - 1 <= first_pos;
             const bool all_far = BIAS == 2 && first_pos - (t * KEYS + KEYS - 1) >= bias_len - 1;
+            const int at = t * KEYS + t4 * 2;
+            // a score in units of log2 e, before its bias
+            auto scaled = [&](float x) { return softcap > 0.f ? cap_out * tanh_fast(x * cap_in) : x * sl2; };
+            if (all_far) {
+#pragma unroll
+                for (int nt = 0; nt < KEYS / 8; ++nt) {
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) s[nt][e] = scaled(s[nt][e]) + (e < 2 ? r1_a : r1_b);
+                }
+            } else if (split_mode) {  // (the two rows may be different heads')
+#pragma unroll
+                for (int nt = 0; nt < KEYS / 8; ++nt) {
+#pragma unroll
+                    for (int e = 0; e < 4; ++e)
+                        s[nt][e] = scaled(s[nt][e]) +
+                                   distance_bias((e < 2 ? bpos_a : bpos_b) - (at + nt * 8 + (e & 1)), e < 2 ? r1_a : r1_b,
+                                                 e < 2 ? r2_a : r2_b, e < 2 ? tab_a : tab_b, bias_len);
+                }
+            } else {
+                // row b lies eight positions behind row a, so its bias at one group of eight keys is row a's
+                // at the next group: eighteen values serve 32 scores
+                const int d0 = bpos_a + 8 - at;  // row b's distance to the first key of this thread
+                const float f0 = (float)d0;      // (below 2^24: the differences to it are exact)
+                auto bias_at = [&](int off) {
+                    if constexpr (BIAS == 1) return log_bias_at(f0 - (float)off, r1_a, r2_a);
+                    else return distance_bias(d0 - off, r1_a, r2_a, tab_a, bias_len);
+                };
+                float behind[2];
+#pragma unroll
+                for (int e = 0; e < 2; ++e) behind[e] = bias_at(e);
+#pragma unroll
+                for (int nt = 0; nt < KEYS / 8; ++nt) {
+#pragma unroll
+                    for (int e = 0; e < 2; ++e) {
+                        float bias = bias_at(8 + nt * 8 + e);
+                        s[nt][e] = scaled(s[nt][e]) + bias;
+                        s[nt][2 + e] = scaled(s[nt][2 + e]) + behind[e];
+                        behind[e] = bias;
+                    }
+                }
+            }
+            if (!whole) {
+#pragma unroll
+                for (int nt = 0; nt < KEYS / 8; ++nt) {
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        int key_pos = at + nt * 8 + (e & 1);
+                        int pos = e < 2 ? pos_a : pos_b, lo = e < 2 ? lo_a : lo_b;
+                        bool visible = key_pos <= pos && (key_pos >= lo || key_pos < keep_first);
+                        s[nt][e] = visible ? s[nt][e] : -INFINITY;
+                    }
+                }
+            }
 #pragma unroll
             for (int nt = 0; nt < KEYS / 8; ++nt) {
-                int kp = t * KEYS + nt * 8 + t4 * 2;
-#pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    int key_pos = kp + (e & 1);
-                    int dist = (e < 2 ? pos_a : pos_b) - key_pos;
-                    float sc = s[nt][e] * sl2;
-                    if (softcap > 0.f) sc = cap_out * tanh_fast(s[nt][e] * cap_in);
-                    if constexpr (BIAS == 1) {
-                        // -r1 ln(1 + r2 n) in units of log2 e is -r1 log2(1 + r2 n)
-                        float n = (float)max(dist, 0);
-                        sc = fmaf(-(e < 2 ? r1_a : r1_b), log2_fast(fmaf(e < 2 ? r2_a : r2_b, n, 1.0f)), sc);
-                    } else if (all_far) {
-                        sc += e < 2 ? r1_a : r1_b;
-                    } else {
-                        sc = fmaf(__ldg((e < 2 ? tab_a : tab_b) + min(max(dist, 0), bias_len - 1)), LOG2E, sc);
-                    }
-                    if (!whole) {
-                        int lo = e < 2 ? lo_a : lo_b;
-                        bool visible = dist >= 0 && (key_pos >= lo || key_pos < keep_first);
-                        sc = visible ? sc : -INFINITY;
-                    }
-                    s[nt][e] = sc;
-                }
                 mx_a = fmaxf(mx_a, fmaxf(s[nt][0], s[nt][1]));
                 mx_b = fmaxf(mx_b, fmaxf(s[nt][2], s[nt][3]));
             }
@@ -478,8 +534,9 @@ IE_API int ie_sink_attention_mma(const void* q, const void* k_cache, const void*
         (BIAS == 2 && bias_len < 1))
         return (int)cudaErrorInvalidValue;  // (the library was built for another kind of bias)
     size_t smem = (size_t)(ROWS * LDK + 2 * KEYS * LDK + 2 * KEYS * LDV) * sizeof(__nv_bfloat16);
-    static IePerDevice allowed;
-    cudaError_t e = ie_allow_smem(allowed, sink_attention_mma_kernel, smem);
+    static IePerDevice allowed, allowed_split;
+    cudaError_t e = ie_allow_smem(allowed, sink_attention_mma_kernel<false>, smem);
+    if (e == cudaSuccess) e = ie_allow_smem(allowed_split, sink_attention_mma_kernel<true>, smem);
     if (e != cudaSuccess) return (int)e;
     if (partial != nullptr) {
         // ranges of key tiles: a request's tokens times the heads of a group are one tile of rows, and
@@ -487,7 +544,7 @@ IE_API int ie_sink_attention_mma(const void* q, const void* k_cache, const void*
         if (max_q_len * (heads / kv_heads) > ROWS || splits < 1 || splits > MERGE_MAX_SPLITS || tiles_per_split < 1 ||
             num_tokens < 1 || kept_splits >= splits)
             return (int)cudaErrorInvalidValue;
-        int rc = ie_launch(sink_attention_mma_kernel, dim3(splits, kv_heads, num_seqs), dim3(THREADS), smem,
+        int rc = ie_launch(sink_attention_mma_kernel<true>, dim3(splits, kv_heads, num_seqs), dim3(THREADS), smem,
                            (cudaStream_t)stream, (const __nv_bfloat16*)q, (const __nv_bfloat16*)k_cache,
                            (const __nv_bfloat16*)v_cache, block_tables, table_width, cu_q, ctx_lens, (__nv_bfloat16*)out,
                            heads, kv_heads, page_size, total_pages, scale, window, sinks, out_gate, gate_ld, partial,
@@ -499,7 +556,7 @@ IE_API int ie_sink_attention_mma(const void* q, const void* k_cache, const void*
                          gate_ld, gate_elements);
     }
     dim3 grid((max_q_len + ROWS - 1) / ROWS, heads, num_seqs);
-    return ie_launch(sink_attention_mma_kernel, grid, dim3(THREADS), smem, (cudaStream_t)stream,
+    return ie_launch(sink_attention_mma_kernel<false>, grid, dim3(THREADS), smem, (cudaStream_t)stream,
                      (const __nv_bfloat16*)q, (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache, block_tables,
                      table_width, cu_q, ctx_lens, (__nv_bfloat16*)out, heads, kv_heads, page_size, total_pages, scale,
                      window, sinks, out_gate, gate_ld, (float*)nullptr, 1, 0, softcap, keep_first, 0,

@@ -175,6 +175,15 @@ def build_sink_attention(dim: int, vdim: int, bias: str = "none") -> Path:
                          [f"-DSK_D={dim}", f"-DSK_DV={vdim}"] + ([f"-DSK_BIAS={kind}"] if kind else []))
 
 
+def build_retention(dim: int, vdim: int) -> Path:
+    """The bfloat16 path's retention kernels for one pair of key and value sizes, each rounded up to a
+    multiple of 16 (compiled on first use for the sizes the loaded model has)."""
+    if not 1 <= dim <= 128 or not 1 <= vdim <= 128:
+        raise BuildError(f"the retention kernels take key and value sizes up to 128, not {dim} and {vdim}")
+    d, dv = -(-dim // 16) * 16, -(-vdim // 16) * 16
+    return build_library(f"ie_b200_retention_d{d}_v{dv}", ["retention.cu"], [f"-DRT_D={d}", f"-DRT_DV={dv}"])
+
+
 # Kernels only some mixers and feed-forwards need, each a library of its own that is built the
 # first time a model with such a part runs: name -> sources.
 PART_LIBRARIES = {
@@ -206,7 +215,8 @@ def build_all(prune: bool = True) -> list[Path]:
         libs += list(pool.map(build_attention, ATTENTION_HEAD_DIMS))
         libs += list(pool.map(build_part_library, PART_LIBRARIES))
         libs += [build_sigmoid_attention(64, 64), build_sink_attention(64, 64),
-                 build_sink_attention(64, 64, "log"), build_sink_attention(64, 64, "table")]
+                 build_sink_attention(64, 64, "log"), build_sink_attention(64, 64, "table"),
+                 build_retention(64, 64)]
     if prune:
         keep = {lib.name for lib in libs}
         for old in build_dir().glob("libie_b200_*.so"):

@@ -18,7 +18,7 @@ import os
 from ctypes import c_float, c_int, c_void_p
 
 from .build import (ATTENTION_HEAD_DIMS, build_attention, build_core, build_part_library,
-                    build_sigmoid_attention, build_sink_attention)
+                    build_retention, build_sigmoid_attention, build_sink_attention)
 
 _ERRORS = {
     1: "a token id outside the vocabulary",
@@ -137,6 +137,8 @@ class CudaOps:
         self._attn_libs: dict[int, object] = {}
         self._part_libs: dict[str, object] = {}
         self._sigattn_libs: dict[tuple[int, int], object] = {}
+        self._retention_libs: dict[tuple[int, int], object] = {}
+        self.retention_fused = os.environ.get("IE_B200_RETENTION", "1") != "0"  # the retention kernels of the bfloat16 path
         self._sinkattn_libs: dict[tuple[int, int, str], object] = {}
         self.sink_mma = os.environ.get("IE_B200_SINK_MMA", "1") != "0"  # tensor-core sink attention
         # residual gates' products as partial sums: faster by themselves, slower inside a captured step
@@ -1315,6 +1317,68 @@ class CudaOps:
         self._check(self._part_lib("recurrent").ie_rotate_heads(
             x.data_ptr(), x.stride(0), positions.data_ptr(), table.data_ptr(), rot_dims, table.shape[0], x.shape[0],
             units, dim, self._err_ptr, self._stream()), "rotate_heads")
+
+    def _retention_lib(self, dim: int, vdim: int):
+        key = (-(-dim // 16), -(-vdim // 16))
+        lib = self._retention_libs.get(key)
+        if lib is None:
+            path = build_retention(dim, vdim)
+            try:
+                lib = ctypes.CDLL(str(path))
+            except OSError as exc:
+                raise KernelError(f"the kernel library {path} could not be loaded: {exc}") from exc
+            P, I, F, L = c_void_p, c_int, c_float, ctypes.c_longlong
+            lib.ie_retention.argtypes = [P, I, I, I, I, P, I, I, P, P, P, L, P, P, I, F, F, P, I, I, I, P, P, P]
+            lib.ie_retention.restype = c_int
+            self._retention_libs[key] = lib
+        return lib
+
+    # requests that bring at most so many tokens each go through the kernel that takes them one by one;
+    # longer portions are cut into chunks of so many
+    RETENTION_STEP, RETENTION_CHUNK = 8, 64
+
+    def retention(self, proj, ctx, table, rot_dims, gates, powers, state, slots, out, heads, dim, vdim, eps, ws) -> None:
+        """Retention from the fused 32-bit projection (columns: ``heads * dim`` queries, as many keys, ``heads *
+        vdim`` values and gates): rotation of the first ``rot_dims`` entries of queries and keys (``table``; 0:
+        none), ``S <- decay S + k v^T`` and ``o = S^T q * dim^-1/2`` per head from and to the requests' slots
+        (``[heads, vdim, dim]``), ``out = o / rms(o) * silu(gate)``.  ``gates``: ``[1, heads, 3]`` = (decay, 1, 1);
+        ``powers``: ``[heads, 65]``, the decays' powers 0 to 64.  A bfloat16 ``out`` with sizes up to 128 runs the
+        fused kernels (a step of few tokens per request: one launch; prompt portions in chunks on the
+        tensor cores); 32-bit and other sizes rotation, recurrence and read-out one after the other, whose
+        order of operations does not depend on the cutting."""
+        qk = heads * dim
+        if proj.dtype != self.torch.float32 or proj.stride(1) != 1 or proj.shape[1] < 2 * heads * (dim + vdim):
+            raise KernelError("retention reads the fused 32-bit projection of queries, keys, values and gates")
+        if rot_dims and table.shape[2] * 2 != rot_dims:
+            raise KernelError("rotary table does not match the rotated dims")
+        if self.retention_fused and out.dtype == self.torch.bfloat16 and dim <= 128 and vdim <= 128:
+            return self._retention(proj, ctx, table, rot_dims, powers, state, slots, out, heads, dim, vdim, eps, ws)
+        if rot_dims:
+            self.rotate_heads(proj, ctx.positions, table, rot_dims, 2 * heads, dim)
+        o = ws.buffer("retention.o", proj.shape[0], heads * vdim, self.torch.float32)
+        at_g = 2 * qk + heads * vdim
+        self.gated_recurrence(proj[:, :qk], None, proj[:, qk: 2 * qk], gates, proj[:, 2 * qk: at_g], state, slots, ctx, o,
+                              heads, dim, vdim, vdim, dim ** -0.5)
+        self.recurrence_readout(o, None, None, eps, proj[:, at_g: at_g + heads * vdim], out, heads, vdim, vdim,
+                                gate_act="silu")
+
+    @_kind("recurrent.retention")
+    def _retention(self, proj, ctx, table, rot_dims, powers, state, slots, out, heads, dim, vdim, eps, ws) -> None:
+        lib = self._retention_lib(dim, vdim)
+        bounds = getattr(ctx, "bounds", None)
+        longest = bounds[0] if bounds is not None else ctx.max_q_len  # (a captured step: its token bound)
+        chunks, scratch = 0, None
+        if longest > self.RETENTION_STEP:
+            size = self.RETENTION_CHUNK
+            chunks = bounds[0] // size + bounds[1] if bounds is not None else sum(-(-n // size) for n in ctx.q_lens)
+            scratch = ws.buffer("retention.state", chunks * heads, dim * vdim, self.torch.float32, rows_cap=None)
+        self._check(lib.ie_retention(
+            proj.data_ptr(), proj.stride(0), heads, dim, vdim, self._ptr(table), rot_dims,
+            0 if table is None else table.shape[0], ctx.ctx_lens.data_ptr(), powers.data_ptr(), state.data_ptr(),
+            state.stride(0), slots.data_ptr(), ctx.cu_q.data_ptr(), ctx.num_seqs, dim ** -0.5, eps, out.data_ptr(),
+            state.shape[0], longest, chunks, self._ptr(scratch), self._err_ptr, self._stream()),
+            "retention_chunks" if chunks else "retention_step")
+        self.launches += 2 if chunks else 0
 
     @_kind("recurrent.gates")
     def lowrank_decay(self, y, w2, bias, tau: float, decay) -> None:

@@ -275,6 +275,7 @@ class GatedLinearAttention(Mixer):
 class Retention(Mixer):
     allow_split = True
     accepts_input_rows = True
+    CHUNK = 64  # tokens the kernels take at a time in a prompt portion
 
     def __init__(self, *, names: dict, hidden_size: int, heads: int, dim: int, vdim: int, decay, eps: float, position,
                  dtype) -> None:
@@ -308,6 +309,9 @@ class Retention(Mixer):
         n = self.names
         self.w_in, self.extra_at = self._with_extra_rows([tensors[n[k]].to(self.dtype) for k in ("q", "k", "v", "g")])
         self.w_o = tensors[n["o"]].to(self.dtype).contiguous()
+        # the decays' powers, worked out in 64-bit, for the kernels that take a prompt in chunks
+        exact = torch.tensor(self.decay, dtype=torch.float64)
+        self.powers = (exact[:, None] ** torch.arange(self.CHUNK + 1, dtype=torch.float64)).float().to(self.w_o.device)
         # (decay, write gate, unused) per head, the same for every token
         self.gates = torch.tensor([[[d, 1.0, 1.0] for d in self.decay]], dtype=torch.float32, device=self.w_o.device)
 
@@ -317,20 +321,13 @@ class Retention(Mixer):
     def forward(self, x, ctx, binding):
         import torch
 
-        f32, n, qk, vs = torch.float32, x.shape[0], self.qk_size, self.v_size
+        f32, n = torch.float32, x.shape[0]
         group = ctx.groups[binding.group]
         ops, ws = ctx.ops, ctx.ws
         proj = ops.linear(x, self.w_in, ws=ws, tag="retention.in", out_dtype=f32)
         self.extra_out = self._extra_columns(proj, self.extra_at)
-        at_g = 2 * qk + vs
-        if self.position is not None and self.position.rotary_dim:
-            ops.rotate_heads(proj, ctx.positions, self.position.rotary_table(), self.position.rotary_dim,
-                             2 * self.heads, self.dim)
-        o = ws.buffer("retention.o", n, vs, f32)
-        ops.gated_recurrence(proj[:, :qk], None, proj[:, qk: 2 * qk], self.gates, proj[:, 2 * qk: at_g],
-                             group.state[binding.slot], group.slots, ctx, o, self.heads, self.dim, self.vdim,
-                             self.vdim, self.dim ** -0.5)
-        out = ws.buffer("retention.out", n, vs, self.dtype)
-        ops.recurrence_readout(o, None, None, self.eps, proj[:, at_g: at_g + vs], out, self.heads, self.vdim,
-                               self.vdim, gate_act="silu")
+        rot_dims = self.position.rotary_dim if self.position is not None else 0
+        out = ws.buffer("retention.out", n, self.v_size, self.dtype)
+        ops.retention(proj, ctx, self.position.rotary_table() if rot_dims else None, rot_dims, self.gates, self.powers,
+                      group.state[binding.slot], group.slots, out, self.heads, self.dim, self.vdim, self.eps, ws)
         return ops.linear(out, self.w_o, ws=ws, tag="retention.delta", out_dtype=f32, allow_split=self.allow_split)

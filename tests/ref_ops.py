@@ -310,6 +310,17 @@ class RefOps:
         cos, sin = table[positions.long(), 0][:, None, :], table[positions.long(), 1][:, None, :]
         heads[..., :half], heads[..., half:rot_dims] = u * cos - v * sin, v * cos + u * sin
 
+    def retention(self, proj, ctx, table, rot_dims, gates, powers, state, slots, out, heads, dim, vdim, eps, ws):
+        qk, at_g = heads * dim, heads * (2 * dim + vdim)
+        proj = proj.clone()
+        if rot_dims:
+            self.rotate_heads(proj, ctx.positions, table, rot_dims, 2 * heads, dim)
+        o = torch.zeros(proj.shape[0], heads * vdim)
+        self.gated_recurrence(proj[:, :qk], None, proj[:, qk: 2 * qk], gates, proj[:, 2 * qk: at_g], state, slots, ctx, o,
+                              heads, dim, vdim, vdim, dim ** -0.5)
+        self.recurrence_readout(o, None, None, eps, proj[:, at_g: at_g + heads * vdim], out, heads, vdim, vdim,
+                                gate_act="silu")
+
     def stream_mix_norm(self, h, streams, delta, mix, out_coef, read, weight, bias, alpha, eps, out, rows=None):
         x = (h if rows is None else h[rows.long()]).unflatten(1, (streams, -1))  # [n, S, width]
         if delta is not None:
