@@ -36,3 +36,11 @@ class EngineConfig:
             raise ValueError("gpu_memory_utilization must be in (0, 1]")
         if self.max_model_len is not None and self.max_model_len < 1:
             raise ValueError("max_model_len must be >= 1")
+
+    @property
+    def most_positions(self) -> int | None:
+        """The most positions a request can reach by these settings alone (None: they do not say): tables by
+        position need be no longer.  A model with no cache pages can be given a ``max_model_len``."""
+        if self.max_model_len is not None or self.num_blocks is None:
+            return self.max_model_len
+        return self.num_blocks * self.block_size

@@ -115,7 +115,7 @@ class LLMEngine:
         tokenizer = settings.pop("tokenizer", None)
         stop_ids = settings.pop("stop_token_ids", None)
         config = cls._settings(config, dtype, settings)
-        model, _ = load_model(model_dir, config.dtype, device, max_positions=config.max_model_len)
+        model, _ = load_model(model_dir, config.dtype, device, max_positions=config.most_positions)
         if stop_ids is None:
             stop_ids = load_stop_token_ids(model_dir)
         return cls(model, tokenizer, stop_ids, config, ops=settings.pop("ops", None))
@@ -131,7 +131,7 @@ class LLMEngine:
         stop_ids = settings.pop("stop_token_ids", ())
         ops = settings.pop("ops", None)
         config = cls._settings(config, dtype, settings)
-        model, _ = random_model(model_config, seed, config.dtype, device, max_positions=config.max_model_len)
+        model, _ = random_model(model_config, seed, config.dtype, device, max_positions=config.most_positions)
         return cls(model, tokenizer, stop_ids, config, ops=ops)
 
     @staticmethod

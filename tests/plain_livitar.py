@@ -80,10 +80,10 @@ def log_distance_bias(dist, r1, r2):
 
 
 def bucket(n: int, buckets: int, bias_max: float) -> int:
-    half = buckets // 2
+    half = buckets / 2
     if n < half:
         return n
-    return min(buckets - 1, half + math.floor(math.log(n / half) / math.log(bias_max / half) * (buckets - half)))
+    return int(min(buckets - 1, half + math.floor(math.log(n / half) / math.log(bias_max / half) * (buckets - half))))
 
 
 def bucket_bias(dist, rel, bias_max, h):
