@@ -53,9 +53,9 @@ def without_bucket_counts(cfg: dict) -> dict:
 MIXED = config(72, 131, [
     (retention(3, 16, 8, (0.9, 0.99, 0.5), rot=8, base=500.0), moe(8, 2, 24, shared=40, scale=1.5)),
     (attention(6, 2, 16, 24), moe(5, 1, 16, shared=16)),
-    (attention_2(4, 1, 12, 20, 40, q_temp=(0.7, 8), scale=1.1), None),
+    (attention_2(4, 1, 12, 20, 40, q_temp=(0.7, 8), scale=0.45), None),
     (retention(2, 20, 36, (1.0, 0.97), rot=20), moe(6, 6, 20)),
-    (attention_2(2, 2, 8, 8, 9, scale=0.8, buckets=6), moe(4, 3, 12, shared=8, scale=2.5)),
+    (attention_2(2, 2, 8, 8, 9, scale=0.6, buckets=6), moe(4, 3, 12, shared=8, scale=2.5)),
 ], streams=3)
 # nothing a multiple of four; one stream; the state forgets almost at once in one head; no rotation
 ODD = config(50, 61, [
@@ -67,8 +67,8 @@ ODD = config(50, 61, [
 # one that never does
 STREAMS = config(64, 97, [
     (retention(4, 8, 8, (0.8, 0.9, 0.96, 0.99), rot=4, base=77.0), moe(4, 2, 20, shared=12, scale=2.2)),
-    (attention_2(4, 4, 16, 8, 5, q_temp=(0.5, 16), scale=1.0, buckets=8), moe(3, 1, 12)),
-    (attention_2(2, 1, 8, 16, 5000, q_temp=(1.0, 300), scale=0.7, buckets=32), None),
+    (attention_2(4, 4, 16, 8, 5, q_temp=(0.5, 16), scale=0.4, buckets=8), moe(3, 1, 12)),
+    (attention_2(2, 1, 8, 16, 5000, q_temp=(1.0, 300), scale=0.6, buckets=32), None),
     (attention(4, 2, 8, 8), None),
     (retention(1, 33, 17, (0.98,), rot=32), moe(2, 1, 18, shared=6)),
 ], streams=5)
@@ -81,9 +81,9 @@ ONE_BUCKET = config(48, 83, [
 WIDE = config(128, 211, [
     (retention(4, 64, 48, (0.9, 0.99, 0.995, 0.97), rot=32), moe(8, 2, 64, shared=96, scale=2.0)),
     (attention(8, 2, 64, 32), moe(8, 3, 32)),
-    (attention_2(6, 3, 32, 128, 150, q_temp=(0.4, 64), scale=1.3, buckets=24), None),
+    (attention_2(6, 3, 32, 128, 150, q_temp=(0.4, 64), scale=0.3, buckets=24), None),
     (retention(2, 128, 128, (0.98, 0.999), rot=128, base=2e5), moe(4, 1, 48, shared=32)),
-    (attention_2(4, 1, 48, 48, 3000, scale=1.0, buckets=32), moe(4, 2, 32, shared=64)),
+    (attention_2(4, 1, 48, 48, 3000, scale=0.25, buckets=32), moe(4, 2, 32, shared=64)),
 ], streams=4)
 
 CONFIGS = {"mixed": MIXED, "odd": ODD, "streams": STREAMS, "one_bucket": ONE_BUCKET}
@@ -164,7 +164,7 @@ def make_weights(cfg: dict, seed: int = 0) -> dict:
         else:
             t = torch.randn(shape, generator=g) / shape[-1] ** 0.5
             if name.endswith(("mix.q", "mix.k")):
-                t = t * 2.0
+                t = t * 1.5
             if name.endswith("mlp.router"):
                 t = t * 4.0
         out[name] = t.to(torch.bfloat16)

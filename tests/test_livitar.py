@@ -19,7 +19,6 @@ from tests import livitar_configs as V
 from tests import plain_livitar as P
 
 LENGTHS = [50, 21, 37, 64, 9, 1]
-BF16_TOL = dict(atol=0.35, rtol=0.0, pos_rel_rms=0.08, rel_rms=0.04)
 # (under these names the run's summary lists this file's comparisons: their bounds are measured)
 LABEL = {"float32": "float32, Livitar", "bfloat16": "bfloat16, Livitar"}
 DEVICES = ["cpu", pytest.param("cuda", marks=pytest.mark.gpu)]
@@ -43,29 +42,47 @@ def _float32_bound(cfg, weights, requests, want) -> dict:
     return dict(atol=max(3 * worst, H.TOL["float32"]["atol"]), rtol=H.TOL["float32"]["rtol"])
 
 
+def _position_errors(got, want):
+    """Per position, over all requests: the root mean square of the difference over that of the logits."""
+    err = [(got[rid].double() - want[rid].double()).pow(2).mean(-1).sqrt() / want[rid].double().pow(2).mean(-1).sqrt()
+           for rid in want]
+    return torch.cat(err)
+
+
 def _bfloat16_bound(tmp_path, cfg, weights, requests, want) -> dict:
-    """Three times what rounding does to the same requests on the plain stand-ins of the kernels run
-    in bfloat16 (activations rounded between the parts, as the kernels round them), and never below
-    the fixed bounds."""
+    """From the same requests on the plain stand-ins of the kernels run in bfloat16 (activations rounded
+    between the parts, as the kernels round them): three times the median error of a position (never below
+    0.04), and the share of positions that rounding alone carries beyond that.  Such positions there are:
+    where a token's experts are a close call, rounding chooses another one, and everything after sees it."""
     from tests.ref_ops import RefOps
 
     room = sum(H.round64(len(t)) for t in requests.values())
     got = H.collect(_session(tmp_path / "bound", cfg, weights, "bfloat16", "cpu", RefOps(), room, 16),
                     H.trace_whole(requests))
-    tol = dict(BF16_TOL)
-    for rid in requests:
-        diff = (got[rid].double() - want[rid].double()).abs()
-        pos_rel = diff.pow(2).mean(-1).sqrt() / want[rid].double().pow(2).mean(-1).sqrt().clamp_min(1e-12)
-        rel = float(diff.pow(2).mean().sqrt() / want[rid].double().pow(2).mean().sqrt())
-        tol["atol"] = max(tol["atol"], 3 * float(diff.max()))
-        tol["pos_rel_rms"] = max(tol["pos_rel_rms"], 3 * float(pos_rel.max()))
-        tol["rel_rms"] = max(tol["rel_rms"], 3 * rel)
-    return tol
+    err = _position_errors(got, want)
+    bound = max(3 * float(err.median()), 0.04)
+    assert bound < 0.3, "the test weights magnify rounding so much that a fault would hide in it"
+    return dict(pos_rel_rms=bound, share=float((err > bound).float().mean()))
 
 
 def _bound(tmp_path, dtype, cfg, weights, requests, want):
     return (_float32_bound(cfg, weights, requests, want) if dtype == "float32"
             else _bfloat16_bound(tmp_path, cfg, weights, requests, want))
+
+
+def _check(got, want, dtype, what, tol) -> None:
+    """32-bit: every position within the bound.  bfloat16: at most twice the share of positions beyond it that
+    rounding alone brings, and 4 % (a fault of a cache, a state or a batch is not limited to a few)."""
+    if dtype == "float32":
+        for rid in want:
+            H.assert_close(got[rid], want[rid], LABEL[dtype], f"{what} {rid}", tol)
+        return
+    assert all(got[rid].shape == want[rid].shape and bool(torch.isfinite(got[rid]).all()) for rid in want), what
+    err = _position_errors(got, want)
+    share, allowed = float((err > tol["pos_rel_rms"]).float().mean()), 2 * tol["share"] + 0.04
+    H._record(LABEL[dtype], max_median_pos_rel_rms=float(err.median()), max_share_beyond=share)
+    assert float(err.median()) < tol["pos_rel_rms"] / 1.5, (what, float(err.median()), tol)
+    assert share <= allowed, (what, share, tol)
 
 
 def _session(tmp_path, cfg, weights, dtype, device, ops, max_tokens, page_size):
@@ -91,8 +108,7 @@ def _run_all_modes(tmp_path, name, dtype, device, ops, page_size=4, lengths=LENG
                                 "mixed": (mixed, peak)}.items():
         session = _session(tmp_path, cfg, weights, dtype, device, ops, room, page_size)
         got = H.collect(session, trace)
-        for rid in requests:
-            H.assert_close(got[rid], want[rid], LABEL[dtype], f"livitar {name} {mode} {rid}", tol)
+        _check(got, want, dtype, f"livitar {name} {mode}", tol)
         # everything went back to the pools
         assert session.cache.num_free_pages == [p.num_pages for p in session.cache.pools]
         assert session.cache.slots.num_free == session.cache.slots.num_slots
@@ -155,8 +171,7 @@ def test_a_wider_model_with_long_prompts(tmp_path, dtype):
                                  "mixed": (mixed, peak)}.items():
         session = _session(tmp_path / mode, cfg, weights, dtype, "cuda", get_ops("cuda"), space, 16)
         results[mode] = H.collect(session, trace)
-        for rid in requests:
-            H.assert_close(results[mode][rid], want[rid], LABEL[dtype], f"wide {mode} {rid}", tol)
+        _check(results[mode], want, dtype, f"wide {mode}", tol)
         assert session.cache.num_free_pages == [p.num_pages for p in session.cache.pools]
     ran = {n: get_ops("cuda").launch_counts.get(n, 0) - before[n] for n in names}
     if dtype == "float32":
@@ -782,7 +797,7 @@ def test_long_decoding(tmp_path, dtype):
     want = P.forward(cfg, weights, toks, D).float()
     session = _session(tmp_path, cfg, weights, dtype, "cuda", get_ops("cuda"), 448, 16)
     got = H.collect(session, H.trace_decode_tail({"a": toks}, 400))["a"]
-    H.assert_close(got, want, LABEL[dtype], "long decoding", _bound(tmp_path, dtype, cfg, weights, {"a": toks}, {"a": want}))
+    _check({"a": got}, {"a": want}, dtype, "long decoding", _bound(tmp_path, dtype, cfg, weights, {"a": toks}, {"a": want}))
 
 
 def _greedy_plain(cfg, weights, prompt, count):
@@ -871,8 +886,7 @@ def test_captured_short_steps_with_portions(tmp_path, dtype):
                 eager = session.runner.step
                 session.runner.step = lambda entries, g=graphs, e=eager: g.run(entries) if g.can_run(entries) else e(entries)
             got = H.collect(session, trace)
-            for rid in requests:
-                H.assert_close(got[rid], want[rid], LABEL[dtype], f"captured={captured} {mode} {rid}", tol)
+            _check(got, want, dtype, f"captured={captured} {mode}", tol)
             if captured:
                 assert graphs.replays > len(requests)
             results[(captured, mode)] = got
@@ -908,8 +922,7 @@ def test_captured_decoding_in_bfloat16(tmp_path):
         steps.append({"step": i + 1, "entries": [{"id": rid, "tokens": [toks[heads[rid] + i]], "want": [0]}
                                                  for rid, toks in requests.items()], "end": []})
     got = H.collect(session, steps)
-    for rid in requests:
-        H.assert_close(got[rid], want[rid], LABEL["bfloat16"], f"captured decoding {rid}", tol)
+    _check(got, want, "bfloat16", "captured decoding", tol)
     get_ops("cuda").check_errors()
 
 
