@@ -449,7 +449,7 @@ RETENTION_STEPS = [([1, 1, 3], [5, 0, 9]), ([8, 2], [0, 600]), ([150, 1, 64, 63,
 
 @pytest.mark.parametrize("device", DEVICES)
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("H,d,dv,rot", [(3, 64, 32, 64), (2, 128, 128, 64), (4, 20, 28, 10), (1, 33, 17, 0), (5, 16, 112, 16),
+@pytest.mark.parametrize("H,d,dv,rot", [(3, 64, 48, 64), (2, 128, 128, 64), (4, 20, 28, 10), (1, 33, 17, 0), (5, 16, 112, 16),
                                         (2, 100, 120, 100), (1, 1, 1, 0), (2, 144, 40, 16), (1, 6, 130, 6)])
 def test_retention_in_every_kind_of_step(device, dtype, H, d, dv, rot):
     """Requests of one to hundreds of tokens in one step, from states that others left in scattered slots:
@@ -577,7 +577,7 @@ def test_attention_with_a_bias_by_distance(device, kind):
 
 
 @pytest.mark.gpu
-@pytest.mark.parametrize("d,dv,heads,kv", [(64, 32, 6, 6), (96, 96, 6, 2), (128, 128, 4, 1), (16, 48, 5, 5), (48, 16, 8, 2),
+@pytest.mark.parametrize("d,dv,heads,kv", [(64, 48, 5, 5), (80, 112, 6, 3), (128, 128, 4, 1), (16, 48, 5, 5), (48, 16, 8, 2),
                                            (256, 64, 2, 1)])
 @pytest.mark.parametrize("kind", ["log", (16, 40), (32, 5000), (24, 150), (1, 3)], ids=str)
 def test_biased_attention_on_the_tensor_cores(d, dv, heads, kv, kind):
