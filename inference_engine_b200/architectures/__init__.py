@@ -1,1 +1,1 @@
-from . import livitar, llama, puposun, ravapel, rugedra, vofanex  # noqa: F401 (register Livitar, LlamaForCausalLM, Puposun, Ravapel, Rugedra and Vofanex)
+from . import kolisun, livitar, llama, puposun, ravapel, rugedra, vofanex  # noqa: F401 (register Kolisun, Livitar, LlamaForCausalLM, Puposun, Ravapel, Rugedra and Vofanex)

@@ -25,7 +25,7 @@
 // beside its window; they keep their own positions.
 // A bias by distance n = (query's position - key's position), added to the score after the scale:
 // -log_r1[head] * ln(1 + log_r2[head] * n), and/or a table, bias_table[head * bias_len + min(n, bias_len -
-// 1)].  `gate_elements` 1: `out_gate` holds a number per head and value entry ([token * gate_ld + head *
+// 1)].  Rows of the output lie `out_ld` entries apart.  `gate_elements` 1: `out_gate` holds a number per head and value entry ([token * gate_ld + head *
 // hdv + d]) instead of one per head.
 #include "common.cuh"
 #include <math.h>
@@ -75,7 +75,7 @@ paged_attention_generic_kernel(const T* __restrict__ q, const T* __restrict__ k_
                                const float* __restrict__ sinks, const float* __restrict__ out_gate, int gate_ld,
                                float softcap, int keep_first, int gate_elements, const float* __restrict__ log_r1,
                                const float* __restrict__ log_r2, const float* __restrict__ bias_table, int bias_len,
-                               int* err) {
+                               int out_ld, int* err) {
     extern __shared__ float q_smem[];  // [WARPS][hd]
     ie_pdl_trigger();
     ie_pdl_wait();
@@ -151,7 +151,7 @@ paged_attention_generic_kernel(const T* __restrict__ q, const T* __restrict__ k_
         }
         m = m_new;
     }
-    T* orow = out + ((size_t)token * nh + head) * hdv;
+    T* orow = out + (size_t)token * out_ld + (size_t)head * hdv;
     float inv = gated ? 1.0f : (l > 0.f ? 1.0f / l : 0.f);
     if (out_gate != nullptr && !gate_elements) inv *= 1.0f / (1.0f + expf(-out_gate[(size_t)token * gate_ld + head]));
 #pragma unroll
@@ -175,9 +175,9 @@ IE_API int ie_paged_attention_generic(const void* q, const void* k_cache, const 
                                       const float* head_bias, const float* sinks, const float* out_gate,
                                       int gate_ld, float softcap, int keep_first, int gate_elements,
                                       const float* log_r1, const float* log_r2, const float* bias_table,
-                                      int bias_len, int* err, void* stream) {
+                                      int bias_len, int out_ld, int* err, void* stream) {
     if (num_tokens <= 0) return 0;
-    if (hd < 1 || hdv < 1 || hdv > 32 * MAX_ACC || nkv <= 0 || nh % nkv != 0) return (int)cudaErrorInvalidValue;
+    if (hd < 1 || hdv < 1 || hdv > 32 * MAX_ACC || nkv <= 0 || nh % nkv != 0 || out_ld < nh * hdv) return (int)cudaErrorInvalidValue;
     if (keep_first < 0 || softcap < 0.f || (keep_first > 0 && chunk > 0)) return (int)cudaErrorInvalidValue;
     if ((log_r1 == nullptr) != (log_r2 == nullptr) || (bias_table != nullptr && bias_len < 1))
         return (int)cudaErrorInvalidValue;
@@ -189,12 +189,12 @@ IE_API int ie_paged_attention_generic(const void* q, const void* k_cache, const 
             (const __nv_bfloat16*)q, (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache,
             block_tables, table_width, seq_of_token, positions, (__nv_bfloat16*)out,
             nh, nkv, hd, hdv, v_stride, page_size, total_pages, scale, window, chunk, head_bias, sinks, out_gate, gate_ld, softcap, keep_first,
-            gate_elements, log_r1, log_r2, bias_table, bias_len, err);
+            gate_elements, log_r1, log_r2, bias_table, bias_len, out_ld, err);
     else
         paged_attention_generic_kernel<<<grid, WARPS * 32, smem, s>>>(
             (const float*)q, (const float*)k_cache, (const float*)v_cache,
             block_tables, table_width, seq_of_token, positions, (float*)out,
             nh, nkv, hd, hdv, v_stride, page_size, total_pages, scale, window, chunk, head_bias, sinks, out_gate, gate_ld, softcap, keep_first,
-            gate_elements, log_r1, log_r2, bias_table, bias_len, err);
+            gate_elements, log_r1, log_r2, bias_table, bias_len, out_ld, err);
     return IE_LAUNCH_CHECK();
 }

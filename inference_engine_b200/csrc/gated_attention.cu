@@ -17,6 +17,11 @@
 // queries go to q_out [N, heads * dim], keys and values into the request's page rows
 // (k_cache [pages, kv_heads, page_size, dim], v_cache [pages, kv_heads, page_size, vdim]).
 // One warp per (token, head of q, k or v); the sums do not depend on the rest of the step.
+//
+// qk_wide_norm_rope_write: the same stage with one norm over all query columns of a token and one over all
+// its key columns, before they are split into heads (weights as long as the columns).  A block per token.
+// `value_scale` (both kernels) multiplies the values before they are cached, for a mixer whose output is
+// wanted times a constant.
 #include "common.cuh"
 #include <math.h>
 
@@ -30,7 +35,7 @@ qk_norm_rope_write_kernel(const float* __restrict__ proj, int ld, const int* __r
                           const float* __restrict__ bias, int value_norm, int values_from_keys, int interleaved,
                           const float* __restrict__ q_weight, const float* __restrict__ k_weight, float eps,
                           int unit_norm, const float* __restrict__ q_head_scale, float warm_coef, int warm_every,
-                          T* __restrict__ q_out, T* __restrict__ k_cache, T* __restrict__ v_cache,
+                          float value_scale, T* __restrict__ q_out, T* __restrict__ k_cache, T* __restrict__ v_cache,
                           const int* __restrict__ slot_mapping, int heads, int kv_heads, int dim, int vdim,
                           int page_size, int total_pages, int* err) {
     extern __shared__ float rows[];  // [QW_WARPS][dim]
@@ -59,7 +64,7 @@ qk_norm_rope_write_kernel(const float* __restrict__ proj, int ld, const int* __r
         size_t col = values_from_keys ? (size_t)(heads + g) * dim : (size_t)(heads + kv_heads) * dim + (size_t)g * vdim;
         const float* v = src + col;
         const float* vb = bias != nullptr ? bias + col : nullptr;
-        float inv = 1.0f;
+        float inv = value_scale;
         if (value_norm) {
             float ss = 0.f;
             for (int d = lane; d < vdim; d += 32) {
@@ -67,7 +72,7 @@ qk_norm_rope_write_kernel(const float* __restrict__ proj, int ld, const int* __r
                 ss = fmaf(e, e, ss);
             }
             ss = warp_sum(ss);
-            inv = 1.0f / sqrtf(ss / (float)vdim + eps);
+            inv = value_scale / sqrtf(ss / (float)vdim + eps);
         }
         for (int d = lane; d < vdim; d += 32)
             ie_store(v_cache + cache_row * vdim + d, (vb != nullptr ? v[d] + vb[d] : v[d]) * inv);
@@ -119,13 +124,83 @@ qk_norm_rope_write_kernel(const float* __restrict__ proj, int ld, const int* __r
         ie_store(dst + d, r * factor);
     }
 }
+
+constexpr int WN_THREADS = 256;
+
+__device__ __forceinline__ float wide_sum(float v, float* red) {
+    v = warp_sum(v);
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+    __syncthreads();
+    float total = 0.f;
+#pragma unroll
+    for (int w = 0; w < WN_THREADS / 32; ++w) total += red[w];
+    return total;
+}
+
+template <typename T>
+__global__ void __launch_bounds__(WN_THREADS)
+qk_wide_norm_rope_write_kernel(const float* __restrict__ proj, int ld, const int* __restrict__ positions,
+                               const float* __restrict__ table, int rot_dims, int table_positions,
+                               const float* __restrict__ bias, int interleaved, const float* __restrict__ q_weight,
+                               const float* __restrict__ k_weight, float eps, float value_scale, T* __restrict__ q_out,
+                               T* __restrict__ k_cache, T* __restrict__ v_cache, const int* __restrict__ slot_mapping,
+                               int heads, int kv_heads, int dim, int vdim, int page_size, int total_pages, int* err) {
+    extern __shared__ float row[];  // the token's query columns, then its key columns
+    __shared__ float red_q[WN_THREADS / 32], red_k[WN_THREADS / 32];
+    ie_pdl_trigger();
+    ie_pdl_wait();
+    const int n = blockIdx.x, tid = threadIdx.x, nq = heads * dim, nqk = (heads + kv_heads) * dim;
+    const float* src = proj + (size_t)n * ld;
+    float sq = 0.f, sk = 0.f;
+    for (int i = tid; i < nqk; i += WN_THREADS) {
+        float e = bias != nullptr ? src[i] + bias[i] : src[i];
+        row[i] = e;
+        if (i < nq) sq = fmaf(e, e, sq);
+        else sk = fmaf(e, e, sk);
+    }
+    const float inv_q = 1.0f / sqrtf(wide_sum(sq, red_q) / (float)nq + eps);
+    const float inv_k = 1.0f / sqrtf(wide_sum(sk, red_k) / (float)(nqk - nq) + eps);
+    for (int i = tid; i < nqk; i += WN_THREADS) row[i] = (row[i] * (i < nq ? inv_q : inv_k)) * (i < nq ? q_weight[i] : k_weight[i - nq]);
+    __syncthreads();
+    const int pos = positions[n], half = rot_dims / 2;
+    if (half > 0 && (pos < 0 || pos >= table_positions)) {
+        if (tid == 0) ie_report(err, IE_ERR_POSITION, pos, n);
+        return;
+    }
+    int slot = slot_mapping != nullptr ? slot_mapping[n] : -1, page = slot / page_size;
+    bool writes = slot_mapping != nullptr;
+    if (writes && (slot < 0 || page >= total_pages)) {
+        if (tid == 0) ie_report(err, IE_ERR_PAGE, slot, n);
+        writes = false;
+    }
+    const float* cs = table + (size_t)max(pos, 0) * rot_dims;  // cos of the angles, then their sin
+    const long long first_row = (long long)page * kv_heads * page_size + (slot - page * page_size);
+    for (int i = tid; i < (writes ? nqk : nq); i += WN_THREADS) {
+        int unit = i / dim, d = i - unit * dim;
+        float r = row[i];
+        if (d < rot_dims) {
+            int j = interleaved ? d >> 1 : (d < half ? d : d - half);
+            bool second = interleaved ? (d & 1) : d >= half;
+            float c = cs[j], s = cs[half + j], other = row[interleaved ? (second ? i - 1 : i + 1) : (second ? i - half : i + half)];
+            r = second ? r * c + other * s : r * c - other * s;
+        }
+        if (i < nq) ie_store(q_out + (size_t)n * nq + i, r);
+        else ie_store(k_cache + (first_row + (long long)(unit - heads) * page_size) * dim + d, r);
+    }
+    if (!writes) return;
+    for (int i = tid; i < kv_heads * vdim; i += WN_THREADS) {
+        int g = i / vdim, d = i - g * vdim;
+        float e = bias != nullptr ? src[nqk + i] + bias[nqk + i] : src[nqk + i];
+        ie_store(v_cache + (first_row + (long long)g * page_size) * vdim + d, e * value_scale);
+    }
+}
 }  // namespace
 
 IE_API int ie_qk_norm_rope_write(const float* proj, int ld, const int* positions, const float* table, int rot_dims,
                                  int table_positions, const float* bias, int value_norm, int values_from_keys,
                                  int interleaved, const float* q_weight,
                                  const float* k_weight, float eps, int unit_norm, const float* q_head_scale,
-                                 float warm_coef, int warm_every, void* q_out, void* k_cache, void* v_cache, int dtype, const int* slot_mapping,
+                                 float warm_coef, int warm_every, float value_scale, void* q_out, void* k_cache, void* v_cache, int dtype, const int* slot_mapping,
                                  int num_tokens, int heads, int kv_heads, int dim, int vdim, int page_size,
                                  int total_pages, int* err, void* stream) {
     if (num_tokens <= 0) return 0;
@@ -139,10 +214,40 @@ IE_API int ie_qk_norm_rope_write(const float* proj, int ld, const int* positions
     cudaStream_t s = (cudaStream_t)stream;
     if (dtype == IE_BF16)
         return ie_launch(qk_norm_rope_write_kernel<__nv_bfloat16>, grid, dim3(QW_WARPS * 32), smem, s, proj, ld,
-                         positions, table, rot_dims, table_positions, bias, value_norm, values_from_keys, interleaved, q_weight, k_weight, eps, unit_norm, q_head_scale, warm_coef, warm_every, (__nv_bfloat16*)q_out,
+                         positions, table, rot_dims, table_positions, bias, value_norm, values_from_keys, interleaved, q_weight, k_weight, eps, unit_norm, q_head_scale, warm_coef, warm_every, value_scale, (__nv_bfloat16*)q_out,
                          (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, slot_mapping, heads, kv_heads, dim, vdim,
                          page_size, total_pages, err);
     return ie_launch(qk_norm_rope_write_kernel<float>, grid, dim3(QW_WARPS * 32), smem, s, proj, ld, positions, table,
-                     rot_dims, table_positions, bias, value_norm, values_from_keys, interleaved, q_weight, k_weight, eps, unit_norm, q_head_scale, warm_coef, warm_every, (float*)q_out, (float*)k_cache,
+                     rot_dims, table_positions, bias, value_norm, values_from_keys, interleaved, q_weight, k_weight, eps, unit_norm, q_head_scale, warm_coef, warm_every, value_scale, (float*)q_out, (float*)k_cache,
                      (float*)v_cache, slot_mapping, heads, kv_heads, dim, vdim, page_size, total_pages, err);
+}
+
+IE_API int ie_qk_wide_norm_rope_write(const float* proj, int ld, const int* positions, const float* table, int rot_dims,
+                                      int table_positions, const float* bias, int interleaved, const float* q_weight,
+                                      const float* k_weight, float eps, float value_scale, void* q_out, void* k_cache,
+                                      void* v_cache, int dtype, const int* slot_mapping, int num_tokens, int heads,
+                                      int kv_heads, int dim, int vdim, int page_size, int total_pages, int* err,
+                                      void* stream) {
+    if (num_tokens <= 0) return 0;
+    if (rot_dims < 0 || rot_dims % 2 || rot_dims > dim || (rot_dims > 0 && table == nullptr) || q_weight == nullptr ||
+        k_weight == nullptr)
+        return (int)cudaErrorInvalidValue;
+    size_t smem = (size_t)(heads + kv_heads) * dim * sizeof(float);
+    if (smem > 200 * 1024) return (int)cudaErrorInvalidValue;
+    cudaStream_t s = (cudaStream_t)stream;
+#define IE_WN_LAUNCH(T)                                                                                              \
+    do {                                                                                                             \
+        static IePerDevice allowed;                                                                                  \
+        if (smem > 40 * 1024) {                                                                                      \
+            cudaError_t e = ie_allow_smem(allowed, qk_wide_norm_rope_write_kernel<T>, 200 * 1024);                   \
+            if (e != cudaSuccess) return (int)e;                                                                     \
+        }                                                                                                            \
+        return ie_launch(qk_wide_norm_rope_write_kernel<T>, dim3(num_tokens), dim3(WN_THREADS), smem, s, proj, ld,   \
+                         positions, table, rot_dims, table_positions, bias, interleaved, q_weight, k_weight, eps,    \
+                         value_scale, (T*)q_out, (T*)k_cache, (T*)v_cache, slot_mapping, heads, kv_heads, dim, vdim, \
+                         page_size, total_pages, err);                                                               \
+    } while (0)
+    if (dtype == IE_BF16) IE_WN_LAUNCH(__nv_bfloat16);
+    IE_WN_LAUNCH(float);
+#undef IE_WN_LAUNCH
 }

@@ -19,7 +19,14 @@
 //    token's numbers for all of them: a token stride of 0), w_t = k_t, u_t = v_t with q and k rotated by
 //    position; the read-out's unit root mean square has no weight.
 //
-// Kernels: rotate_heads (in place in the 32-bit projection: the first rot_dims entries of every head, by
+//  * state-space duality (Mamba-2): a_t = exp(-exp(A_log) dt_t) and the write gate dt_t are one number per head,
+//    dt_t = softplus(. + dt_bias); w_t = B_t and q_t = C_t belong to groups of heads (`heads_per_unit` heads read the
+//    same rows of q and w), u_t = dt_t x_t; x, B and C come from a short convolution with a bias and silu.
+//    y_t = S_t^T C_t + D x_t, times silu(z_t), then divided by its root mean square in equal parts of the row.
+//
+// Kernels: conv_silu (the convolution over the step's tokens and, before them, the slot's kept inputs; a thread
+// takes a channel through sixteen tokens) with the heads' gates in the same launch; gated_group_norm (skip, gate, norm in parts,
+// weight; it also moves the slot's kept convolution inputs on, which no earlier kernel of the step may do); rotate_heads (in place in the 32-bit projection: the first rot_dims entries of every head, by
 // pairs (i, i + rot_dims / 2), from the 32-bit table of angles); lowrank_decay (a block takes sixteen tokens and 128 channels, so that a row of W2 is read
 // once per sixteen tokens); short_conv_residual (+ tail update): out = x + causal convolution of x over time per
 // channel, the last taps - 1 inputs kept per request; hgrn2_gates; mlstm_gates (a warp per request
@@ -223,6 +230,132 @@ lowrank_decay_kernel(const float* __restrict__ y, int y_ld, const float* __restr
         if (t < cnt) decay[(size_t)(n0 + t) * channels + c] = expf(logsigmoid_f(acc[t] + b) * inv_tau);
 }
 
+// The short convolution with bias and silu of a 32-bit projection, and the state-space heads' gates.
+// grid: (blocks of CS_TOKENS tokens, blocks of 128 channels, + 1 for the gates).  x: [N, x_ld] 32-bit; w: [channels,
+// taps], the last tap weighs the token itself; tail: the slot's kept inputs [taps - 1][channels], oldest first, at
+// `tail_at` of the slot; out: [N, out_ld].  TAPS 0: any number of taps, each fetched anew.
+// gates: [N, heads, 3] = (exp(-exp(A_log) dt), dt, -exp(A_log) dt), dt = softplus(dt_pre + dt_bias).
+constexpr int CS_TOKENS = 16;
+__device__ __forceinline__ float softplus_f(float y) { return y > 20.0f ? y : log1pf(expf(y)); }
+
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(128)
+conv_silu_kernel(const float* __restrict__ x, int x_ld, const float* __restrict__ w, const float* __restrict__ bias,
+                 const float* __restrict__ state, long long state_stride, long long tail_at,
+                 const int* __restrict__ slots, const int* __restrict__ seq_of_token, const int* __restrict__ cu_q,
+                 T* __restrict__ out, int out_ld, int num_tokens, int channels, int taps, int num_slots,
+                 const float* __restrict__ dt_pre, const float* __restrict__ dt_bias, const float* __restrict__ A_log,
+                 float* __restrict__ gates, int heads, int* err) {
+    ie_pdl_trigger();
+    ie_pdl_wait();
+    const int n0 = blockIdx.x * CS_TOKENS, n1 = min(n0 + CS_TOKENS, num_tokens);
+    if (blockIdx.y + 1 == gridDim.y) {
+        for (int i = threadIdx.x; i < (n1 - n0) * heads; i += blockDim.x) {
+            int r = i / heads, h = i - r * heads;
+            size_t n = (size_t)(n0 + r);
+            float dt = softplus_f(dt_pre[n * x_ld + h] + dt_bias[h]);
+            float a = -expf(A_log[h]) * dt;
+            float* g = gates + (n * heads + h) * 3;
+            g[0] = expf(a);
+            g[1] = dt;
+            g[2] = a;
+        }
+        return;
+    }
+    const int c = blockIdx.y * 128 + threadIdx.x;
+    const bool live = c < channels;
+    const float b = live && bias != nullptr ? bias[c] : 0.f;
+    constexpr int KEEP = TAPS > 1 ? TAPS - 1 : 1;
+    float wt[TAPS > 0 ? TAPS : 1], before[KEEP];  // before[i]: the input i + 1 tokens back
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) wt[j] = live ? w[(size_t)c * taps + j] : 0.f;
+    int seq = -1, first = 0, slot = -1;
+    const float* tail = nullptr;
+    for (int n = n0; n < n1; ++n) {
+        int s = seq_of_token[n];
+        bool fresh = s != seq;
+        if (fresh) {
+            seq = s;
+            first = cu_q[seq];
+            slot = slots[seq];
+            if (slot < 0 || slot >= num_slots) {
+                if (threadIdx.x == 0) ie_report(err, IE_ERR_PAGE, slot, n);
+                return;
+            }
+            tail = state + (size_t)slot * state_stride + tail_at;
+        }
+        if (!live) continue;
+        const int t = n - first;
+        auto earlier = [&](int back) {
+            return t - back >= 0 ? x[(size_t)(n - back) * x_ld + c] : tail[(size_t)(taps - 1 + t - back) * channels + c];
+        };
+        float acc = b, own = x[(size_t)n * x_ld + c];
+        if (TAPS > 0) {
+            if (fresh)
+#pragma unroll
+                for (int i = 0; i < TAPS - 1; ++i) before[i] = earlier(i + 1);
+#pragma unroll
+            for (int j = 0; j < TAPS - 1; ++j) acc = fmaf(wt[j], before[TAPS - 2 - j], acc);
+            acc = fmaf(wt[TAPS > 0 ? TAPS - 1 : 0], own, acc);
+#pragma unroll
+            for (int i = KEEP - 1; i > 0; --i) before[i] = before[i - 1];
+            before[0] = own;
+        } else {
+            for (int j = 0; j < taps - 1; ++j) acc = fmaf(w[(size_t)c * taps + j], earlier(taps - 1 - j), acc);
+            acc = fmaf(w[(size_t)c * taps + taps - 1], own, acc);
+        }
+        ie_store(out + (size_t)n * out_ld + c, silu_f(acc));
+    }
+}
+
+// grid: (tokens, parts).  y: [N, size] 32-bit; with `x` (the convolved values, [N, x_ld]) D[head] x is added, and
+// with `z` ([N, z_ld] 32-bit) the sum is multiplied by silu(z); then each of the row's equal parts is divided by
+// its root mean square and multiplied by the weight.  The blocks of a request's last token also move its kept
+// convolution inputs on: channels [part's share] of `raw` ([N, raw_ld], 32-bit).
+constexpr int GN_THREADS = 256;
+template <typename T>
+__global__ void __launch_bounds__(GN_THREADS)
+gated_group_norm_kernel(const float* __restrict__ y, const float* __restrict__ x, int x_ld, const float* __restrict__ skip,
+                        const float* __restrict__ z, int z_ld, const float* __restrict__ weight, float eps,
+                        T* __restrict__ out, int out_ld, int size, int parts, int vdim,
+                        const float* __restrict__ raw, int raw_ld, float* __restrict__ state, long long state_stride,
+                        long long tail_at, const int* __restrict__ slots, const int* __restrict__ seq_of_token,
+                        const int* __restrict__ cu_q, int channels, int taps, int num_slots) {
+    extern __shared__ float part_buf[];  // [size / parts]
+    __shared__ float red[GN_THREADS / 32];
+    ie_pdl_trigger();
+    ie_pdl_wait();
+    const int n = blockIdx.x, part = blockIdx.y, width = size / parts, at = part * width;
+    const float* yr = y + (size_t)n * size + at;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < width; i += GN_THREADS) {
+        float v = yr[i];
+        if (x != nullptr) v = fmaf(skip[(at + i) / vdim], x[(size_t)n * x_ld + at + i], v);
+        if (z != nullptr) v *= silu_f(z[(size_t)n * z_ld + at + i]);
+        part_buf[i] = v;
+        ss = fmaf(v, v, ss);
+    }
+    ss = warp_sum(ss);
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
+    __syncthreads();
+    float total = 0.f;
+#pragma unroll
+    for (int w = 0; w < GN_THREADS / 32; ++w) total += red[w];
+    const float inv = 1.0f / sqrtf(total / (float)width + eps);
+    for (int i = threadIdx.x; i < width; i += GN_THREADS)
+        ie_store(out + (size_t)n * out_ld + at + i, part_buf[i] * inv * weight[at + i]);
+    if (raw == nullptr || taps < 2) return;
+    const int seq = seq_of_token[n], start = cu_q[seq], end = cu_q[seq + 1], slot = slots[seq];
+    if (n != end - 1 || slot < 0 || slot >= num_slots) return;  // (a captured step's padding belongs to no request)
+    float* tail = state + (size_t)slot * state_stride + tail_at;
+    const int len = end - start, share = (channels + parts - 1) / parts;
+    for (int c = part * share + threadIdx.x; c < min(channels, (part + 1) * share); c += GN_THREADS)
+        for (int j = 0; j < taps - 1; ++j) {  // (rising: a kept row is read before it is overwritten)
+            int tt = len - (taps - 1) + j;
+            tail[(size_t)j * channels + c] = tt >= 0 ? raw[(size_t)(start + tt) * raw_ld + c] : tail[(size_t)(taps - 1 + tt) * channels + c];
+        }
+}
+
 constexpr int GR_THREADS = 128;
 constexpr int GR_CHUNK = 8;  // tokens staged in shared memory at a time
 constexpr int GR_STAGES = 4;  // ... in a ring of so many buffers: three chunks are on their way while one is worked on
@@ -237,7 +370,8 @@ __device__ __forceinline__ void cp_async16(float* dst, const float* src) {
 }
 
 // grid: (column blocks, heads, requests).  Lane `sub` of a column's TPC lanes holds rows sub, sub + TPC,
-// ..., R of them.  q, a, w: element (n, head, d) at [n * ld + head * dim + d]; SCALAR: a and the write
+// ..., R of them.  q, a, w: element (n, head, d) at [n * ld + head * dim + d] (q and w: head / heads_per_unit in
+// head's place); SCALAR: a and the write
 // gate b come from gates[n * gate_stride + head * 3 + {0, 1}] and column `vdim` (if cols > vdim) has the
 // value 1.  v: (n, head, c) at [n * v_ld + head * vdim + c].  out: [N, heads, cols], times q_scale.
 template <int R, int TPC, bool SCALAR>
@@ -246,8 +380,8 @@ gated_recurrence_kernel(const float* __restrict__ q, int q_ld, const float* __re
                         const float* __restrict__ w, int w_ld, const float* __restrict__ gates,
                         int gate_stride, const float* __restrict__ v, int v_ld, float* __restrict__ state,
                         long long state_stride, const int* __restrict__ slots, const int* __restrict__ cu_q,
-                        float* __restrict__ out, int heads, int dim, int vdim, int cols, float q_scale,
-                        int num_slots) {
+                        float* __restrict__ out, int heads, int heads_per_unit, int dim, int vdim, int cols,
+                        float q_scale, int num_slots) {
     extern __shared__ __align__(16) float sm[];
     constexpr int COLS = GR_THREADS / TPC, DP = R * TPC;
     constexpr int ROWS = SCALAR ? 2 : 3;  // arrays of DP floats per token: q, w (, a)
@@ -258,6 +392,7 @@ gated_recurrence_kernel(const float* __restrict__ q, int q_ld, const float* __re
     int start = cu_q[seq], len = cu_q[seq + 1] - start;
     int slot = slots[seq];
     if (len <= 0 || slot < 0 || slot >= num_slots) return;
+    const int unit = head / heads_per_unit;
     int tid = threadIdx.x;
     int sub = tid % TPC, my_col = tid / TPC, col = blockIdx.x * COLS + my_col;
     bool live = col < cols;
@@ -293,16 +428,16 @@ gated_recurrence_kernel(const float* __restrict__ q, int q_ld, const float* __re
             for (int i = tid; i < cnt * dq; i += GR_THREADS) {
                 int tt = i / dq, d = (i - tt * dq) * 4;
                 size_t n = (size_t)(start + t0 + tt);
-                cp_async16(qs + tt * DP + d, q + n * q_ld + head * dim + d);
-                cp_async16(ws + tt * DP + d, w + n * w_ld + head * dim + d);
+                cp_async16(qs + tt * DP + d, q + n * q_ld + unit * dim + d);
+                cp_async16(ws + tt * DP + d, w + n * w_ld + unit * dim + d);
                 if (!SCALAR) cp_async16(as + tt * DP + d, a + n * a_ld + head * dim + d);
             }
         } else {
             for (int i = tid; i < cnt * dim; i += GR_THREADS) {
                 int tt = i / dim, d = i - tt * dim;
                 size_t n = (size_t)(start + t0 + tt);
-                cp_async4(qs + tt * DP + d, q + n * q_ld + head * dim + d);
-                cp_async4(ws + tt * DP + d, w + n * w_ld + head * dim + d);
+                cp_async4(qs + tt * DP + d, q + n * q_ld + unit * dim + d);
+                cp_async4(ws + tt * DP + d, w + n * w_ld + unit * dim + d);
                 if (!SCALAR) cp_async4(as + tt * DP + d, a + n * a_ld + head * dim + d);
             }
         }
@@ -422,8 +557,8 @@ inline int grid_for(size_t total, int threads) {
 template <int R, int TPC, bool SCALAR>
 int launch_recurrence(const float* q, int q_ld, const float* a, int a_ld, const float* w, int w_ld,
                       const float* gates, int gate_stride, const float* v, int v_ld, float* state,
-                      long long state_stride, const int* slots, const int* cu_q, float* out, int num_seqs, int heads, int dim, int vdim,
-                      int cols, float q_scale, int num_slots, cudaStream_t s) {
+                      long long state_stride, const int* slots, const int* cu_q, float* out, int num_seqs, int heads,
+                      int heads_per_unit, int dim, int vdim, int cols, float q_scale, int num_slots, cudaStream_t s) {
     constexpr int COLS = GR_THREADS / TPC;
     size_t smem = (size_t)GR_STAGES * GR_CHUNK * ((SCALAR ? 2 : 3) * R * TPC + COLS + 4) * sizeof(float);
     static IePerDevice allowed;
@@ -431,8 +566,8 @@ int launch_recurrence(const float* q, int q_ld, const float* a, int a_ld, const 
     if (e != cudaSuccess) return (int)e;
     dim3 grid((cols + COLS - 1) / COLS, heads, num_seqs);
     return ie_launch(gated_recurrence_kernel<R, TPC, SCALAR>, grid, dim3(GR_THREADS), smem, s, q, q_ld, a, a_ld, w,
-                     w_ld, gates, gate_stride, v, v_ld, state, state_stride, slots, cu_q, out, heads, dim, vdim, cols, q_scale,
-                     num_slots);
+                     w_ld, gates, gate_stride, v, v_ld, state, state_stride, slots, cu_q, out, heads, heads_per_unit, dim, vdim, cols,
+                     q_scale, num_slots);
 }
 }  // namespace
 
@@ -505,13 +640,14 @@ IE_API int ie_mlstm_gates(const float* gi, const float* gf, int ld, const float*
 // `gate_stride` numbers apart (0: the same for every token).
 IE_API int ie_gated_recurrence(const float* q, int q_ld, const float* a, int a_ld, const float* w, int w_ld,
                                const float* gates, int gate_stride, const float* v, int v_ld, float* state,
-                               long long state_stride, const int* slots, const int* cu_q, float* out, int num_seqs, int heads, int dim,
-                               int vdim, int cols, float q_scale, int num_slots, void* stream) {
+                               long long state_stride, const int* slots, const int* cu_q, float* out, int num_seqs, int heads,
+                               int heads_per_unit, int dim, int vdim, int cols, float q_scale, int num_slots, void* stream) {
     if (num_seqs <= 0) return 0;
+    if (heads_per_unit < 1 || heads % heads_per_unit) return (int)cudaErrorInvalidValue;
     if (cols < vdim || cols > vdim + 1 || (gates == nullptr && (a == nullptr || cols != vdim)))
         return (int)cudaErrorInvalidValue;
     cudaStream_t s = (cudaStream_t)stream;
-#define IE_GR_ARGS q, q_ld, a, a_ld, w, w_ld, gates, gate_stride, v, v_ld, state, state_stride, slots, cu_q, out, num_seqs, heads, dim, vdim, cols, q_scale, num_slots, s
+#define IE_GR_ARGS q, q_ld, a, a_ld, w, w_ld, gates, gate_stride, v, v_ld, state, state_stride, slots, cu_q, out, num_seqs, heads, heads_per_unit, dim, vdim, cols, q_scale, num_slots, s
 #define IE_GR_PICK(SC)                                                        \
     if (dim <= 8) return launch_recurrence<8, 1, SC>(IE_GR_ARGS);             \
     if (dim <= 16) return launch_recurrence<8, 2, SC>(IE_GR_ARGS);            \
@@ -537,4 +673,57 @@ IE_API int ie_recurrence_readout(const float* o, int cols, const float* gates, c
                          weight_per_head, eps, gate_pre, gate_ld, gate_silu, (__nv_bfloat16*)out, rows, heads, vdim);
     return ie_launch(recurrence_readout_kernel<float>, grid, dim3(128), 0, s, o, cols, gates, weight,
                      weight_per_head, eps, gate_pre, gate_ld, gate_silu, (float*)out, rows, heads, vdim);
+}
+
+// `out_dtype`: of the convolved values.  gates == nullptr: the convolution alone.
+IE_API int ie_conv_silu(const float* x, int x_ld, const float* w, const float* bias, const float* state,
+                        long long state_stride, long long tail_at, const int* slots, const int* seq_of_token,
+                        const int* cu_q, void* out, int out_ld, int out_dtype, int num_tokens, int channels, int taps,
+                        int num_slots, const float* dt_pre, const float* dt_bias, const float* A_log, float* gates,
+                        int heads, int* err, void* stream) {
+    if (num_tokens <= 0) return 0;
+    if (taps < 1 || channels < 1 || out_ld < channels) return (int)cudaErrorInvalidValue;
+    cudaStream_t s = (cudaStream_t)stream;
+    dim3 grid((num_tokens + CS_TOKENS - 1) / CS_TOKENS, (channels + 127) / 128 + 1);
+    if (gates == nullptr) heads = 0;
+#define IE_CS_LAUNCH(T, TAPS)                                                                                        \
+    return ie_launch(conv_silu_kernel<T, TAPS>, grid, dim3(128), 0, s, x, x_ld, w, bias, state, state_stride,        \
+                     tail_at, slots, seq_of_token, cu_q, (T*)out, out_ld, num_tokens, channels, taps, num_slots,     \
+                     dt_pre, dt_bias, A_log, gates, heads, err)
+#define IE_CS_PICK(T)                      \
+    if (taps == 2) IE_CS_LAUNCH(T, 2);     \
+    if (taps == 3) IE_CS_LAUNCH(T, 3);     \
+    if (taps == 4) IE_CS_LAUNCH(T, 4);     \
+    IE_CS_LAUNCH(T, 0)
+    if (out_dtype == IE_BF16) { IE_CS_PICK(__nv_bfloat16); }
+    IE_CS_PICK(float);
+#undef IE_CS_PICK
+#undef IE_CS_LAUNCH
+}
+
+// x, z, raw may be null: no skip, no gate, no kept inputs to move on.
+IE_API int ie_gated_group_norm(const float* y, const float* x, int x_ld, const float* skip, const float* z, int z_ld,
+                               const float* weight, float eps, void* out, int out_ld, int out_dtype, int num_tokens,
+                               int size, int parts, int vdim, const float* raw, int raw_ld, float* state,
+                               long long state_stride, long long tail_at, const int* slots, const int* seq_of_token,
+                               const int* cu_q, int channels, int taps, int num_slots, void* stream) {
+    if (num_tokens <= 0) return 0;
+    if (parts < 1 || size % parts || vdim < 1 || out_ld < size) return (int)cudaErrorInvalidValue;
+    size_t smem = (size_t)(size / parts) * sizeof(float);
+    if (smem > 200 * 1024) return (int)cudaErrorInvalidValue;
+    cudaStream_t s = (cudaStream_t)stream;
+#define IE_GG_LAUNCH(T)                                                                                              \
+    do {                                                                                                             \
+        static IePerDevice allowed;                                                                                  \
+        if (smem > 40 * 1024) {                                                                                      \
+            cudaError_t e = ie_allow_smem(allowed, gated_group_norm_kernel<T>, 200 * 1024);                          \
+            if (e != cudaSuccess) return (int)e;                                                                     \
+        }                                                                                                            \
+        return ie_launch(gated_group_norm_kernel<T>, dim3(num_tokens, parts), dim3(GN_THREADS), smem, s, y, x, x_ld, \
+                         skip, z, z_ld, weight, eps, (T*)out, out_ld, size, parts, vdim, raw, raw_ld, state,         \
+                         state_stride, tail_at, slots, seq_of_token, cu_q, channels, taps, num_slots);               \
+    } while (0)
+    if (out_dtype == IE_BF16) IE_GG_LAUNCH(__nv_bfloat16);
+    IE_GG_LAUNCH(float);
+#undef IE_GG_LAUNCH
 }

@@ -1,34 +1,70 @@
 // Kernels of the latent attention mixer besides the attention itself (which is the general paged
-// kernel with value rows inside the key rows):
+// kernel with value rows inside the key rows, or the tensor-core kernel of latent_attention_mma.cu):
 //
-//  * latent_prep: from the fused input projection's 32-bit output, per token: the queries'
-//    unrotated parts, the queries' rotated parts (turned, written behind the latent part of the
-//    query rows the attention reads), the heads' output gates, and the cached row: the latent
-//    (divided by its root mean square, times a weight) followed by the shared rotated key part.
+//  * latent_prep: from the 32-bit products of the mixer's input, per token, whichever of these are asked for:
+//    the queries' unrotated parts and their rotated parts (turned, written behind the latent part of the
+//    query rows the attention reads); the heads' output gates; the cached row: the latent (divided by
+//    its root mean square, times a weight) followed by the shared rotated key part; the queries' own
+//    latent (divided by its root mean square, times a weight), from which another product makes the queries.
 //  * headwise_linear: out[n, h, :] = W[h] x[n, h, :] (times an optional factor per token and
 //    head): the products that move the per-head key and value matrices to the query side.
+//  * headwise_mma: the same on the tensor cores (bfloat16) for steps of up to some hundred tokens; it can
+//    read the 32-bit queries themselves and turn their rotated parts on the way, so that a step that follows
+//    the queries' product needs one launch for everything up to the attention.
 //
-// Rotation: entries 2i and 2i+1 of the rotated part form a pair for i < rot_dims / 2,
-// (u, v) -> (u cos a - v sin a, v cos a + u sin a) with a = position * base^(-2i / rot_dims) from the
-// 32-bit table [positions, 2, rot_dims / 2]; entries from rot_dims on pass unchanged.
+// Rotation of the first rot_dims entries of the rotated part, a = position * frequency from the 32-bit table
+// [positions, 2, rot_dims / 2] (cosines, then sines, with whatever factor the encoding has): entries 2i and
+// 2i+1 form a pair, or (halves) entries i and i + rot_dims / 2; (u, v) -> (u cos a - v sin a, v cos a + u sin a);
+// entries from rot_dims on pass unchanged.
 // All arithmetic is 32-bit; results are rounded once to the output's dtype.
 #include "common.cuh"
 
 namespace {
 
+// entry d of a rotated part `src`, turned by the angles at `cs` (null: not turned)
+__device__ __forceinline__ float turned(const float* src, int d, const float* cs, int rot_dims, int interleaved) {
+    float v = src[d];
+    if (cs == nullptr || d >= rot_dims) return v;
+    int half = rot_dims / 2;
+    int j = interleaved ? d >> 1 : (d < half ? d : d - half);
+    bool second = interleaved ? (d & 1) != 0 : d >= half;
+    float c = cs[j], s = cs[half + j];
+    if (second) return fmaf(v, c, src[interleaved ? d - 1 : d - half] * s);
+    return fmaf(v, c, -src[interleaved ? d + 1 : d + half] * s);
+}
+
+__device__ __forceinline__ float rms_factor(const float* x, int size, float eps, float* red) {
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < size; i += blockDim.x) ss = fmaf(x[i], x[i], ss);
+    ss = warp_sum(ss);
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
+    __syncthreads();
+    return 1.0f / sqrtf((red[0] + red[1] + red[2] + red[3]) / (float)size + eps);
+}
+
+// What a call asks for is what has a pointer: queries (q), gates (gate_pre), the cached row (dkv and
+// slot_mapping), the queries' latent (cq).  Each input is a row `*_ld` numbers long per token.
+struct LatentIn {
+    const float* q; int q_ld;
+    const float* gate_pre; int gate_ld;
+    const float* dkv; int dkv_ld;
+    const float* cq; int cq_ld, q_rank;
+    const float* norm_w;
+    const float* cq_norm_w;
+    float eps;
+};
+
 template <typename T>
 __global__ void __launch_bounds__(128)
-latent_prep_kernel(const float* __restrict__ proj, int ld, const int* __restrict__ positions,
-                   const float* __restrict__ table, int rot_dims, int table_rows,
-                   const float* __restrict__ norm_w, float eps, T* __restrict__ q_plain,
-                   T* __restrict__ q_abs, float* __restrict__ gate, T* __restrict__ cache,
-                   const int* __restrict__ slot_mapping, int heads, int dim, int rot_dim, int rank,
-                   int total_slots, int* err) {
-    __shared__ float red[4];
+latent_prep_kernel(LatentIn in, const int* __restrict__ positions,
+                   const float* __restrict__ table, int rot_dims, int table_rows, int interleaved,
+                   T* __restrict__ q_plain, T* __restrict__ q_abs, float* __restrict__ gate, T* __restrict__ cq_out,
+                   T* __restrict__ cache, const int* __restrict__ slot_mapping, int heads, int dim, int rot_dim,
+                   int rank, int total_slots, int* err) {
+    __shared__ float red[4], red_cq[4];
     ie_pdl_trigger();
     ie_pdl_wait();
     int n = blockIdx.x, tid = threadIdx.x;
-    const float* row = proj + (size_t)n * ld;
     int hq = dim + rot_dim, krow = rank + rot_dim;
     int pos = positions[n];
     bool turn = table != nullptr && rot_dims > 0;
@@ -37,52 +73,40 @@ latent_prep_kernel(const float* __restrict__ proj, int ld, const int* __restrict
         turn = false;
     }
     const float* cs = turn ? table + (size_t)pos * rot_dims : nullptr;  // cos [rot_dims/2], then sin
-    int half = rot_dims / 2;
 
-    // queries: unrotated parts as they are, rotated parts behind the latent part of the query rows
-    for (int i = tid; i < heads * dim; i += blockDim.x) {
-        int h = i / dim, d = i - h * dim;
-        ie_store(q_plain + (size_t)n * heads * dim + i, row[h * hq + d]);
-    }
-    for (int i = tid; i < heads * rot_dim; i += blockDim.x) {
-        int h = i / rot_dim, d = i - h * rot_dim;
-        const float* src = row + h * hq + dim;
-        float v = src[d];
-        if (turn && d < rot_dims) {
-            int j = d >> 1;
-            float c = cs[j], s = cs[half + j];
-            v = (d & 1) ? fmaf(src[d], c, src[d - 1] * s) : fmaf(src[d], c, -src[d + 1] * s);
+    if (in.q != nullptr) {
+        // queries: unrotated parts as they are, rotated parts behind the latent part of the query rows
+        const float* row = in.q + (size_t)n * in.q_ld;
+        for (int i = tid; i < heads * dim; i += blockDim.x) {
+            int h = i / dim, d = i - h * dim;
+            ie_store(q_plain + (size_t)n * heads * dim + i, row[h * hq + d]);
         }
-        ie_store(q_abs + ((size_t)n * heads + h) * krow + rank + d, v);
+        for (int i = tid; i < heads * rot_dim; i += blockDim.x) {
+            int h = i / rot_dim, d = i - h * rot_dim;
+            ie_store(q_abs + ((size_t)n * heads + h) * krow + rank + d, turned(row + h * hq + dim, d, cs, rot_dims, interleaved));
+        }
     }
-    const float* dkv = row + heads * hq;
-    const float* g = dkv + krow;
-    for (int h = tid; h < heads; h += blockDim.x) gate[(size_t)n * heads + h] = 1.0f / (1.0f + expf(-g[h]));
-
-    if (slot_mapping == nullptr) return;  // a run that borrows another layer's cache writes none
+    if (in.gate_pre != nullptr) {
+        const float* g = in.gate_pre + (size_t)n * in.gate_ld;
+        for (int h = tid; h < heads; h += blockDim.x) gate[(size_t)n * heads + h] = 1.0f / (1.0f + expf(-g[h]));
+    }
+    if (in.cq != nullptr) {
+        const float* src = in.cq + (size_t)n * in.cq_ld;
+        float inv = rms_factor(src, in.q_rank, in.eps, red_cq);
+        for (int i = tid; i < in.q_rank; i += blockDim.x)
+            ie_store(cq_out + (size_t)n * in.q_rank + i, src[i] * inv * in.cq_norm_w[i]);
+    }
+    if (in.dkv == nullptr || slot_mapping == nullptr) return;  // a run that borrows another layer's cache writes none
     int slot = slot_mapping[n];
     if (slot < 0 || slot >= total_slots) {
         if (tid == 0) ie_report(err, IE_ERR_PAGE, slot, n);
         return;
     }
-    float ss = 0.f;
-    for (int i = tid; i < rank; i += blockDim.x) ss = fmaf(dkv[i], dkv[i], ss);
-    ss = warp_sum(ss);
-    if ((tid & 31) == 0) red[tid >> 5] = ss;
-    __syncthreads();
-    float inv = 1.0f / sqrtf((red[0] + red[1] + red[2] + red[3]) / (float)rank + eps);
+    const float* dkv = in.dkv + (size_t)n * in.dkv_ld;
+    float inv = rms_factor(dkv, rank, in.eps, red);
     T* dst = cache + (size_t)slot * krow;
-    for (int i = tid; i < rank; i += blockDim.x) ie_store(dst + i, dkv[i] * inv * norm_w[i]);
-    for (int d = tid; d < rot_dim; d += blockDim.x) {
-        const float* src = dkv + rank;
-        float v = src[d];
-        if (turn && d < rot_dims) {
-            int j = d >> 1;
-            float c = cs[j], s = cs[half + j];
-            v = (d & 1) ? fmaf(src[d], c, src[d - 1] * s) : fmaf(src[d], c, -src[d + 1] * s);
-        }
-        ie_store(dst + rank + d, v);
-    }
+    for (int i = tid; i < rank; i += blockDim.x) ie_store(dst + i, dkv[i] * inv * in.norm_w[i]);
+    for (int d = tid; d < rot_dim; d += blockDim.x) ie_store(dst + rank + d, turned(dkv + rank, d, cs, rot_dims, interleaved));
 }
 
 // out[n, h, o] = scale[n, h] * sum_k x[n, h, k] * W[h, o, k], k ascending per output.
@@ -147,6 +171,139 @@ __global__ void scale_head_rows_kernel(__nv_bfloat16* __restrict__ out, long lon
         *p = __float2bfloat16_rn(__bfloat162float(*p) * scale[(size_t)n * heads + h]);
     }
 }
+
+// The same products on the tensor cores (bfloat16 weights, K a multiple of 16): W's rows are the
+// instruction's 16 rows, tokens its columns.  XT float: x is the queries' 32-bit product (rounded to bfloat16
+// here), and the blocks of a head's first outputs also turn the rotated part that follows x in its row
+// (`rot`).  A block of four warps takes either 64 outputs, a warp each sixteen (SPLIT false), or sixteen
+// outputs with K cut among its warps, whose sums are added in order (SPLIT true: long K, few outputs).
+// grid: (output blocks, heads, blocks of 8 * NT tokens).
+struct RotatedPart {
+    const int* positions;
+    const float* table;
+    int rot_dims, table_rows, interleaved, rot_dim, at;  // the part starts `at` entries behind x; 0 entries: none
+    int dst_at;                                           // ... and goes so many entries behind out
+    int* err;
+};
+
+__device__ __forceinline__ void mma_m16n8k16(float* c, const unsigned* a, unsigned b0, unsigned b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+
+template <typename XT, int NT, bool SPLIT>
+__global__ void __launch_bounds__(128)
+headwise_mma_kernel(const XT* __restrict__ x, long long x_ld, long long x_hs, const __nv_bfloat16* __restrict__ w,
+                    __nv_bfloat16* __restrict__ out, long long o_ld, long long o_hs, const float* __restrict__ scale,
+                    RotatedPart rot, int N, int heads, int O, int K) {
+    extern __shared__ __align__(16) unsigned char raw[];
+    __nv_bfloat16* xs = reinterpret_cast<__nv_bfloat16*>(raw);  // [8 * NT][K + 8]
+    float* sums = reinterpret_cast<float*>(xs + 8 * NT * (K + 8));  // SPLIT: [4][16][8 * NT]
+    ie_pdl_trigger();
+    const int h = blockIdx.y, n0 = blockIdx.z * 8 * NT, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int g = lane >> 2, t4 = lane & 3, ld = K + 8;
+    const int o0 = SPLIT ? blockIdx.x * 16 : (blockIdx.x * 4 + warp) * 16;
+    const int steps = K / 16, k_begin = SPLIT ? warp * steps / 4 : 0, k_end = SPLIT ? (warp + 1) * steps / 4 : steps;
+    ie_pdl_wait();
+    const int cnt = min(8 * NT, N - n0);
+    for (int i = tid; i < 8 * NT * (K / 4); i += 128) {
+        int r = i / (K / 4), c = (i - r * (K / 4)) * 4;
+        uint2 v = make_uint2(0u, 0u);
+        if (r < cnt) {
+            const XT* p = x + (size_t)(n0 + r) * x_ld + (size_t)h * x_hs + c;
+            __nv_bfloat162 lo = __floats2bfloat162_rn(ie_load(p), ie_load(p + 1)), hi = __floats2bfloat162_rn(ie_load(p + 2), ie_load(p + 3));
+            v = make_uint2(*reinterpret_cast<unsigned*>(&lo), *reinterpret_cast<unsigned*>(&hi));
+        }
+        *reinterpret_cast<uint2*>(xs + r * ld + c) = v;
+    }
+    if (rot.rot_dim > 0 && blockIdx.x == 0) {
+        for (int i = tid; i < cnt * rot.rot_dim; i += 128) {
+            int r = i / rot.rot_dim, d = i - r * rot.rot_dim, pos = rot.positions[n0 + r];
+            bool turn = rot.table != nullptr && rot.rot_dims > 0;
+            if (turn && (pos < 0 || pos >= rot.table_rows)) {
+                if (d == 0) ie_report(rot.err, IE_ERR_POSITION, pos, n0 + r);
+                turn = false;
+            }
+            const XT* p = x + (size_t)(n0 + r) * x_ld + (size_t)h * x_hs + rot.at;
+            float v = 0.f;
+            if constexpr (sizeof(XT) == 4)
+                v = turned(p, d, turn ? rot.table + (size_t)pos * rot.rot_dims : nullptr, rot.rot_dims, rot.interleaved);
+            out[(size_t)(n0 + r) * o_ld + (size_t)h * o_hs + rot.dst_at + d] = __float2bfloat16_rn(v);
+        }
+    }
+    __syncthreads();
+    float c[NT][4];
+#pragma unroll
+    for (int t = 0; t < NT; ++t) c[t][0] = c[t][1] = c[t][2] = c[t][3] = 0.f;
+    if (o0 < O) {
+        // a thread's four consecutive entries of a row are the instruction's columns 2 t4, 2 t4 + 1 and 2 t4 + 8,
+        // 2 t4 + 9: the same renaming of k for both operands
+        const bool in_a = o0 + g < O, in_b = o0 + g + 8 < O;
+        const __nv_bfloat16* wa = w + ((size_t)h * O + (in_a ? o0 + g : 0)) * K + t4 * 4;
+        const __nv_bfloat16* wb = w + ((size_t)h * O + (in_b ? o0 + g + 8 : 0)) * K + t4 * 4;
+#pragma unroll 8
+        for (int kk = k_begin; kk < k_end; ++kk) {
+            uint2 ra = *reinterpret_cast<const uint2*>(wa + kk * 16), rb = *reinterpret_cast<const uint2*>(wb + kk * 16);
+            unsigned a[4] = {ra.x, rb.x, ra.y, rb.y};
+#pragma unroll
+            for (int t = 0; t < NT; ++t) {
+                uint2 b = *reinterpret_cast<const uint2*>(xs + (t * 8 + g) * ld + kk * 16 + t4 * 4);
+                mma_m16n8k16(c[t], a, b.x, b.y);
+            }
+        }
+    }
+    if constexpr (SPLIT) {
+#pragma unroll
+        for (int t = 0; t < NT; ++t) {
+            float* dst = sums + (warp * 16 + g) * 8 * NT + t * 8 + t4 * 2;
+            dst[0] = c[t][0]; dst[1] = c[t][1];
+            dst[64 * NT] = c[t][2]; dst[64 * NT + 1] = c[t][3];
+        }
+        __syncthreads();
+        for (int i = tid; i < 16 * 8 * NT; i += 128) {
+            int o = i % 16, r = i / 16, at = o * 8 * NT + r;
+            if (r >= cnt || o0 + o >= O) continue;
+            float v = ((sums[at] + sums[128 * NT + at]) + sums[256 * NT + at]) + sums[384 * NT + at];
+            if (scale) v *= scale[(size_t)(n0 + r) * heads + h];
+            out[(size_t)(n0 + r) * o_ld + (size_t)h * o_hs + o0 + o] = __float2bfloat16_rn(v);
+        }
+    } else {
+#pragma unroll
+        for (int t = 0; t < NT; ++t)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                int o = o0 + g + (e >> 1) * 8, r = t * 8 + t4 * 2 + (e & 1);
+                if (o >= O || r >= cnt) continue;
+                float v = c[t][e];
+                if (scale) v *= scale[(size_t)(n0 + r) * heads + h];
+                out[(size_t)(n0 + r) * o_ld + (size_t)h * o_hs + o] = __float2bfloat16_rn(v);
+            }
+    }
+}
+
+template <typename XT, int NT, bool SPLIT>
+int launch_headwise_mma(const void* x, long long x_ld, long long x_hs, const void* w, void* out, long long o_ld,
+                        long long o_hs, const float* scale, RotatedPart rot, int N, int heads, int O, int K, cudaStream_t s) {
+    size_t smem = (size_t)8 * NT * (K + 8) * 2 + (SPLIT ? (size_t)4 * 16 * 8 * NT * 4 : 0);
+    static IePerDevice allowed;
+    cudaError_t e = ie_allow_smem(allowed, headwise_mma_kernel<XT, NT, SPLIT>, 96 * 1024);
+    if (e != cudaSuccess) return (int)e;
+    dim3 grid(SPLIT ? (O + 15) / 16 : (O + 63) / 64, heads, (N + 8 * NT - 1) / (8 * NT));
+    return ie_launch(headwise_mma_kernel<XT, NT, SPLIT>, grid, dim3(128), smem, s, (const XT*)x, x_ld, x_hs,
+                     (const __nv_bfloat16*)w, (__nv_bfloat16*)out, o_ld, o_hs, scale, rot, N, heads, O, K);
+}
+
+template <typename XT>
+int pick_headwise_mma(const void* x, long long x_ld, long long x_hs, const void* w, void* out, long long o_ld,
+                      long long o_hs, const float* scale, RotatedPart rot, int N, int heads, int O, int K, cudaStream_t s) {
+#define IE_HM_ARGS x, x_ld, x_hs, w, out, o_ld, o_hs, scale, rot, N, heads, O, K, s
+    // (the cut must not change with the number of tokens: a token's sums depend on the sizes alone)
+    bool split = K >= 256;
+    if (N <= 8) return split ? launch_headwise_mma<XT, 1, true>(IE_HM_ARGS) : launch_headwise_mma<XT, 1, false>(IE_HM_ARGS);
+    return split ? launch_headwise_mma<XT, 4, true>(IE_HM_ARGS) : launch_headwise_mma<XT, 4, false>(IE_HM_ARGS);
+#undef IE_HM_ARGS
+}
 }  // namespace
 
 IE_API int ie_scale_head_rows(void* out, long long o_ld, long long o_hs, const float* scale, int N, int heads, int o,
@@ -156,19 +313,42 @@ IE_API int ie_scale_head_rows(void* out, long long o_ld, long long o_hs, const f
                      scale, heads, o);
 }
 
-IE_API int ie_latent_prep(const float* proj, int ld, const int* positions, const float* table, int rot_dims,
-                          int table_rows, const float* norm_w, float eps, void* q_plain, void* q_abs,
-                          float* gate, void* cache, int dtype, const int* slot_mapping, int num_tokens,
-                          int heads, int dim, int rot_dim, int rank, int total_slots, int* err, void* stream) {
+IE_API int ie_latent_prep(const float* q, int q_ld, const float* gate_pre, int gate_ld, const float* dkv, int dkv_ld,
+                          const float* cq, int cq_ld, int q_rank, const float* norm_w, const float* cq_norm_w, float eps,
+                          const int* positions, const float* table, int rot_dims, int table_rows, int interleaved,
+                          void* q_plain, void* q_abs, float* gate, void* cq_out, void* cache, int dtype,
+                          const int* slot_mapping, int num_tokens, int heads, int dim, int rot_dim, int rank,
+                          int total_slots, int* err, void* stream) {
     if (num_tokens <= 0) return 0;
+    if (rot_dims < 0 || rot_dims % 2 || rot_dims > rot_dim) return (int)cudaErrorInvalidValue;
     cudaStream_t s = (cudaStream_t)stream;
+    LatentIn in{q, q_ld, gate_pre, gate_ld, dkv, dkv_ld, cq, cq_ld, q_rank, norm_w, cq_norm_w, eps};
     if (dtype == IE_BF16)
-        return ie_launch(latent_prep_kernel<__nv_bfloat16>, dim3(num_tokens), dim3(128), 0, s, proj, ld, positions,
-                         table, rot_dims, table_rows, norm_w, eps, (__nv_bfloat16*)q_plain, (__nv_bfloat16*)q_abs,
-                         gate, (__nv_bfloat16*)cache, slot_mapping, heads, dim, rot_dim, rank, total_slots, err);
-    return ie_launch(latent_prep_kernel<float>, dim3(num_tokens), dim3(128), 0, s, proj, ld, positions, table,
-                     rot_dims, table_rows, norm_w, eps, (float*)q_plain, (float*)q_abs, gate, (float*)cache,
+        return ie_launch(latent_prep_kernel<__nv_bfloat16>, dim3(num_tokens), dim3(128), 0, s, in, positions, table,
+                         rot_dims, table_rows, interleaved, (__nv_bfloat16*)q_plain, (__nv_bfloat16*)q_abs, gate,
+                         (__nv_bfloat16*)cq_out, (__nv_bfloat16*)cache, slot_mapping, heads, dim, rot_dim, rank,
+                         total_slots, err);
+    return ie_launch(latent_prep_kernel<float>, dim3(num_tokens), dim3(128), 0, s, in, positions, table, rot_dims,
+                     table_rows, interleaved, (float*)q_plain, (float*)q_abs, gate, (float*)cq_out, (float*)cache,
                      slot_mapping, heads, dim, rot_dim, rank, total_slots, err);
+}
+
+// Whether headwise_mma takes this inner size (else headwise_linear runs).
+IE_API int ie_headwise_mma_ok(int K) { return K % 16 == 0 && K >= 16 && K <= 1024; }
+
+// x: bfloat16, or 32-bit (x_f32) with a rotated part of rot_dim entries that starts `rot_at` entries behind x.
+IE_API int ie_headwise_mma(const void* x, int x_f32, long long x_ld, long long x_hs, const void* w, void* out,
+                           long long o_ld, long long o_hs, const float* scale, int N, int heads, int O, int K,
+                           const int* positions, const float* table, int rot_dims, int table_rows, int interleaved,
+                           int rot_dim, int rot_at, int rot_dst, int* err, void* stream) {
+    if (N <= 0 || heads <= 0 || O <= 0) return 0;
+    if (!ie_headwise_mma_ok(K) || (rot_dim > 0 && (!x_f32 || positions == nullptr)) || rot_dims < 0 || rot_dims % 2 ||
+        rot_dims > rot_dim || reinterpret_cast<uintptr_t>(w) % 8)
+        return (int)cudaErrorInvalidValue;
+    RotatedPart rot{positions, table, rot_dims, table_rows, interleaved, rot_dim, rot_at, rot_dst, err};
+    cudaStream_t s = (cudaStream_t)stream;
+    if (x_f32) return pick_headwise_mma<float>(x, x_ld, x_hs, w, out, o_ld, o_hs, scale, rot, N, heads, O, K, s);
+    return pick_headwise_mma<__nv_bfloat16>(x, x_ld, x_hs, w, out, o_ld, o_hs, scale, rot, N, heads, O, K, s);
 }
 
 IE_API int ie_headwise_linear(const void* x, long long x_ld, long long x_hs, const void* w, void* out,

@@ -10,7 +10,9 @@
 //            S = Q K^T over DK by mma.sync.m16n8k16, Q and the key tile in shared memory (key tiles
 //            arrive by cp.async, two buffers);
 //   softmax  a few threads per row: mask (a row sees positions up to its own), running maximum
-//            and sum in 32-bit, weights rounded to bfloat16 into shared memory;
+//            and sum in 32-bit, a weight as two bfloat16 terms (its rounded value and the remainder: 16 bits
+//            of its mantissa) into shared memory; a sink (`sinks`, a number per head) is one more term
+//            of the sum that has no key and no value: a row starts from it, or the merge adds it;
 //   values   warp w owns every eighth 8-column slice of the DV output columns: O = O * alpha + P V,
 //            V's fragments straight from the key tile with ldmatrix.trans.
 // A context may be cut into `splits` ranges of key tiles (few requests, long contexts): the blocks of
@@ -41,7 +43,7 @@ struct LmSmem {
     __nv_bfloat16* q;   // [rows][ld]
     __nv_bfloat16* k;   // [2][keys][ld]
     float* s;           // [rows][keys + 4]
-    __nv_bfloat16* p;   // [rows][keys + 8]
+    __nv_bfloat16* p;   // [2][rows][keys + 8]: the weights rounded, and what the rounding left
     float* alpha;       // [rows]
     float* m;           // [rows]
     float* l;           // [rows]
@@ -50,7 +52,7 @@ struct LmSmem {
 inline __host__ __device__ int lm_ld(int dk) { return ((dk + 15) / 16) * 16 + 8; }
 inline size_t lm_smem_bytes(int dk, int rows, int keys) {
     size_t ld = lm_ld(dk);
-    return (rows + 2 * keys) * ld * 2 + rows * (keys + 4) * 4 + rows * (keys + 8) * 2 + 3 * rows * 4;
+    return (rows + 2 * keys) * ld * 2 + rows * (keys + 4) * 4 + 2 * rows * (keys + 8) * 2 + 3 * rows * 4;
 }
 
 // grid: (row tiles of a request, requests, splits).  MT 16-row tiles and KEYS keys per step, LM_WARPS warps.
@@ -60,7 +62,7 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
                             const int* __restrict__ block_tables, int table_width, const int* __restrict__ cu_q,
                             const int* __restrict__ ctx_lens, __nv_bfloat16* __restrict__ out,
                             float* __restrict__ scratch, int heads, int dk, int dv, int page_size,
-                            int total_pages, float scale, int splits, int* err) {
+                            int total_pages, float scale, const float* __restrict__ sinks, int splits, int* err) {
     extern __shared__ __align__(16) unsigned char raw[];
     constexpr int LM_ROWS = 16 * MT, LM_KEYS = KEYS, LM_THREADS = LM_WARPS * 32;
     constexpr int LM_MAX_NT = LM_MAX_DV / 8 / LM_WARPS;  // 8-column slices of the output per warp
@@ -92,7 +94,7 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
     sm.k = sm.q + LM_ROWS * ld;
     sm.s = reinterpret_cast<float*>(sm.k + 2 * LM_KEYS * ld);
     sm.p = reinterpret_cast<__nv_bfloat16*>(sm.s + LM_ROWS * (LM_KEYS + 4));
-    sm.alpha = reinterpret_cast<float*>(sm.p + LM_ROWS * (LM_KEYS + 8));
+    sm.alpha = reinterpret_cast<float*>(sm.p + 2 * LM_ROWS * (LM_KEYS + 8));
     sm.m = sm.alpha + LM_ROWS;
     sm.l = sm.m + LM_ROWS;
 
@@ -139,7 +141,11 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
         }
         *reinterpret_cast<uint4*>(sm.q + r * ld + c * 8) = v;
     }
-    if (tid < LM_ROWS) { sm.m[tid] = -INFINITY; sm.l[tid] = 0.f; }
+    if (tid < LM_ROWS) {  // (cut contexts: the merge adds the sink's term)
+        bool with_sink = sinks != nullptr && splits == 1 && tid < rows_here;
+        sm.m[tid] = with_sink ? sinks[(row0 + tid) % heads] : -INFINITY;
+        sm.l[tid] = with_sink ? 1.f : 0.f;
+    }
 
     float acc[MT][LM_MAX_NT][4];
 #pragma unroll
@@ -222,17 +228,21 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
             float m_new = fmaxf(m_old, mx);
             float sum = 0.f;
             __align__(8) __nv_bfloat16 pb[KPT];
+            __align__(8) __nv_bfloat16 pr[KPT];
 #pragma unroll
             for (int i = 0; i < KPT; ++i) {
                 float pv = (v[i] == -INFINITY) ? 0.f : expf(v[i] - m_new);
                 pb[i] = __float2bfloat16_rn(pv);
+                pr[i] = __float2bfloat16_rn(pv - __bfloat162float(pb[i]));
                 sum += pv;
             }
 #pragma unroll
             for (int o = TPR / 2; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
 #pragma unroll
-            for (int i = 0; i < KPT; i += 4)
+            for (int i = 0; i < KPT; i += 4) {
                 *reinterpret_cast<uint2*>(sm.p + r * (LM_KEYS + 8) + j * KPT + i) = *reinterpret_cast<uint2*>(pb + i);
+                *reinterpret_cast<uint2*>(sm.p + (LM_ROWS + r) * (LM_KEYS + 8) + j * KPT + i) = *reinterpret_cast<uint2*>(pr + i);
+            }
             if (j == 0) {
                 float a = (m_old == -INFINITY) ? 0.f : expf(m_old - m_new);
                 if (m_new == -INFINITY) a = 1.f;
@@ -244,7 +254,7 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
         __syncthreads();
         // values
         {
-            unsigned pa[MT][LM_KEYS / 16][4];
+            unsigned pa[MT][LM_KEYS / 16][4], pl[MT][LM_KEYS / 16][4];
             float a0[MT], a1[MT];
             bool moved = false;
 #pragma unroll
@@ -258,6 +268,11 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
                     asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
                                  : "=r"(pa[mt][kk][0]), "=r"(pa[mt][kk][1]), "=r"(pa[mt][kk][2]), "=r"(pa[mt][kk][3])
                                  : "r"(pr + kk * 32));
+#pragma unroll
+                for (int kk = 0; kk < LM_KEYS / 16; ++kk)
+                    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+                                 : "=r"(pl[mt][kk][0]), "=r"(pl[mt][kk][1]), "=r"(pl[mt][kk][2]), "=r"(pl[mt][kk][3])
+                                 : "r"(pr + LM_ROWS * (LM_KEYS + 8) * 2 + kk * 32));
             }
             moved = __any_sync(0xffffffffu, moved);  // (mostly false once the rows' maxima have settled)
 #pragma unroll
@@ -278,7 +293,10 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
 #pragma unroll
                 for (int kk = 0; kk < LM_KEYS / 16; ++kk)
 #pragma unroll
-                    for (int mt = 0; mt < MT; ++mt) mma_bf16(acc[mt][i], pa[mt][kk], b[kk]);
+                    for (int mt = 0; mt < MT; ++mt) {
+                        mma_bf16(acc[mt][i], pa[mt][kk], b[kk]);
+                        mma_bf16(acc[mt][i], pl[mt][kk], b[kk]);
+                    }
             }
         }
     }
@@ -318,14 +336,16 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
 
 // One block per (token, head) row: the ranges' parts added in order.
 __global__ void __launch_bounds__(128)
-latent_attention_merge_kernel(const float* __restrict__ scratch, __nv_bfloat16* __restrict__ out, int dv, int splits) {
+latent_attention_merge_kernel(const float* __restrict__ scratch, __nv_bfloat16* __restrict__ out, int dv, int splits,
+                              const float* __restrict__ sinks, int heads) {
     ie_pdl_trigger();
     ie_pdl_wait();
     size_t row = blockIdx.x;
     const float* base = scratch + row * splits * (dv + 2);
-    float m = -INFINITY;
+    float sink = sinks != nullptr ? sinks[row % heads] : -INFINITY;
+    float m = sink;
     for (int s = 0; s < splits; ++s) m = fmaxf(m, base[(size_t)s * (dv + 2)]);
-    float l = 0.f;
+    float l = sinks != nullptr ? expf(sink - m) : 0.f;
     for (int s = 0; s < splits; ++s) {
         float ms = base[(size_t)s * (dv + 2)];
         if (ms != -INFINITY) l += base[(size_t)s * (dv + 2) + 1] * expf(ms - m);
@@ -358,14 +378,14 @@ IE_API int ie_latent_attention_rows(int longest_rows) { return longest_rows >= 6
 IE_API int ie_latent_attention_mma(const void* q, const void* cache, const int* block_tables, int table_width,
                                    const int* cu_q, const int* ctx_lens, void* out, float* scratch, int num_tokens,
                                    int num_seqs, int max_tiles, int rows, int heads, int dk, int dv, int page_size,
-                                   int total_pages, float scale, int splits, int* err, void* stream) {
+                                   int total_pages, float scale, const float* sinks, int splits, int* err, void* stream) {
     if (num_seqs <= 0 || max_tiles <= 0) return 0;
     if (!ie_latent_attention_mma_ok(dk, dv) || splits < 1 || (splits > 1 && scratch == nullptr)) return (int)cudaErrorInvalidValue;
     if (rows != 16 && rows != 64) return (int)cudaErrorInvalidValue;
     cudaStream_t s = (cudaStream_t)stream;
     int rc;
 #define IE_LM_ARGS (const __nv_bfloat16*)q, (const __nv_bfloat16*)cache, block_tables, table_width, cu_q, ctx_lens, \
-                   (__nv_bfloat16*)out, scratch, heads, dk, dv, page_size, total_pages, scale, splits, err
+                   (__nv_bfloat16*)out, scratch, heads, dk, dv, page_size, total_pages, scale, sinks, splits, err
     if (rows == 64) {
         // (sixteen warps instead of eight take as long: 636 against 633 us on 2,048 tokens of 16 heads)
         cudaError_t e = ie_allow_smem(g_lm_smem64, latent_attention_mma_kernel<4, 32, 8>, 220 * 1024);
@@ -381,5 +401,5 @@ IE_API int ie_latent_attention_mma(const void* q, const void* cache, const int* 
 #undef IE_LM_ARGS
     if (rc != 0 || splits == 1) return rc;
     return ie_launch(latent_attention_merge_kernel, dim3(num_tokens * heads), dim3(128), 0, s, (const float*)scratch,
-                     (__nv_bfloat16*)out, dv, splits);
+                     (__nv_bfloat16*)out, dv, splits, sinks, heads);
 }

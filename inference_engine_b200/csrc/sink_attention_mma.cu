@@ -35,7 +35,7 @@
 // before the block's first query takes the table's last entry without looking.  These variants also
 // leave the mask out in tiles that every row of the block sees whole.
 // `gate_elements` 1: the gate is a number per head and value entry, out_gate[token * gate_ld + head * SK_DV
-// + c], instead of one per head.
+// + c], instead of one per head.  Rows of the output lie `out_ld` entries apart.
 #include "common.cuh"
 #include <math.h>
 
@@ -123,7 +123,7 @@ sink_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat
                           const float* __restrict__ out_gate, int gate_ld, float* __restrict__ partial,
                           int splits, int tiles_per_split, float softcap, int keep_first, int kept_splits,
                           int gate_elements, const float* __restrict__ log_r1, const float* __restrict__ log_r2,
-                          const float* __restrict__ bias_table, int bias_len, int* err) {
+                          const float* __restrict__ bias_table, int bias_len, int out_ld, int* err) {
     extern __shared__ __align__(16) unsigned char raw[];
     __nv_bfloat16* qs = reinterpret_cast<__nv_bfloat16*>(raw);  // [ROWS][LDK]
     __nv_bfloat16* ks = qs + ROWS * LDK;                        // [2][KEYS][LDK]
@@ -434,8 +434,8 @@ sink_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat
         if (pos_a >= 0) f_a *= 1.0f / (1.0f + expf(-out_gate[(size_t)(q0 + row0 + r_a) * gate_ld + head]));
         if (pos_b >= 0) f_b *= 1.0f / (1.0f + expf(-out_gate[(size_t)(q0 + row0 + r_b) * gate_ld + head]));
     }
-    __nv_bfloat16* out_a = out + ((size_t)(q0 + row0 + r_a) * heads + head) * DV;
-    __nv_bfloat16* out_b = out + ((size_t)(q0 + row0 + r_b) * heads + head) * DV;
+    __nv_bfloat16* out_a = out + (size_t)(q0 + row0 + r_a) * out_ld + (size_t)head * DV;
+    __nv_bfloat16* out_b = out + (size_t)(q0 + row0 + r_b) * out_ld + (size_t)head * DV;
 #pragma unroll
     for (int nt = 0; nt < DV / 8; ++nt) {
         int c = nt * 8 + t4 * 2;
@@ -463,7 +463,7 @@ __global__ void __launch_bounds__(128)
 sink_attention_merge_kernel(const float* __restrict__ partial, const int* __restrict__ cu_q, int num_seqs,
                             __nv_bfloat16* __restrict__ out, int heads, int splits,
                             const float* __restrict__ sinks, const float* __restrict__ out_gate, int gate_ld,
-                            int gate_elements) {
+                            int gate_elements, int out_ld) {
     ie_pdl_trigger();
     ie_pdl_wait();
     int token = blockIdx.x / heads, head = blockIdx.x - token * heads;
@@ -506,7 +506,7 @@ sink_attention_merge_kernel(const float* __restrict__ partial, const int* __rest
         float v = acc[i] * f;
         if (out_gate != nullptr && gate_elements)
             v *= sigmoid_of(out_gate[(size_t)token * gate_ld + (size_t)head * DV + c]);
-        out[((size_t)token * heads + head) * DV + c] = __float2bfloat16_rn(v);
+        out[(size_t)token * out_ld + (size_t)head * DV + c] = __float2bfloat16_rn(v);
     }
 }
 }  // namespace
@@ -523,12 +523,13 @@ IE_API int ie_sink_attention_mma(const void* q, const void* k_cache, const void*
                                  float scale, int window, const float* sinks, const float* out_gate, int gate_ld,
                                  float* partial, int splits, int tiles_per_split, int num_tokens, float softcap,
                                  int keep_first, int kept_splits, int gate_elements, const float* log_r1,
-                                 const float* log_r2, const float* bias_table, int bias_len, int* err,
+                                 const float* log_r2, const float* bias_table, int bias_len, int out_ld, int* err,
                                  void* stream) {
     if (num_seqs <= 0 || max_q_len <= 0) return 0;
     if (kv_heads <= 0 || heads % kv_heads != 0 || page_size < 1 || (page_size & (page_size - 1)) || window < 0)
         return (int)cudaErrorInvalidValue;
-    if (softcap < 0.f || keep_first < 0 || kept_splits < 0 || (window == 0 && keep_first > 0))
+    if (softcap < 0.f || keep_first < 0 || kept_splits < 0 || (window == 0 && keep_first > 0) || out_ld < heads * DV ||
+        out_ld % 2)
         return (int)cudaErrorInvalidValue;
     if ((BIAS == 1) != (log_r1 != nullptr && log_r2 != nullptr) || (BIAS == 2) != (bias_table != nullptr) ||
         (BIAS == 2 && bias_len < 1))
@@ -549,16 +550,16 @@ IE_API int ie_sink_attention_mma(const void* q, const void* k_cache, const void*
                            (const __nv_bfloat16*)v_cache, block_tables, table_width, cu_q, ctx_lens, (__nv_bfloat16*)out,
                            heads, kv_heads, page_size, total_pages, scale, window, sinks, out_gate, gate_ld, partial,
                            splits, tiles_per_split, softcap, keep_first, kept_splits, gate_elements, log_r1, log_r2,
-                           bias_table, bias_len, err);
+                           bias_table, bias_len, out_ld, err);
         if (rc != 0) return rc;
         return ie_launch(sink_attention_merge_kernel, dim3(num_tokens * heads), dim3(128), 0, (cudaStream_t)stream,
                          (const float*)partial, cu_q, num_seqs, (__nv_bfloat16*)out, heads, splits, sinks, out_gate,
-                         gate_ld, gate_elements);
+                         gate_ld, gate_elements, out_ld);
     }
     dim3 grid((max_q_len + ROWS - 1) / ROWS, heads, num_seqs);
     return ie_launch(sink_attention_mma_kernel<false>, grid, dim3(THREADS), smem, (cudaStream_t)stream,
                      (const __nv_bfloat16*)q, (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache, block_tables,
                      table_width, cu_q, ctx_lens, (__nv_bfloat16*)out, heads, kv_heads, page_size, total_pages, scale,
                      window, sinks, out_gate, gate_ld, (float*)nullptr, 1, 0, softcap, keep_first, 0,
-                     gate_elements, log_r1, log_r2, bias_table, bias_len, err);
+                     gate_elements, log_r1, log_r2, bias_table, bias_len, out_ld, err);
 }

@@ -8,7 +8,7 @@
 //  * sandwich_norm: y = sum of the parts of `delta` (+ the parts of `delta2`, the output of a second
 //    sublayer that read the same input) (+ bias) (+ the row of `extra`, a second stream of the rows'
 //    shape: the embedding's output that a looped model adds again); y <- rms(y) * post_w (if post_w);
-//    h += y; out = rms(h) * pre_w (if out).  One block per row; both sums of squares are added in
+//    h += y; out = rms(h) * pre_w, or h itself in the output's dtype without a pre_w (if out).  One block per row; both sums of squares are added in
 //    an order that depends on the row's width alone.
 //  * silu_mul_bias: out = silu(g + bg) * (u + bu) from rows that hold gates, then ups (32-bit, or the
 //    compute dtype); biases and activation in 32-bit.
@@ -176,6 +176,11 @@ sandwich_norm_kernel(float* __restrict__ h, const float* __restrict__ delta, int
         }
     }
     if (out == nullptr) return;
+    if (pre_w == nullptr) {  // (a thread's own entries: nothing to wait for)
+        for (int i = threadIdx.x * VEC; i < hidden; i += SN_THREADS * VEC)
+            store_pack<VEC>(out + (size_t)r * hidden + i, load_pack<VEC>(row_buf + i));
+        return;
+    }
     float inv2 = 1.0f / sqrtf(block_sum(ss, red) / (float)hidden + pre_eps);
     for (int i = threadIdx.x * VEC; i < hidden; i += SN_THREADS * VEC) {
         Pack<VEC> x = load_pack<VEC>(row_buf + i), w = load_pack<VEC>(pre_w + i);
@@ -377,7 +382,6 @@ IE_API int ie_sandwich_norm(float* h, const float* delta, int num_partials, long
     if (delta != nullptr && num_partials < 1) return (int)cudaErrorInvalidValue;
     if (delta == nullptr && (delta2 != nullptr || extra != nullptr)) return (int)cudaErrorInvalidValue;
     if (delta2 == nullptr) num_partials2 = 0;
-    if (out != nullptr && pre_w == nullptr) return (int)cudaErrorInvalidValue;
     size_t smem = (size_t)hidden * sizeof(float);
     if (smem > 200 * 1024) return (int)cudaErrorInvalidValue;
     cudaStream_t s = (cudaStream_t)stream;

@@ -184,6 +184,15 @@ def build_retention(dim: int, vdim: int) -> Path:
     return build_library(f"ie_b200_retention_d{d}_v{dv}", ["retention.cu"], [f"-DRT_D={d}", f"-DRT_DV={dv}"])
 
 
+def build_state_space(state: int, vdim: int) -> Path:
+    """The bfloat16 path's state-space kernels for one pair of state and value sizes, each rounded up to a
+    multiple of 16 (compiled on first use for the sizes the loaded model has)."""
+    if not 1 <= state <= 128 or not 1 <= vdim <= 128:
+        raise BuildError(f"the state-space kernels take state and value sizes up to 128, not {state} and {vdim}")
+    n, p = -(-state // 16) * 16, -(-vdim // 16) * 16
+    return build_library(f"ie_b200_statespace_n{n}_p{p}", ["state_space.cu"], [f"-DSS_N={n}", f"-DSS_P={p}"])
+
+
 # Kernels only some mixers and feed-forwards need, each a library of its own that is built the
 # first time a model with such a part runs: name -> sources.
 PART_LIBRARIES = {
@@ -192,7 +201,7 @@ PART_LIBRARIES = {
     "delta": ["delta_rule.cu"],  # the gated delta rule: convolutions, the recurrence, the read-out norm
     "routed": ["routed_experts.cu"],  # routing and the grouped products of the routed feed-forward
     # recurrent mixers with a decaying matrix state (gated-write linear attention, exponential-gate
-    # matrix memory): input convolution, gates, the recurrence, the read-out
+    # matrix memory, state-space duality): input convolutions, gates, the recurrence, the read-outs
     "recurrent": ["gated_recurrence.cu"],
     # attention with normalised queries and keys and sigmoid weights: the input stage
     "gated_attn": ["gated_attention.cu"],
@@ -216,7 +225,7 @@ def build_all(prune: bool = True) -> list[Path]:
         libs += list(pool.map(build_part_library, PART_LIBRARIES))
         libs += [build_sigmoid_attention(64, 64), build_sink_attention(64, 64),
                  build_sink_attention(64, 64, "log"), build_sink_attention(64, 64, "table"),
-                 build_retention(64, 64)]
+                 build_retention(64, 64), build_state_space(64, 64)]
     if prune:
         keep = {lib.name for lib in libs}
         for old in build_dir().glob("libie_b200_*.so"):

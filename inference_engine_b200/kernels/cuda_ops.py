@@ -18,7 +18,7 @@ import os
 from ctypes import c_float, c_int, c_void_p
 
 from .build import (ATTENTION_HEAD_DIMS, build_attention, build_core, build_part_library,
-                    build_retention, build_sigmoid_attention, build_sink_attention)
+                    build_retention, build_sigmoid_attention, build_sink_attention, build_state_space)
 
 _ERRORS = {
     1: "a token id outside the vocabulary",
@@ -138,6 +138,8 @@ class CudaOps:
         self._part_libs: dict[str, object] = {}
         self._sigattn_libs: dict[tuple[int, int], object] = {}
         self._retention_libs: dict[tuple[int, int], object] = {}
+        self._state_space_libs: dict[tuple[int, int], object] = {}
+        self.state_space_fused = os.environ.get("IE_B200_STATE_SPACE", "1") != "0"  # the state-space kernels of the bfloat16 path
         self.retention_fused = os.environ.get("IE_B200_RETENTION", "1") != "0"  # the retention kernels of the bfloat16 path
         self._sinkattn_libs: dict[tuple[int, int, str], object] = {}
         self.sink_mma = os.environ.get("IE_B200_SINK_MMA", "1") != "0"  # tensor-core sink attention
@@ -150,6 +152,7 @@ class CudaOps:
         self.sm_count = torch.cuda.get_device_properties(self.device).multi_processor_count
         self.attn_tc5 = os.environ.get("IE_B200_ATTN_TC5", "1") != "0"  # tcgen05 prefill attention
         self.latent_mma = os.environ.get("IE_B200_LATENT_MMA", "1") != "0"  # tensor-core latent attention
+        self.headwise_mma = os.environ.get("IE_B200_HEADWISE_MMA", "1") != "0"  # its per-head products of few rows
         self.prefill_key_splits = os.environ.get("IE_B200_PREFILL_KEY_SPLITS", "1") != "0"
         # up to this many query tiles x heads per SM a block takes two tiles of a request (a late and an early one)
         self.prefill_paired_max = float(os.environ.get("IE_B200_PREFILL_PAIRED_MAX", 4))
@@ -231,7 +234,7 @@ class CudaOps:
             "ie_gemm_tma_bf16": [P, P, P, I, I, I, I, I, I, P, P],
             "ie_gemm_tc5_bf16": [P, P, P, I, I, I, I, I, I, P, P],
             "ie_gemm_tc5_ok": [I, I, I],
-            "ie_paged_attention_generic": [P, P, P, I, P, I, P, P, P, I, I, I, I, I, I, I, I, F, I, I, P, P, P, I, F, I, I, P, P, P, I, P, P],
+            "ie_paged_attention_generic": [P, P, P, I, P, I, P, P, P, I, I, I, I, I, I, I, I, F, I, I, P, P, P, I, F, I, I, P, P, P, I, I, P, P],
             "ie_sample": [P, I, I, P, P, P, P, P, P, I, P, P, P, P, P],
             "ie_bigram_embedding": [P, P, I, P, P, P, P, P, P, L, I, P, I, I, I, I, L, L, P, P],
             "ie_sandwich_norm": [P, P, I, L, P, I, L, P, P, P, F, P, F, P, I, P, I, I, P],
@@ -750,7 +753,7 @@ class CudaOps:
         return best if cost(best) <= 0.75 * cost(1) else 1
 
     def paged_attention(self, q, k_cache, v_cache, block_tables, ctx, nh, nkv, hd, page_size,
-                        scale, window, out, ragged: bool | None = None, value_dim: int | None = None) -> None:
+                        scale, window, out, ragged: bool | None = None, value_dim: int | None = None, sinks=None) -> None:
         """Attention of every token of the step over its request's cached keys and values.
         bfloat16 with a head size the tensor-core kernels take and at most 16 query heads per
         key/value head: requests with few rows go to the split decode kernel, longer portions
@@ -758,10 +761,12 @@ class CudaOps:
         kernel, whose order of operations does not depend on the batch."""
         if nkv < 1 or nh % nkv:
             raise KernelError(f"{nh} query heads cannot share {nkv} key/value heads")
-        if value_dim is not None and value_dim != hd:
+        if sinks is not None and value_dim is None:
+            raise KernelError("sinks go with value rows of a given size here; sink_attention takes the others")
+        if value_dim is not None and (value_dim != hd or sinks is not None):
             # value rows shorter than key rows (a shared latent row whose first entries are the value)
             return self.latent_paged_attention(q, k_cache, v_cache, block_tables, ctx, nh, nkv, hd, value_dim,
-                                               page_size, scale, window, out)
+                                               page_size, scale, window, out, sinks=sinks)
         if hd % 8 or hd > 256:
             raise KernelError(f"head_dim {hd} is not supported: it must be a multiple of 8, at most 256")
         groups = nh // nkv
@@ -904,14 +909,17 @@ class CudaOps:
             q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), _dtype_code(q),
             block_tables.data_ptr(), block_tables.shape[1], ctx.seq_of_token.data_ptr(),
             ctx.positions.data_ptr(), out.data_ptr(), ctx.num_tokens, nh, nkv, hd, hd, hd, page_size,
-            k_cache.shape[0], scale, window, 0, None, None, None, 0, 0.0, 0, *self._NO_BIAS, self._err_ptr,
+            k_cache.shape[0], scale, window, 0, None, None, None, 0, 0.0, 0, *self._NO_BIAS, nh * hd, self._err_ptr,
             self._stream()), "paged_attention")
 
     @_kind("attention.latent")
     def latent_paged_attention(self, q, k_cache, v_cache, block_tables, ctx, nh, nkv, hd, value_dim,
-                               page_size, scale, window, out) -> None:
+                               page_size, scale, window, out, sinks=None) -> None:
         """Attention whose value rows are the first ``value_dim`` entries of ``v_cache``'s rows
-        (``v_cache`` may be the key cache itself); ``out`` is ``[N, nh * value_dim]``."""
+        (``v_cache`` may be the key cache itself); ``out`` is ``[N, nh * value_dim]``.  ``sinks`` (32-bit, one per head):
+        the softmax's denominator holds one more term ``exp(sinks[head])`` without key or value."""
+        if sinks is not None and (sinks.dtype != self.torch.float32 or sinks.numel() != nh):
+            raise KernelError("latent_paged_attention: the sinks are one 32-bit number per head")
         if not 0 < value_dim <= 512:
             raise KernelError(f"value rows of {value_dim} entries are not supported (1 to 512)")
         if (q.dtype == self.torch.bfloat16 and nkv == 1 and window == 0 and v_cache is k_cache
@@ -933,25 +941,28 @@ class CudaOps:
             self._check(lib.ie_latent_attention_mma(
                 q.data_ptr(), k_cache.data_ptr(), block_tables.data_ptr(), block_tables.shape[1], ctx.cu_q.data_ptr(),
                 ctx.ctx_lens.data_ptr(), out.data_ptr(), self._ptr(scratch), ctx.num_tokens, ctx.num_seqs, max_tiles,
-                rows, nh, hd, value_dim, page_size, k_cache.shape[0], scale, splits, self._err_ptr, self._stream()),
+                rows, nh, hd, value_dim, page_size, k_cache.shape[0], scale, self._ptr(sinks), splits, self._err_ptr,
+                self._stream()),
                 "latent_attention_mma")
             return
         self._check(self._paged_attention_generic(
             q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), _dtype_code(q),
             block_tables.data_ptr(), block_tables.shape[1], ctx.seq_of_token.data_ptr(),
             ctx.positions.data_ptr(), out.data_ptr(), ctx.num_tokens, nh, nkv, hd, value_dim,
-            v_cache.shape[-1], page_size, k_cache.shape[0], scale, window, 0, None, None, None, 0, 0.0, 0,
-            *self._NO_BIAS, self._err_ptr, self._stream()), "paged_attention_latent")
+            v_cache.shape[-1], page_size, k_cache.shape[0], scale, window, 0, None, self._ptr(sinks), None, 0, 0.0, 0,
+            *self._NO_BIAS, nh * value_dim, self._err_ptr, self._stream()), "paged_attention_latent")
 
     # --- kernels of single mixers and feed-forwards (libraries built on first use) -------------
 
     _PART_SIGNATURES = {
         "latent": {
-            "ie_latent_prep": "P I P P I I P F P P P P I P I I I I I I P P",
+            "ie_latent_prep": "P I P I P I P I I P P F P P I I I P P P P P I P I I I I I I P P",
             "ie_headwise_linear": "P L L P P L L P I I I I I P",
             "ie_scale_head_rows": "P L L P I I I P",
+            "ie_headwise_mma_ok": "I",
+            "ie_headwise_mma": "P I L L P P L L P I I I I P P I I I I I I P P",
             "ie_latent_attention_mma_ok": "I I",
-            "ie_latent_attention_mma": "P P P I P P P P I I I I I I I I I F I P P",
+            "ie_latent_attention_mma": "P P P I P P P P I I I I I I I I I F P I P P",
             "ie_latent_attention_rows": "I",
         },
         "delta": {
@@ -970,13 +981,16 @@ class CudaOps:
             "ie_short_conv_residual": "P I P P L P P P P I I I I I P P",
             "ie_hgrn2_gates": "P I P P P I I P",
             "ie_mlstm_gates": "P P I P P F P L L P P P I I I P",
-            "ie_gated_recurrence": "P I P I P I P I P I P L P P P I I I I I F I P",
+            "ie_gated_recurrence": "P I P I P I P I P I P L P P P I I I I I I F I P",
+            "ie_conv_silu": "P I P P P L L P P P P I I I I I I P P P P I P P",
+            "ie_gated_group_norm": "P P I P P I P F P I I I I I I P I P L L P P P I I I P",
             "ie_rotate_heads": "P I P P I I I I I P P",
             "ie_recurrence_readout": "P I P P I F P I I P I L I I P",
             "ie_lowrank_decay": "P I P P F P I I I P",
         },
         "gated_attn": {
-            "ie_qk_norm_rope_write": "P I P P I I P I I I P P F I P F I P P P I P I I I I I I I P P",
+            "ie_qk_norm_rope_write": "P I P P I I P I I I P P F I P F I F P P P I P I I I I I I I P P",
+            "ie_qk_wide_norm_rope_write": "P I P P I I P I P P F F P P P I P I I I I I I I P P",
         },
         "streams": {
             "ie_stream_mix_norm": "P I P I L P P P P P P F P I P I I P",
@@ -999,25 +1013,63 @@ class CudaOps:
         return lib
 
     @_kind("latent.prep")
-    def latent_prep(self, proj, positions, table, rot_dims, norm_w, eps, q_plain, q_abs, gate, cache,
-                    slot_mapping, heads, dim, rot_dim, rank, page_size) -> None:
-        """The latent attention's input stage (see ``csrc/latent_attention.cu``).  ``proj``: the fused
-        projection's 32-bit output ``[N, heads * (dim + rot_dim) + rank + rot_dim + heads]``;
-        ``cache``: ``[pages, 1, page_size, rank + rot_dim]``."""
+    def latent_prep(self, positions, table, rot_dims, *, heads, dim, rot_dim, rank, page_size, eps=0.0,
+                    interleaved: bool = True, q=None, q_plain=None, q_abs=None, gate_pre=None, gate=None, dkv=None,
+                    norm_w=None, cache=None, slot_mapping=None, cq=None, cq_norm_w=None, cq_out=None) -> None:
+        """The latent attention's input stage (see ``csrc/latent_attention.cu``), as much of it as is asked for, from
+        32-bit views ``[N, columns]`` of products of the mixer's input.  ``q`` (``heads * (dim + rot_dim)`` columns):
+        unrotated parts to ``q_plain``, rotated ones behind the latent parts of ``q_abs``; ``gate_pre`` (``heads``):
+        sigmoids to ``gate``; ``dkv`` (``rank + rot_dim``): the row of ``cache`` (``[pages, 1, page_size, rank +
+        rot_dim]``), unless ``slot_mapping`` is None; ``cq``: the queries' own latent, normalised, to ``cq_out``."""
         if table is not None and table.shape[2] * 2 != rot_dims:
             raise KernelError("rotary table does not match the rotated dims")
-        if proj.dtype != self.torch.float32 or proj.dim() != 2 or not proj.is_contiguous():
-            raise KernelError("latent_prep reads a contiguous 32-bit projection")
-        if proj.shape[1] != heads * (dim + rot_dim) + rank + rot_dim + heads or cache.shape[-1] != rank + rot_dim:
-            raise KernelError("latent_prep: the projection or the cache rows do not fit the sizes")
-        total_slots = cache.shape[0] * page_size
+        n = positions.shape[0]
+        for t, columns in ((q, heads * (dim + rot_dim)), (gate_pre, heads), (dkv, rank + rot_dim),
+                           (cq, None if cq_out is None else cq_out.shape[1])):
+            if t is not None and (t.dtype != self.torch.float32 or t.stride(1) != 1 or tuple(t.shape) != (n, columns)):
+                raise KernelError("latent_prep reads 32-bit columns of the sizes' widths")
+        if dkv is not None and cache.shape[-1] != rank + rot_dim:
+            raise KernelError("latent_prep: the cache rows do not fit the sizes")
+        out = next(t for t in (cq_out, q_abs, cache) if t is not None)
+        ld = lambda t: 0 if t is None else t.stride(0)  # noqa: E731
         self._check(self._part_lib("latent").ie_latent_prep(
-            proj.data_ptr(), proj.shape[1], positions.data_ptr(), self._ptr(table), rot_dims,
-            0 if table is None else table.shape[0], norm_w.data_ptr(), eps, q_plain.data_ptr(), q_abs.data_ptr(),
-            gate.data_ptr(), cache.data_ptr(), _dtype_code(q_abs), self._ptr(slot_mapping), proj.shape[0],
-            heads, dim, rot_dim, rank, total_slots, self._err_ptr, self._stream()), "latent_prep")
+            self._ptr(q), ld(q), self._ptr(gate_pre), ld(gate_pre), self._ptr(dkv), ld(dkv), self._ptr(cq), ld(cq),
+            0 if cq is None else cq.shape[1], self._ptr(norm_w), self._ptr(cq_norm_w), eps, positions.data_ptr(),
+            self._ptr(table), rot_dims, 0 if table is None else table.shape[0], 1 if interleaved else 0,
+            self._ptr(q_plain), self._ptr(q_abs), self._ptr(gate), self._ptr(cq_out), self._ptr(cache), _dtype_code(out),
+            self._ptr(slot_mapping), n, heads, dim, rot_dim, rank, 0 if cache is None else cache.shape[0] * page_size,
+            self._err_ptr, self._stream()), "latent_prep")
 
     HEADWISE_LIBRARY_ROWS = 128  # from this many rows on the per-head products go to the library (bfloat16)
+
+    def latent_queries(self, q, w, q_abs, positions, table, rot_dims, *, heads, dim, rot_dim, rank, page_size,
+                       interleaved: bool = True, ws) -> None:
+        """From the queries' 32-bit product ``q`` (``[N, heads * (dim + rot_dim)]``) the rows the attention reads,
+        ``q_abs`` ``[N, heads * (rank + rot_dim)]``: per head ``w[head] @ (unrotated part)`` (``w``: ``[heads, rank,
+        dim]``), then the rotated part turned by its position.  bfloat16 steps of few tokens: one launch."""
+        n = q.shape[0]
+        rows = q_abs.view(n, heads, rank + rot_dim)
+        if (q_abs.dtype == self.torch.bfloat16 and 0 < n < self.HEADWISE_LIBRARY_ROWS and self.headwise_mma
+                and self._part_lib("latent").ie_headwise_mma_ok(dim)):
+            return self._latent_queries_mma(q, w, rows, positions, table, rot_dims, dim, rot_dim, rank, interleaved)
+        plain = ws.buffer("latent.q_plain", n, heads * dim, q_abs.dtype)
+        self.latent_prep(positions, table, rot_dims, heads=heads, dim=dim, rot_dim=rot_dim, rank=rank,
+                         page_size=page_size, interleaved=interleaved, q=q, q_plain=plain, q_abs=q_abs)
+        self.headwise_linear(plain.view(n, heads, dim), w, rows[:, :, :rank])
+
+    @_kind("latent.headwise")
+    def _latent_queries_mma(self, q, w, rows, positions, table, rot_dims, dim, rot_dim, rank, interleaved) -> None:
+        n, heads, _ = rows.shape
+        if (q.dtype != self.torch.float32 or q.stride(1) != 1 or q.shape[1] != heads * (dim + rot_dim)
+                or w.shape != (heads, rank, dim) or not w.is_contiguous() or w.dtype != rows.dtype):
+            raise KernelError("latent_queries: shapes, strides or dtypes do not fit")
+        if table is not None and table.shape[2] * 2 != rot_dims:
+            raise KernelError("rotary table does not match the rotated dims")
+        self._check(self._part_lib("latent").ie_headwise_mma(
+            q.data_ptr(), 1, q.stride(0), dim + rot_dim, w.data_ptr(), rows.data_ptr(), rows.stride(0), rows.stride(1),
+            None, n, heads, rank, dim, positions.data_ptr(), self._ptr(table), rot_dims,
+            0 if table is None else table.shape[0], 1 if interleaved else 0, rot_dim, dim, rank, self._err_ptr,
+            self._stream()), "headwise_mma")
 
     @_kind("latent.headwise")
     def headwise_linear(self, x, w, out, row_scale=None) -> None:
@@ -1029,16 +1081,23 @@ class CudaOps:
         if (x.stride(2) != 1 or out.stride(2) != 1 or not w.is_contiguous() or w.shape != (heads, o, k)
                 or out.shape != (n, heads, o) or x.dtype != w.dtype or out.dtype != w.dtype):
             raise KernelError("headwise_linear: shapes, strides or dtypes do not fit")
+        lib = self._part_lib("latent")
         if x.dtype == self.torch.bfloat16 and n >= self.HEADWISE_LIBRARY_ROWS and o % 8 == 0 and k % 8 == 0:
             # many rows: one strided batched product of the library over the heads, written in place
             # (both views are batches of row-major matrices with a leading dimension), then the factors
             self.torch.bmm(x.permute(1, 0, 2), w.transpose(1, 2), out=out.permute(1, 0, 2))
             if row_scale is not None:
-                self._check(self._part_lib("latent").ie_scale_head_rows(
+                self._check(lib.ie_scale_head_rows(
                     out.data_ptr(), out.stride(0), out.stride(1), row_scale.data_ptr(), n, heads, o,
                     self._stream()), "scale_head_rows")
             return
-        self._check(self._part_lib("latent").ie_headwise_linear(
+        if x.dtype == self.torch.bfloat16 and self.headwise_mma and lib.ie_headwise_mma_ok(k):
+            self._check(lib.ie_headwise_mma(
+                x.data_ptr(), 0, x.stride(0), x.stride(1), w.data_ptr(), out.data_ptr(), out.stride(0), out.stride(1),
+                self._ptr(row_scale), n, heads, o, k, None, None, 0, 0, 0, 0, 0, 0, self._err_ptr, self._stream()),
+                "headwise_mma")
+            return
+        self._check(lib.ie_headwise_linear(
             x.data_ptr(), x.stride(0), x.stride(1), w.data_ptr(), out.data_ptr(), out.stride(0), out.stride(1),
             self._ptr(row_scale), _dtype_code(x), n, heads, o, k, self._stream()), "headwise_linear")
 
@@ -1156,8 +1215,8 @@ class CudaOps:
     def sandwich_norm(self, h, delta, bias, post_weight, post_eps, weight, eps, out, rows=None, second=None,
                       extra=None) -> None:
         """``y = delta (+ second) (+ bias) (+ extra)``; ``y <- rms(y) * post_weight`` if given; ``h += y``
-        (not with ``rows``); ``out = rms(h) * weight`` unless ``out`` is None.  ``delta`` may be None.
-        ``second``: another sublayer's output, whole or in parts like ``delta``; ``extra``: a 32-bit array
+        (not with ``rows``); ``out = rms(h) * weight``, or ``h`` in ``out``'s dtype if there is no ``weight``, unless
+        ``out`` is None.  ``delta`` may be None.  ``second``: another sublayer's output, whole or in parts like ``delta``; ``extra``: a 32-bit array
         of the stream's shape, added row by row."""
         n = h.shape[0] if rows is None else rows.shape[0]
         parts, stride = self._partials(delta)
@@ -1278,18 +1337,21 @@ class CudaOps:
             ctx.num_seqs, heads, state.shape[0], self._stream()), "mlstm_gates")
 
     @_kind("recurrent.rule")
-    def gated_recurrence(self, q, a, w, gates, v, state, slots, ctx, out, heads, dim, vdim, cols, q_scale) -> None:
+    def gated_recurrence(self, q, a, w, gates, v, state, slots, ctx, out, heads, dim, vdim, cols, q_scale,
+                         heads_per_unit: int = 1) -> None:
         """``S <- diag(a) S + w u^T; o = S^T q`` per head over every request's tokens of the step, from
         and to its slot (``[heads, cols, dim]``).  ``q``, ``a``, ``w``: views ``[N, heads * dim]``;
         ``v``: view ``[N, heads * vdim]``; with ``gates`` (``[N, heads, 3]``) ``a`` is the gates' decay,
         ``u = gate * v``, and column ``vdim`` (if ``cols = vdim + 1``) carries the value 1.  Gates of shape
-        ``[1, heads, 3]`` are every token's (a decay that is a constant per head)."""
+        ``[1, heads, 3]`` are every token's (a decay that is a constant per head).  So many neighbouring heads as
+        ``heads_per_unit`` share their rows of ``q`` and ``w``, which then hold that many times fewer columns."""
         if dim > 512:
             raise KernelError(f"the recurrence kernel takes key sizes up to 512, not {dim}")
         self._check(self._part_lib("recurrent").ie_gated_recurrence(
             q.data_ptr(), q.stride(0), self._ptr(a), 0 if a is None else a.stride(0), w.data_ptr(), w.stride(0),
             self._ptr(gates), 0 if gates is None or (gates.dim() == 3 and gates.shape[0] == 1) else 3 * heads,
-            v.data_ptr(), v.stride(0), state.data_ptr(), state.stride(0), slots.data_ptr(), ctx.cu_q.data_ptr(), out.data_ptr(), ctx.num_seqs, heads, dim, vdim, cols, float(q_scale),
+            v.data_ptr(), v.stride(0), state.data_ptr(), state.stride(0), slots.data_ptr(), ctx.cu_q.data_ptr(), out.data_ptr(), ctx.num_seqs, heads,
+            heads_per_unit, dim, vdim, cols, float(q_scale),
             state.shape[0], self._stream()), "gated_recurrence")
 
     @_kind("recurrent.out")
@@ -1380,6 +1442,115 @@ class CudaOps:
             "retention_chunks" if chunks else "retention_step")
         self.launches += 2 if chunks else 0
 
+    def _state_space_lib(self, n: int, p: int):
+        key = (-(-n // 16), -(-p // 16))
+        lib = self._state_space_libs.get(key)
+        if lib is None:
+            path = build_state_space(n, p)
+            try:
+                lib = ctypes.CDLL(str(path))
+            except OSError as exc:
+                raise KernelError(f"the kernel library {path} could not be loaded: {exc}") from exc
+            P, I, L = c_void_p, c_int, ctypes.c_longlong
+            lib.ie_state_space_step.argtypes = [P, I, I, I, I, I, P, P, I, P, P, P, P, L, P, P, I, I, P, I, P, P]
+            lib.ie_state_space_chunks.argtypes = [P, I, P, I, I, I, I, P, I, P, P, L, P, P, I, I, P, P, P, P, I, P, P]
+            lib.ie_state_space_step.restype = lib.ie_state_space_chunks.restype = c_int
+            self._state_space_libs[key] = lib
+        return lib
+
+    # requests that bring at most so many tokens each go through the kernel that takes them one by one;
+    # longer portions are cut into chunks of so many
+    STATE_SPACE_STEP, STATE_SPACE_CHUNK = 8, 64
+
+    def state_space(self, proj, ctx, conv_w, conv_b, dt_bias, A_log, skip, norm_w, norm_parts, eps, state, slots, out,
+                    heads, groups, dim, vdim, ws) -> None:
+        """State-space duality (Mamba-2) from the fused 32-bit projection, a view ``[N, >= columns]`` of (``heads *
+        vdim`` gates z, as many x, ``groups * dim`` B, as many C, ``heads`` step sizes): x, B and C pass a causal
+        convolution (``conv_w``: ``[channels, taps]``) with a bias and silu; ``dt = softplus(. + dt_bias)``; per head ``S
+        <- exp(-exp(A_log) dt) S + dt B x^T`` and ``y = S^T C + skip x`` from and to the requests' slots (``[heads, vdim,
+        dim]``, then the last ``taps - 1`` convolution inputs); ``out`` = ``y silu(z)``, each of the row's
+        ``norm_parts`` equal parts divided by its root mean square, times ``norm_w``.  A bfloat16 ``out`` with sizes up
+        to 128 runs the fused kernels (steps of few tokens per request: two launches; prompt portions in
+        chunks on the tensor cores); 32-bit and other sizes convolution, recurrence and norm one after the other, whose
+        order of operations does not depend on the cutting."""
+        n, inner, channels, taps = proj.shape[0], heads * vdim, conv_w.shape[0], conv_w.shape[1]
+        f32, bf16 = self.torch.float32, self.torch.bfloat16
+        if (proj.dtype != f32 or proj.stride(1) != 1 or channels != inner + 2 * groups * dim or heads % groups
+                or proj.shape[1] < 2 * inner + 2 * groups * dim + heads or inner % norm_parts or dim > 512
+                or state.shape[1] < inner * dim + (taps - 1) * channels or out.stride(1) != 1):
+            raise KernelError("state_space: the sizes do not fit the projection, the state or the kernels")
+        raw, dt_pre = proj[:, inner: inner + channels], proj[:, inner + channels: inner + channels + heads]
+        y = ws.buffer("state_space.y", n, inner, f32)
+        fused = self.state_space_fused and out.dtype == bf16 and dim <= 128 and vdim <= 128
+        x_skip = z = None
+        if not fused:
+            conv = ws.buffer("state_space.conv", n, channels, f32)
+            gates = ws.buffer("state_space.gates", n, 3 * heads, f32).view(n, heads, 3)
+            self._conv_silu(raw, conv_w, conv_b, state, inner * dim, slots, ctx, conv, dt_pre, dt_bias, A_log, gates, heads)
+            at_b, at_c = inner, inner + groups * dim
+            # (a token of a fixed-size launch's padding has gates too: the view is per token, never shared)
+            self.gated_recurrence(conv[:, at_c:], None, conv[:, at_b: at_c], gates.view(n, 3 * heads), conv[:, :inner], state,
+                                  slots, ctx, y, heads, dim, vdim, vdim, 1.0, heads_per_unit=heads // groups)
+            x_skip, z = conv, proj
+        else:
+            bounds = getattr(ctx, "bounds", None)
+            longest = bounds[0] if bounds is not None else ctx.max_q_len  # (a captured step: its token bound)
+            if longest <= self.STATE_SPACE_STEP:
+                self._state_space_step(proj, conv_w, conv_b, dt_bias, A_log, skip, state, slots, ctx, y, heads, groups, dim,
+                                       vdim, longest)
+            else:
+                ld = -(-channels // 8) * 8
+                conv = ws.buffer("state_space.conv", n, ld, bf16)
+                gates = ws.buffer("state_space.gates", n, 3 * heads, f32).view(n, heads, 3)
+                self._conv_silu(raw, conv_w, conv_b, state, inner * dim, slots, ctx, conv, dt_pre, dt_bias, A_log, gates, heads)
+                size = self.STATE_SPACE_CHUNK
+                chunks = bounds[0] // size + bounds[1] if bounds is not None else sum(-(-q // size) for q in ctx.q_lens)
+                self._state_space_chunks(proj, conv, gates, skip, state, slots, ctx, y, heads, groups, dim, vdim, chunks, ws)
+        self._gated_group_norm(y, x_skip, skip, z, norm_w, eps, out, norm_parts, vdim, raw, state, inner * dim, slots, ctx,
+                               channels, taps)
+
+    @_kind("recurrent.conv")
+    def _conv_silu(self, raw, w, bias, state, tail_at, slots, ctx, out, dt_pre, dt_bias, A_log, gates, heads) -> None:
+        self._check(self._part_lib("recurrent").ie_conv_silu(
+            raw.data_ptr(), raw.stride(0), w.data_ptr(), bias.data_ptr(), state.data_ptr(), state.stride(0), tail_at,
+            slots.data_ptr(), ctx.seq_of_token.data_ptr(), ctx.cu_q.data_ptr(), out.data_ptr(), out.stride(0),
+            _dtype_code(out), raw.shape[0], w.shape[0], w.shape[1], state.shape[0], dt_pre.data_ptr(),
+            dt_bias.data_ptr(), A_log.data_ptr(), gates.data_ptr(), heads, self._err_ptr, self._stream()), "conv_silu")
+
+    @_kind("recurrent.state_space")
+    def _state_space_step(self, proj, conv_w, conv_b, dt_bias, A_log, skip, state, slots, ctx, y, heads, groups, dim, vdim,
+                          longest) -> None:
+        self._check(self._state_space_lib(dim, vdim).ie_state_space_step(
+            proj.data_ptr(), proj.stride(0), heads, groups, dim, vdim, conv_w.data_ptr(), conv_b.data_ptr(),
+            conv_w.shape[1], dt_bias.data_ptr(), A_log.data_ptr(), skip.data_ptr(), state.data_ptr(), state.stride(0),
+            slots.data_ptr(), ctx.cu_q.data_ptr(), ctx.num_seqs, longest, y.data_ptr(), state.shape[0], self._err_ptr,
+            self._stream()), "state_space_step")
+
+    @_kind("recurrent.state_space")
+    def _state_space_chunks(self, proj, conv, gates, skip, state, slots, ctx, y, heads, groups, dim, vdim, chunks, ws) -> None:
+        torch = self.torch
+        # (one buffer: the chunks' sums, the states before them as two terms, the chunks' decays)
+        size = chunks * heads * dim * vdim
+        pad = -(-size // 4) * 4
+        scratch = ws.buffer("state_space.state", 1, 2 * pad + chunks * heads, torch.float32, rows_cap=None)[0]
+        u, before, total = scratch[:size], scratch[pad: pad + size], scratch[2 * pad:]
+        self._check(self._state_space_lib(dim, vdim).ie_state_space_chunks(
+            conv.data_ptr(), conv.stride(0), gates.data_ptr(), heads, groups, dim, vdim, proj.data_ptr(),
+            proj.stride(0), skip.data_ptr(), state.data_ptr(), state.stride(0), slots.data_ptr(), ctx.cu_q.data_ptr(),
+            ctx.num_seqs, chunks, u.data_ptr(), total.data_ptr(), before.data_ptr(), y.data_ptr(), state.shape[0],
+            self._err_ptr, self._stream()), "state_space_chunks")
+        self.launches += 2
+
+    @_kind("recurrent.out")
+    def _gated_group_norm(self, y, x_skip, skip, z, norm_w, eps, out, parts, vdim, raw, state, tail_at, slots, ctx, channels,
+                          taps) -> None:
+        self._check(self._part_lib("recurrent").ie_gated_group_norm(
+            y.data_ptr(), self._ptr(x_skip), 0 if x_skip is None else x_skip.stride(0), skip.data_ptr(), self._ptr(z),
+            0 if z is None else z.stride(0), norm_w.data_ptr(), eps, out.data_ptr(), out.stride(0), _dtype_code(out),
+            y.shape[0], y.shape[1], parts, vdim, raw.data_ptr(), raw.stride(0), state.data_ptr(), state.stride(0), tail_at,
+            slots.data_ptr(), ctx.seq_of_token.data_ptr(), ctx.cu_q.data_ptr(), channels, taps, state.shape[0],
+            self._stream()), "gated_group_norm")
+
     @_kind("recurrent.gates")
     def lowrank_decay(self, y, w2, bias, tau: float, decay) -> None:
         """``decay = sigmoid(y @ w2^T + bias) ** (1 / tau)`` as ``exp(logsigmoid(.) / tau)``, all 32-bit.
@@ -1397,7 +1568,8 @@ class CudaOps:
                            v_cache, slot_mapping, heads, kv_heads, dim, vdim, page_size, bias=None,
                            value_norm: bool = False, values_from_keys: bool = False,
                            interleaved: bool = False, unit_norm: bool = False, q_head_scale=None,
-                           warm_coef: float = 0.0, warm_every: int = 0) -> None:
+                           warm_coef: float = 0.0, warm_every: int = 0, norm_over: str = "head",
+                           value_scale: float = 1.0) -> None:
         """The input stage of an attention with per-head norms (see ``csrc/gated_attention.cu``).
         ``q_weight`` / ``k_weight`` None: queries and keys are not normalised; ``bias``: one row laid
         out like the projection's first columns, added first; ``value_norm``: value heads are divided
@@ -1407,7 +1579,11 @@ class CudaOps:
         rotation pairs entry ``2i`` with ``2i + 1`` instead of ``i`` with ``i + rot_dims / 2``.
         ``unit_norm`` (without weights): queries and keys are divided by their root mean square.
         ``q_head_scale`` (32-bit, one per head) multiplies the query heads; with ``warm_every`` > 0 the
-        queries at position ``p`` are multiplied by ``1 + warm_coef * ln(floor((p + 1) / warm_every) + 1)``."""
+        queries at position ``p`` are multiplied by ``1 + warm_coef * ln(floor((p + 1) / warm_every) + 1)``.  ``norm_over="all"``: one norm over all of
+        a token's query columns and one over its key columns, with weights of those lengths.  ``value_scale``
+        multiplies the cached values."""
+        if norm_over not in ("head", "all"):
+            raise KernelError(f"qk_norm_rope_write: no norm over {norm_over!r}")
         if unit_norm and q_weight is not None:
             raise KernelError("qk_norm_rope_write: a norm with weights or one without, not both")
         if q_head_scale is not None and (q_head_scale.dtype != self.torch.float32 or q_head_scale.numel() != heads):
@@ -1421,12 +1597,24 @@ class CudaOps:
             raise KernelError("qk_norm_rope_write reads the fused 32-bit projection of queries, keys and values")
         if bias is not None and (bias.dtype != self.torch.float32 or bias.numel() < need):
             raise KernelError("qk_norm_rope_write: the bias must be a 32-bit row of the projection's width")
+        if norm_over == "all":
+            if (q_weight is None or q_weight.numel() != heads * dim or k_weight.numel() != kv_heads * dim or unit_norm
+                    or value_norm or values_from_keys or q_head_scale is not None or warm_every):
+                raise KernelError("qk_norm_rope_write: norms over all heads take weights of all query and all key "
+                                  "columns, and nothing else is done to the heads")
+            self._check(self._part_lib("gated_attn").ie_qk_wide_norm_rope_write(
+                proj.data_ptr(), proj.stride(0), positions.data_ptr(), self._ptr(table), rot_dims,
+                0 if table is None else table.shape[0], self._ptr(bias), 1 if interleaved else 0, q_weight.data_ptr(),
+                k_weight.data_ptr(), eps, float(value_scale), q_out.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(),
+                _dtype_code(q_out), self._ptr(slot_mapping), proj.shape[0], heads, kv_heads, dim, vdim, page_size,
+                k_cache.shape[0], self._err_ptr, self._stream()), "qk_wide_norm_rope_write")
+            return
         self._check(self._part_lib("gated_attn").ie_qk_norm_rope_write(
             proj.data_ptr(), proj.stride(0), positions.data_ptr(), self._ptr(table), rot_dims,
             0 if table is None else table.shape[0], self._ptr(bias), 1 if value_norm else 0,
             1 if values_from_keys else 0, 1 if interleaved else 0,
             self._ptr(q_weight), self._ptr(k_weight), eps, 1 if unit_norm else 0, self._ptr(q_head_scale),
-            float(warm_coef), int(warm_every), q_out.data_ptr(),
+            float(warm_coef), int(warm_every), float(value_scale), q_out.data_ptr(),
             k_cache.data_ptr(), v_cache.data_ptr(), _dtype_code(q_out), self._ptr(slot_mapping), proj.shape[0],
             heads, kv_heads, dim, vdim, page_size, k_cache.shape[0], self._err_ptr, self._stream()),
             "qk_norm_rope_write")
@@ -1471,7 +1659,7 @@ class CudaOps:
             block_tables.data_ptr(), block_tables.shape[1], ctx.seq_of_token.data_ptr(),
             ctx.positions.data_ptr(), out.data_ptr(), ctx.num_tokens, nh, nkv, hd, vdim, vdim, page_size,
             k_cache.shape[0], scale, 0, int(chunk or 0), head_bias.data_ptr(), None, None, 0, 0.0, 0, *self._NO_BIAS,
-            self._err_ptr, self._stream()), "sigmoid_attention")
+            nh * vdim, self._err_ptr, self._stream()), "sigmoid_attention")
 
     def _sink_attention_lib(self, hd: int, vdim: int, bias: str = "none"):
         lib = self._sinkattn_libs.get((hd, vdim, bias))
@@ -1483,7 +1671,7 @@ class CudaOps:
                 raise KernelError(f"the kernel library {path} could not be loaded: {exc}") from exc
             P, I, F = c_void_p, c_int, c_float
             lib.ie_sink_attention_mma.argtypes = [P, P, P, P, I, P, P, P, I, I, I, I, I, I, F, I, P, P, I, P, I, I, I,
-                                                  F, I, I, I, P, P, P, I, P, P]
+                                                  F, I, I, I, P, P, P, I, I, P, P]
             lib.ie_sink_attention_mma.restype = c_int
             self._sinkattn_libs[(hd, vdim, bias)] = lib
         return lib
@@ -1531,8 +1719,10 @@ class CudaOps:
         keep = int(keep_first or 0) if window else 0
         if cap < 0 or keep < 0:
             raise KernelError("sink_attention: the cap of the scores and the kept keys cannot be negative")
+        if out.stride(1) != 1 or out.stride(0) < nh * vdim:
+            raise KernelError("sink_attention: the output's rows must have unit stride")
         if (self.sink_mma and q.dtype == self.torch.bfloat16 and hd % 16 == 0 and vdim % 16 == 0
-                and 16 <= hd <= 256 and 16 <= vdim <= 256 and page_size & (page_size - 1) == 0):
+                and out.stride(0) % 2 == 0 and out.data_ptr() % 4 == 0 and 16 <= hd <= 256 and 16 <= vdim <= 256 and page_size & (page_size - 1) == 0):
             lib = self._sink_attention_lib(hd, vdim, kind)
             bounds = getattr(ctx, "bounds", None)
             longest = bounds[0] if bounds is not None else ctx.max_q_len  # (a captured step: its token bound)
@@ -1559,7 +1749,7 @@ class CudaOps:
                 block_tables.shape[1], ctx.cu_q.data_ptr(), ctx.ctx_lens.data_ptr(), out.data_ptr(), ctx.num_seqs,
                 longest, nh, nkv, page_size, k_cache.shape[0], scale, int(window or 0), self._ptr(sinks),
                 self._ptr(gate), 0 if gate is None else gate.stride(0), self._ptr(scratch), splits, per_split,
-                ctx.num_tokens, cap, keep, kept_splits if scratch is not None else 0, *by_distance, self._err_ptr,
+                ctx.num_tokens, cap, keep, kept_splits if scratch is not None else 0, *by_distance, out.stride(0), self._err_ptr,
                 self._stream()),
                 "sink_attention_mma")
             if scratch is not None:  # (the call launched the merge kernel too)
@@ -1571,7 +1761,8 @@ class CudaOps:
             block_tables.data_ptr(), block_tables.shape[1], ctx.seq_of_token.data_ptr(),
             ctx.positions.data_ptr(), out.data_ptr(), ctx.num_tokens, nh, nkv, hd, vdim, vdim, page_size,
             k_cache.shape[0], scale, int(window or 0), 0, None, self._ptr(sinks), self._ptr(gate),
-            0 if gate is None else gate.stride(0), cap, keep, *by_distance, self._err_ptr, self._stream()), "sink_attention")
+            0 if gate is None else gate.stride(0), cap, keep, *by_distance, out.stride(0), self._err_ptr,
+            self._stream()), "sink_attention")
 
     @_kind("activation")
     def silu_mul(self, gate_up, out, interleave: int = 0) -> None:

@@ -176,7 +176,20 @@ class CarriesInputRows:
         return None if self._extra_rows is None else proj[:, at: at + self._extra_count]
 
 
-class Mixer(CarriesInputRows, Part):
+class LeavesProducts:
+    """A mixer that starts with one product over its input and ends with one over its result can leave both
+    products to whoever runs several mixers side by side: then one product over the stacked input rows serves them
+    all, and one over the results next to each other adds their outputs up.  Such a mixer says so with
+    ``leaves_products`` and offers ``input_rows(tensors)`` (the stacked row blocks, in the compute dtype),
+    ``output_matrix(tensors)`` (``[hidden, out_size]``) and ``run(proj, ctx, binding, out)``: from its columns of the
+    32-bit input product to its columns of the array the output product reads, times ``output_scale``."""
+
+    leaves_products = False
+    output_scale = 1.0  # the factor of the mixer's result, set before ``bind``
+    products_elsewhere = False  # set by whoever takes the products over
+
+
+class Mixer(LeavesProducts, CarriesInputRows, Part):
     category = "mixer"
 
     def cache_request(self) -> PagedKVRequest | StateRequest | None | tuple:

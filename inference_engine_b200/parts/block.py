@@ -10,7 +10,8 @@ feed-forward's output as a pending ``delta`` for the next norm to add.
 ``x <- x + post'(feed_forward(pre'(x)))``.  The norm after a sublayer, the add and the norm before the
 next sublayer are one kernel: the block hands its last sublayer's raw output on as the pending delta
 together with what is to be done to it before the add (``output_post``: an output bias, if the
-sublayer has one, and the norm).
+sublayer has one, and the norm).  With ``identity`` for the norms before the sublayers this is the
+post-norm arrangement, ``x <- x + post(mixer(x))``, in as many kernels.
 
 ``gated_prenorm_residual``: the pre-norm arrangement with a learned gate on each sublayer's way into
 the stream: ``x <- x + sigmoid(W1 h + b1) * mixer(h)`` with ``h = norm(x)``, then the same with

@@ -1,5 +1,5 @@
 """Norms over the last dimension, with the residual add fused in: root mean square, layer norm, dynamic
-tanh; and what may be done to a sublayer's output on its way into the residual stream or streams.
+tanh, none at all; and what may be done to a sublayer's output on its way into the residual stream or streams.
 
 Formula (engine/model/layers.py:41-43): ``normed = x * rsqrt(mean(x^2) + eps)`` in 32-bit,
 then ``weight * normed``.  The residual stream is kept in 32-bit here, so square, mean,
@@ -51,6 +51,34 @@ class RMSNorm(Norm):
         return out
 
 
+@register_part("norm", "identity")
+class NoNorm(Norm):
+    """No norm where an arrangement has one: a sublayer that reads the residual stream as it is.  The stream is
+    brought up to date and handed on in the compute dtype (the 32-bit stream itself where that is 32-bit
+    and nothing selects rows)."""
+
+    def __init__(self, size: int, dtype) -> None:
+        self.size, self.dtype = int(size), dtype
+
+    @classmethod
+    def from_spec(cls, params: dict, env: BuildEnv, **_):
+        return cls(params.get("size", env.hidden_size), env.torch_dtype)
+
+    def add_norm(self, h, delta, ctx, rows=None, tag: str = "norm", delta_scale: float = 1.0, delta_post=None):
+        import torch
+
+        if delta_scale != 1.0:
+            raise ValueError("a stream that is handed on as it is takes a delta without a residual multiplier")
+        out = None
+        if rows is not None or self.dtype != torch.float32:
+            out = ctx.ws.buffer(tag, h.shape[0] if rows is None else rows.shape[0], self.size, self.dtype)
+        if delta_post is not None:
+            delta_post.add_norm(h, delta, ctx, None, 0.0, out, rows)
+        elif delta is not None or out is not None:
+            ctx.ops.sandwich_norm(h, delta, None, None, 0.0, None, 0.0, out, rows)
+        return h if out is None else out
+
+
 class PostNorm:
     """What a block wants done to a sublayer's output before it enters the residual stream: a bias
     (or None), then an RMS norm.  Carried beside the pending delta to whoever adds it."""
@@ -59,7 +87,7 @@ class PostNorm:
         self.norm, self.bias = norm, bias
 
     def add_norm(self, h, delta, ctx, weight, eps, out, rows) -> None:
-        """``h += norm(delta + bias)`` (not with ``rows``); ``out = rms(h) * weight``."""
+        """``h += norm(delta + bias)`` (not with ``rows``); ``out = rms(h) * weight`` (no weight: ``h`` as it is)."""
         ctx.ops.sandwich_norm(h, delta, self.bias, self.norm.weight, self.norm.eps, weight, eps, out, rows)
 
     def settle(self, h, delta, ctx) -> None:

@@ -3,7 +3,7 @@
 ``learned``: a table of vectors added to the embedding.
 
 ``rotary``: rotation of query and key halves by position-dependent angles, with the
-optional Llama 3 frequency scaling.  Frequencies follow engine/model/layers.py:55-73 and
+optional Llama 3 or YaRN frequency scaling.  Frequencies follow engine/model/layers.py:55-73 and
 angles engine/model/layers.py:75-79: everything is 32-bit; the table holds cos and sin of
 ``position * inv_freq`` for every position the engine can feed, so the kernels read the
 same values a whole-sequence computation would.
@@ -37,6 +37,39 @@ def rotary_inv_freq(rotary_dim: int, theta: float, scaling: dict | None):
     return torch.where(medium, smoothed, scaled)
 
 
+def exact_frequencies(rotary_dim: int, theta: float, scaling: dict | None):
+    """``(frequencies, amplitude)`` worked out in 64-bit: ``theta^(-2j/dim)``, then the scaling.  ``kind`` ``llama3``
+    (the default): as in :func:`rotary_inv_freq`.  ``kind`` ``yarn`` (``factor``, ``original``, ``fast``, ``slow``): the pair
+    that turns ``t`` times over the original length is number ``dim * ln(original / (2 pi t)) / (2 ln theta)``; pairs up
+    to the one at ``fast`` turns keep their frequency, pairs from the one at ``slow`` turns on have it divided by
+    ``factor``, a straight line between; cos and sin are multiplied by the amplitude ``0.1 ln(factor) + 1``."""
+    import torch
+
+    j = torch.arange(0, rotary_dim, 2, dtype=torch.float64)
+    freq = torch.exp(-(j / rotary_dim) * math.log(theta))
+    if not scaling:
+        return freq, 1.0
+    factor = float(scaling["factor"])
+    kind = scaling.get("kind", "llama3")
+    if kind == "yarn":
+        def pair_at(turns: float) -> float:
+            return rotary_dim * math.log(float(scaling["original"]) / (2 * math.pi * turns)) / (2 * math.log(theta))
+
+        low = max(math.floor(pair_at(float(scaling["fast"]))), 0)
+        high = min(math.ceil(pair_at(float(scaling["slow"]))), rotary_dim - 1)
+        ramp = ((torch.arange(rotary_dim // 2, dtype=torch.float64) - low) / max(high - low, 0.001)).clamp(0.0, 1.0)
+        return freq / factor * ramp + freq * (1.0 - ramp), 0.1 * math.log(factor) + 1.0
+    if kind != "llama3":
+        raise ValueError(f"no rotary frequency scaling of kind {kind!r}")
+    low_f, high_f = float(scaling["low_freq_factor"]), float(scaling["high_freq_factor"])
+    original = float(scaling["original_max_position_embeddings"])
+    wavelength = 2 * math.pi / freq
+    blend = (original / wavelength - low_f) / (high_f - low_f) if high_f != low_f else torch.zeros_like(freq)
+    between = (1 - blend) * freq / factor + blend * freq
+    scaled = torch.where(wavelength > original / low_f, freq / factor, between)
+    return torch.where(wavelength < original / high_f, freq, scaled), 1.0
+
+
 @register_part("position", "rotary")
 class RotaryEncoding(PositionEncoding):
     LAYOUTS = ("halves", "interleaved")
@@ -52,9 +85,11 @@ class RotaryEncoding(PositionEncoding):
         self.layout = layout
         if angles not in ("float32", "float64"):
             raise ValueError(f"rotary angles are computed in float32 or float64, not {angles!r}")
-        # "float64": frequencies theta^(-2j/dim), angles and their cos and sin are worked out in
-        # 64-bit and rounded once to the 32-bit table (no frequency scaling in this mode)
+        # "float64": frequencies (scaled or not), angles and their cos and sin are worked out in
+        # 64-bit and rounded once to the 32-bit table
         self.angles = angles
+        if angles == "float32" and scaling and scaling.get("kind", "llama3") != "llama3":
+            raise ValueError("32-bit rotary angles know the llama3 frequency scaling only")
         self.rotary_dim, self.theta, self.scaling = int(rotary_dim), float(theta), scaling
         self.max_positions = int(max_positions)
         self.inv_freq = self._table = None
@@ -70,13 +105,10 @@ class RotaryEncoding(PositionEncoding):
         import torch
 
         if self.angles == "float64":
-            if self.scaling:
-                raise ValueError("64-bit rotary angles take no frequency scaling")
-            j = torch.arange(0, self.rotary_dim, 2, dtype=torch.float64)
-            inv_freq = torch.exp(-(j / self.rotary_dim) * math.log(self.theta))
+            inv_freq, amplitude = exact_frequencies(self.rotary_dim, self.theta, self.scaling)
             freqs = torch.arange(self.max_positions, dtype=torch.float64)[:, None] * inv_freq[None, :]
             self.inv_freq = inv_freq.float().to(env.device)
-            self._table = torch.stack((freqs.cos(), freqs.sin()), dim=1).float().contiguous().to(env.device)
+            self._table = (torch.stack((freqs.cos(), freqs.sin()), dim=1) * amplitude).float().contiguous().to(env.device)
             return
         self.inv_freq = rotary_inv_freq(self.rotary_dim, self.theta, self.scaling).to(env.device)
         pos = torch.arange(self.max_positions, device=env.device).float()

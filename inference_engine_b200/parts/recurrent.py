@@ -29,6 +29,12 @@ rotated by position, if a rotary encoding is named), ``v = W_v h``; ``S <- decay
 q * dim^-1/2``; each head's ``o`` is divided by its root mean square over ``vdim`` (no weight); the heads
 together are multiplied by ``silu(W_g h)``; ``W_o``.
 
+``state_space``: state-space duality (Mamba-2).  ``W_in h`` holds a gate ``z`` and values ``x`` (``heads * vdim`` each),
+``B`` and ``C`` (``groups * state`` each, a group's heads share them) and a step size per head; ``x``, ``B`` and ``C``
+together pass a short causal convolution per channel with a bias and silu; ``dt = softplus(dt + bias)``; ``S <- exp(-exp(A_log)
+dt) S + dt B x^T``, ``y = S^T C + D x``; ``y silu(z)`` is divided by its root mean square in ``norm_parts`` equal
+parts and multiplied by a weight; ``W_o``.  The convolution's last ``taps - 1`` inputs are kept behind ``S``.
+
 Gates, decays, the state and the read-out are 32-bit in every precision; the projections run in
 the compute dtype with 32-bit sums.  The state lives in the request's state slot: ``S`` column by
 column (``[heads, columns, dim]``; the normaliser is one more column), then the maxima.
@@ -331,3 +337,78 @@ class Retention(Mixer):
         ops.retention(proj, ctx, self.position.rotary_table() if rot_dims else None, rot_dims, self.gates, self.powers,
                       group.state[binding.slot], group.slots, out, self.heads, self.dim, self.vdim, self.eps, ws)
         return ops.linear(out, self.w_o, ws=ws, tag="retention.delta", out_dtype=f32, allow_split=self.allow_split)
+
+
+@register_part("mixer", "state_space")
+class StateSpace(Mixer):
+    allow_split = True
+    leaves_products = True
+
+    def __init__(self, *, names: dict, hidden_size: int, heads: int, vdim: int, state: int, groups: int, taps: int,
+                 norm_parts: int, eps: float, dtype) -> None:
+        if heads % groups:
+            raise ValueError(f"{heads} heads cannot share {groups} groups of B and C")
+        if taps < 1:
+            raise ValueError("the convolution needs at least one tap")
+        if norm_parts < 1 or (heads * vdim) % norm_parts:
+            raise ValueError(f"rows of {heads * vdim} entries cannot be normalised in {norm_parts} equal parts")
+        self.names, self.hidden_size = dict(names), hidden_size
+        self.heads, self.vdim, self.state, self.groups, self.taps = heads, vdim, state, groups, int(taps)
+        self.norm_parts, self.eps, self.dtype = int(norm_parts), float(eps), dtype
+        self.out_size = heads * vdim
+        self.channels = self.out_size + 2 * groups * state
+        self.in_size = self.out_size + self.channels + heads
+        self.w_in = self.w_o = None
+
+    @classmethod
+    def from_spec(cls, params: dict, env: BuildEnv, **_):
+        return cls(names=params["names"], hidden_size=params.get("hidden_size", env.hidden_size),
+                   heads=params["heads"], vdim=params["vdim"], state=params["state"], groups=params.get("groups", 1),
+                   taps=params["taps"], norm_parts=params.get("norm_parts", 1), eps=params["eps"], dtype=env.torch_dtype)
+
+    def weights(self) -> dict[str, WeightDecl]:
+        n, h = self.names, self.hidden_size
+        per_head = {n[k]: WeightDecl((self.heads,), "vector", init)
+                    for k, init in (("dt_bias", "normal"), ("A_log", "zeros"), ("skip", "ones"))}
+        return {
+            n["in"]: WeightDecl((self.in_size, h)), n["conv"]: WeightDecl((self.channels, self.taps), "vector"),
+            n["conv_bias"]: WeightDecl((self.channels,), "vector"), **per_head,
+            n["out_norm"]: WeightDecl((self.out_size,), "vector", "ones_plus_normal"),
+            n["o"]: WeightDecl((h, self.out_size)),
+        }
+
+    def input_rows(self, tensors) -> list:
+        return [tensors[self.names["in"]].to(self.dtype)]
+
+    def output_matrix(self, tensors):
+        return tensors[self.names["o"]].to(self.dtype).contiguous()
+
+    def bind(self, tensors, env: BuildEnv) -> None:
+        n = self.names
+        if not self.products_elsewhere:
+            self.w_in, self.w_o = self.input_rows(tensors)[0].contiguous(), self.output_matrix(tensors)
+        vec = lambda key: tensors[n[key]].float().contiguous()  # noqa: E731
+        self.conv, self.conv_bias, self.dt_bias, self.A_log, self.skip = map(
+            vec, ("conv", "conv_bias", "dt_bias", "A_log", "skip"))
+        self.out_norm = (vec("out_norm") * self.output_scale).contiguous()
+
+    def cache_request(self) -> StateRequest:
+        return StateRequest((self.out_size * self.state + (self.taps - 1) * self.channels,))
+
+    def run(self, proj, ctx, binding, out) -> None:
+        """From the input product's 32-bit columns to the normalised rows, times ``output_scale`` (a part of the norm's
+        weight)."""
+        group = ctx.groups[binding.group]
+        ctx.ops.state_space(proj, ctx, self.conv, self.conv_bias, self.dt_bias, self.A_log, self.skip, self.out_norm,
+                            self.norm_parts, self.eps, group.state[binding.slot], group.slots, out, self.heads, self.groups,
+                            self.state, self.vdim, ctx.ws)
+
+    def forward(self, x, ctx, binding):
+        import torch
+
+        ops, ws = ctx.ops, ctx.ws
+        proj = ops.linear(x, self.w_in, ws=ws, tag="state_space.in", out_dtype=torch.float32)
+        out = ws.buffer("state_space.out", x.shape[0], self.out_size, self.dtype)
+        self.run(proj, ctx, binding, out)
+        return ops.linear(out, self.w_o, ws=ws, tag="state_space.delta", out_dtype=torch.float32,
+                          allow_split=self.allow_split)

@@ -25,7 +25,9 @@ residual stream (``output_bias``).  ``unit_qk``: query and key heads are divided
 square over ``dim`` (no weight).  ``temp`` among the names: a number per head that multiplies its scores
 (taken into the queries before they are rounded).  ``warmth = (coef, every)``: the queries at position
 ``p`` are multiplied by ``1 + coef * ln(floor((p + 1) / every) + 1)``.  ``gate`` among the names, in
-place of a head gate: a sigmoid of a linear map of the input per head and value entry.
+place of a head gate: a sigmoid of a linear map of the input per head and value entry.  ``q_norm`` and
+``k_norm`` among the names: all query columns of a token together are divided by their root mean square and
+multiplied by a weight as long, and so are its key columns, before they are split into heads and rotated.
 
 A bias by the distance ``n`` of query and key, added to the score after scale and temperature: with
 ``r1`` and ``r2`` among the names ``-r1[head] * ln(1 + r2[head] * n)``; with ``rel`` among them ``rel[bucket(n),
@@ -106,6 +108,10 @@ class SinkAttention(Mixer):
                 raise ValueError("the bucketed bias needs its number of buckets and a largest distance beyond half of them")
         if names.get("gate") and names.get("head_gate"):
             raise ValueError("a gate per head or one per value entry, not both")
+        if (names.get("q_norm") is None) != (names.get("k_norm") is None):
+            raise ValueError("queries and keys are normalised together or not at all")
+        if names.get("q_norm") and (unit_qk or value_norm or values != "projected" or names.get("temp") or warmth is not None):
+            raise ValueError("norms over all heads leave nothing else to be done to heads before the rotation")
         if warmth is not None and int(warmth[1]) < 1:
             raise ValueError("the queries' warmth steps up after at least one position")
         self.unit_qk = bool(unit_qk)
@@ -121,7 +127,10 @@ class SinkAttention(Mixer):
         self.sink_value = None if sink_value is None else float(sink_value)
         self.keep_first = int(keep_first)
         self.qkv_size = (heads + kv_heads) * dim + (0 if self.values_from_keys else kv_heads * vdim)
-        self.w_in = self.w_o = self.bias = self.sinks = self.output_bias = None
+        self.w_in = self.w_o = self.bias = self.sinks = self.output_bias = self.qk_norms = None
+        self.out_size = heads * vdim
+        # (an output bias is left to the add, which a mixer beside another one does not see)
+        self.leaves_products = "o_bias" not in self.names
 
     @classmethod
     def from_spec(cls, params: dict, env: BuildEnv, **_):
@@ -150,6 +159,9 @@ class SinkAttention(Mixer):
                 out[n["v_bias"]] = WeightDecl((self.kv_heads * self.vdim,), "vector")
         if "o_bias" in n:
             out[n["o_bias"]] = WeightDecl((h,), "vector")
+        if "q_norm" in n:
+            out[n["q_norm"]] = WeightDecl((self.heads * self.dim,), "vector", "ones_plus_normal")
+            out[n["k_norm"]] = WeightDecl((self.kv_heads * self.dim,), "vector", "ones_plus_normal")
         if "sink" in n:
             out[n["sink"]] = WeightDecl((self.heads,), "vector")
         if "head_gate" in n:
@@ -163,17 +175,21 @@ class SinkAttention(Mixer):
             out[n["rel"]] = WeightDecl((self.rel_buckets, self.heads), "vector")
         return out
 
+    def input_rows(self, tensors) -> list:
+        return [tensors[self.names[k]].to(self.dtype) for k in (*self.projected, "head_gate", "gate") if k in self.names]
+
+    def output_matrix(self, tensors):
+        return tensors[self.names["o"]].to(self.dtype).contiguous()
+
     def bind(self, tensors, env: BuildEnv) -> None:
         import torch
 
         n = self.names
-        rows = [tensors[n[k]].to(self.dtype) for k in self.projected]
-        if "head_gate" in n:
-            rows.append(tensors[n["head_gate"]].to(self.dtype))
-        if "gate" in n:
-            rows.append(tensors[n["gate"]].to(self.dtype))
-        self.w_in, self.extra_at = self._with_extra_rows(rows)
-        self.w_o = tensors[n["o"]].to(self.dtype).contiguous()
+        if not self.products_elsewhere:
+            self.w_in, self.extra_at = self._with_extra_rows(self.input_rows(tensors))
+            self.w_o = self.output_matrix(tensors)
+        if "q_norm" in n:
+            self.qk_norms = tuple(tensors[n[k]].float().contiguous() for k in ("q_norm", "k_norm"))
         if "q_bias" in n:
             self.bias = torch.cat([tensors[n[k]].float() for k in self.bias_names]).contiguous()
         if "o_bias" in n:
@@ -189,35 +205,43 @@ class SinkAttention(Mixer):
         if "sink" in n:
             self.sinks = tensors[n["sink"]].float().contiguous()
         elif self.sink_value is not None:
-            self.sinks = torch.full((self.heads,), self.sink_value, dtype=torch.float32, device=self.w_o.device)
+            self.sinks = torch.full((self.heads,), self.sink_value, dtype=torch.float32, device=tensors[n["o"]].device)
 
     def cache_request(self) -> PagedKVRequest:
         return PagedKVRequest(self.kv_heads, self.dim, self.window, value_dim=self.vdim, keep_first=self.keep_first)
 
-    def forward(self, x, ctx, binding: CacheBinding):
-        import torch
-
-        n = x.shape[0]
+    def run(self, proj, ctx, binding: CacheBinding, out) -> None:
+        """From the input product's 32-bit columns to the heads' results, times ``output_scale`` (taken into the values
+        before they are cached: the result is linear in them)."""
+        n = proj.shape[0]
         group = ctx.groups[binding.group]
         k_cache, v_cache = group.k[binding.slot], group.v[binding.slot]
-        ops, ws = ctx.ops, ctx.ws
-        proj = ops.linear(x, self.w_in, ws=ws, tag="sinkattn.in", out_dtype=torch.float32)
-        self.extra_out = self._extra_columns(proj, self.extra_at)
-        q = ws.buffer("sinkattn.q", n, self.heads * self.dim, self.dtype)
+        ops = ctx.ops
+        q = ctx.ws.buffer("sinkattn.q", n, self.heads * self.dim, self.dtype)
         table = self.position.rotary_table() if self.position is not None else None
         rot_dims = self.position.rotary_dim if self.position is not None else 0
-        ops.qk_norm_rope_write(proj, ctx.positions, table, rot_dims, None, None, self.eps, q, k_cache, v_cache,
+        q_norm, k_norm = self.qk_norms or (None, None)
+        ops.qk_norm_rope_write(proj, ctx.positions, table, rot_dims, q_norm, k_norm, self.eps, q, k_cache, v_cache,
                                group.slot_mapping if binding.writes else None, self.heads, self.kv_heads,
                                self.dim, self.vdim, group.page_size, bias=self.bias, value_norm=self.value_norm,
                                values_from_keys=self.values_from_keys,
                                interleaved=getattr(self.position, "layout", "halves") == "interleaved",
                                unit_norm=self.unit_qk, q_head_scale=self.temp, warm_coef=self.warmth[0],
-                               warm_every=self.warmth[1])
+                               warm_every=self.warmth[1], norm_over="head" if self.qk_norms is None else "all",
+                               value_scale=self.output_scale)
         gate = proj[:, self.qkv_size: self.qkv_size + self.gate_size] if self.gate_size else None
-        out = ws.buffer("sinkattn.out", n, self.heads * self.vdim, self.dtype)
         ops.sink_attention(q, k_cache, v_cache, group.block_tables, ctx, self.heads, self.kv_heads, self.dim,
                            self.vdim, group.page_size, self.scale, self.window, self.sinks, gate, out,
                            softcap=self.softcap, keep_first=self.keep_first, log_bias=self.log_bias,
                            bias_table=self.bias_table)
+
+    def forward(self, x, ctx, binding: CacheBinding):
+        import torch
+
+        ops, ws = ctx.ops, ctx.ws
+        proj = ops.linear(x, self.w_in, ws=ws, tag="sinkattn.in", out_dtype=torch.float32)
+        self.extra_out = self._extra_columns(proj, self.extra_at)
+        out = ws.buffer("sinkattn.out", x.shape[0], self.out_size, self.dtype)
+        self.run(proj, ctx, binding, out)
         return ops.linear(out, self.w_o, ws=ws, tag="sinkattn.delta", out_dtype=torch.float32,
                           allow_split=self.allow_split)

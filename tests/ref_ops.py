@@ -54,35 +54,52 @@ class RefOps:
 
     # --- latent attention ---------------------------------------------------------------------
 
-    def latent_prep(self, proj, positions, table, rot_dims, norm_w, eps, q_plain, q_abs, gate, cache,
-                    slot_mapping, heads, dim, rot_dim, rank, page_size):
-        n = proj.shape[0]
+    @staticmethod
+    def _turned(x, positions, table, rot_dims, interleaved):  # [n, ..., rot_dim]
+        if table is None or rot_dims == 0:
+            return x
+        cos, sin = table[positions.long(), 0], table[positions.long(), 1]  # [n, rot_dims/2]
+        while cos.dim() < x.dim():
+            cos, sin = cos.unsqueeze(1), sin.unsqueeze(1)
+        half = rot_dims // 2
+        first, second = ((slice(0, rot_dims, 2), slice(1, rot_dims, 2)) if interleaved
+                         else (slice(0, half), slice(half, rot_dims)))
+        out = x.clone()
+        u, v = x[..., first], x[..., second]
+        out[..., first] = u * cos - v * sin
+        out[..., second] = v * cos + u * sin
+        return out
+
+    def latent_prep(self, positions, table, rot_dims, *, heads, dim, rot_dim, rank, page_size, eps=0.0, interleaved=True,
+                    q=None, q_plain=None, q_abs=None, gate_pre=None, gate=None, dkv=None, norm_w=None, cache=None,
+                    slot_mapping=None, cq=None, cq_norm_w=None, cq_out=None):
+        def rms(x, w):
+            return x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * w
+
+        n = positions.shape[0]
         row = rank + rot_dim
-        q = proj[:, : heads * (dim + rot_dim)].reshape(n, heads, dim + rot_dim).float()
-        dkv = proj[:, heads * (dim + rot_dim): heads * (dim + rot_dim) + row].float()
-        g = proj[:, heads * (dim + rot_dim) + row:].float()
-
-        def rot(x):  # [n, ..., rot_dim]
-            if table is None or rot_dims == 0:
-                return x
-            cos, sin = table[positions.long(), 0], table[positions.long(), 1]  # [n, rot_dims/2]
-            while cos.dim() < x.dim():
-                cos, sin = cos.unsqueeze(1), sin.unsqueeze(1)
-            out = x.clone()
-            u, v = x[..., 0:rot_dims:2], x[..., 1:rot_dims:2]
-            out[..., 0:rot_dims:2] = u * cos - v * sin
-            out[..., 1:rot_dims:2] = v * cos + u * sin
-            return out
-
-        q_plain.copy_(q[..., :dim].reshape(n, heads * dim).to(q_plain.dtype))
-        q_abs.view(n, heads, row)[:, :, rank:] = rot(q[..., dim:]).to(q_abs.dtype)
-        gate.copy_(torch.sigmoid(g))
-        if slot_mapping is not None:
-            c = dkv[:, :rank]
-            c = c * torch.rsqrt(c.pow(2).mean(-1, keepdim=True) + eps) * norm_w
-            rows = torch.cat([c, rot(dkv[:, rank:])], dim=-1).to(cache.dtype)
+        if q is not None:
+            q = q.reshape(n, heads, dim + rot_dim).float()
+            q_plain.copy_(q[..., :dim].reshape(n, heads * dim).to(q_plain.dtype))
+            q_abs.view(n, heads, row)[:, :, rank:] = self._turned(q[..., dim:], positions, table, rot_dims, interleaved).to(q_abs.dtype)
+        if gate_pre is not None:
+            gate.copy_(torch.sigmoid(gate_pre.float()))
+        if cq is not None:
+            cq_out.copy_(rms(cq.float(), cq_norm_w).to(cq_out.dtype))
+        if dkv is not None and slot_mapping is not None:
+            dkv = dkv.float()
+            part = self._turned(dkv[:, rank:], positions, table, rot_dims, interleaved)
+            rows = torch.cat([rms(dkv[:, :rank], norm_w), part], dim=-1).to(cache.dtype)
             slots = slot_mapping.long()
             cache[slots // page_size, 0, slots % page_size] = rows
+
+    def latent_queries(self, q, w, q_abs, positions, table, rot_dims, *, heads, dim, rot_dim, rank, page_size,
+                       interleaved=True, ws):
+        n = q.shape[0]
+        plain = torch.empty(n, heads * dim, dtype=q_abs.dtype)
+        self.latent_prep(positions, table, rot_dims, heads=heads, dim=dim, rot_dim=rot_dim, rank=rank,
+                         page_size=page_size, interleaved=interleaved, q=q, q_plain=plain, q_abs=q_abs)
+        self.headwise_linear(plain.view(n, heads, dim), w, q_abs.view(n, heads, rank + rot_dim)[:, :, :rank])
 
     def headwise_linear(self, x, w, out, row_scale=None):
         y = torch.einsum("nhk,hok->nho", x.float(), w.float())
@@ -231,7 +248,8 @@ class RefOps:
             else:
                 x = x + y
         if out is not None:
-            out.copy_((weight * (x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps))).to(out.dtype))
+            y = x if weight is None else weight * (x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps))
+            out.copy_(y.to(out.dtype))
 
     def silu_mul_bias(self, gate_up, bias, out):
         i = out.shape[1]
@@ -283,7 +301,8 @@ class RefOps:
                 m = m_new
             state[slot, m_offset: m_offset + heads] = m
 
-    def gated_recurrence(self, q, a, w, gates, v, state, slots, ctx, out, heads, dim, vdim, cols, q_scale):
+    def gated_recurrence(self, q, a, w, gates, v, state, slots, ctx, out, heads, dim, vdim, cols, q_scale,
+                         heads_per_unit=1):
         matrix = heads * cols * dim
         o = out.view(-1, heads, cols)
         for start, n, slot in zip(ctx.q_starts, ctx.q_lens, slots.tolist()):
@@ -291,7 +310,7 @@ class RefOps:
                 continue
             S = state[slot, :matrix].view(heads, cols, dim).transpose(1, 2).clone()  # [heads, dim, cols]
             for t in range(start, start + n):
-                qt, wt = q[t].view(heads, dim), w[t].view(heads, dim)
+                qt, wt = (r[t].view(heads // heads_per_unit, dim).repeat_interleave(heads_per_unit, 0) for r in (q, w))
                 u = v[t].view(heads, vdim)
                 if cols > vdim:
                     u = torch.cat([u, torch.ones(heads, 1)], dim=-1)
@@ -320,6 +339,32 @@ class RefOps:
                               heads, dim, vdim, vdim, dim ** -0.5)
         self.recurrence_readout(o, None, None, eps, proj[:, at_g: at_g + heads * vdim], out, heads, vdim, vdim,
                                 gate_act="silu")
+
+    def state_space(self, proj, ctx, conv_w, conv_b, dt_bias, A_log, skip, norm_w, norm_parts, eps, state, slots, out,
+                    heads, groups, dim, vdim, ws):
+        n, inner, (channels, taps) = proj.shape[0], heads * vdim, conv_w.shape
+        raw = proj[:, inner: inner + channels].float()
+        conv, tail_at = torch.zeros(n, channels), inner * dim
+        for start, count, slot in zip(ctx.q_starts, ctx.q_lens, slots.tolist()):
+            if count == 0:
+                continue
+            tail = state[slot, tail_at: tail_at + (taps - 1) * channels].view(taps - 1, channels)
+            seen = torch.cat([tail, raw[start: start + count]])
+            acc = conv_b + sum(seen[j: j + count] * conv_w[:, j] for j in range(taps))
+            conv[start: start + count] = torch.nn.functional.silu(acc)
+            tail.copy_(seen[seen.shape[0] - (taps - 1):].clone())
+        if out.dtype == torch.bfloat16:
+            conv = conv.to(out.dtype).float()
+        dt = torch.nn.functional.softplus(proj[:, inner + channels: inner + channels + heads].float() + dt_bias)
+        gates = torch.stack([torch.exp(-torch.exp(A_log) * dt), dt, torch.zeros_like(dt)], dim=-1)
+        y = torch.zeros(n, inner)
+        self.gated_recurrence(conv[:, inner + groups * dim:], None, conv[:, inner: inner + groups * dim],
+                              gates.reshape(n, 3 * heads), conv[:, :inner], state, slots, ctx, y, heads, dim, vdim, vdim,
+                              1.0, heads_per_unit=heads // groups)
+        y = y + skip.repeat_interleave(vdim) * conv[:, :inner]
+        y = (y * torch.nn.functional.silu(proj[:, :inner].float())).view(n, norm_parts, -1)
+        y = y * torch.rsqrt(y.pow(2).mean(-1, keepdim=True) + eps)
+        out.copy_((y.reshape(n, inner) * norm_w).to(out.dtype))
 
     def stream_mix_norm(self, h, streams, delta, mix, out_coef, read, weight, bias, alpha, eps, out, rows=None):
         x = (h if rows is None else h[rows.long()]).unflatten(1, (streams, -1))  # [n, S, width]
@@ -363,7 +408,7 @@ class RefOps:
     def qk_norm_rope_write(self, proj, positions, table, rot_dims, q_weight, k_weight, eps, q_out, k_cache,
                            v_cache, slot_mapping, heads, kv_heads, dim, vdim, page_size, bias=None,
                            value_norm=False, values_from_keys=False, interleaved=False, unit_norm=False,
-                           q_head_scale=None, warm_coef=0.0, warm_every=0):
+                           q_head_scale=None, warm_coef=0.0, warm_every=0, norm_over="head", value_scale=1.0):
         n = proj.shape[0]
         end = (heads + kv_heads) * dim + (0 if values_from_keys else kv_heads * vdim)
         proj = proj[:, :end].float()
@@ -372,7 +417,10 @@ class RefOps:
         q = proj[:, : heads * dim].reshape(n, heads, dim)
         k = proj[:, heads * dim: (heads + kv_heads) * dim].reshape(n, kv_heads, dim)
         v = k if values_from_keys else proj[:, (heads + kv_heads) * dim:].reshape(n, kv_heads, vdim)
-        if q_weight is not None:
+        if norm_over == "all":
+            q = q * torch.rsqrt(q.pow(2).mean((1, 2), keepdim=True) + eps) * q_weight.view(heads, dim)
+            k = k * torch.rsqrt(k.pow(2).mean((1, 2), keepdim=True) + eps) * k_weight.view(kv_heads, dim)
+        elif q_weight is not None:
             q = q * torch.rsqrt(q.pow(2).mean(-1, keepdim=True) + eps) * q_weight
             k = k * torch.rsqrt(k.pow(2).mean(-1, keepdim=True) + eps) * k_weight
         if unit_norm:
@@ -384,6 +432,7 @@ class RefOps:
             q = q * (1.0 + warm_coef * torch.log(((positions + 1) // warm_every + 1).float()))[:, None, None]
         if value_norm:
             v = v * torch.rsqrt(v.pow(2).mean(-1, keepdim=True) + eps)
+        v = v * value_scale
         if table is not None and rot_dims > 0:
             half = rot_dims // 2
             cos, sin = table[positions.long(), 0][:, None, :], table[positions.long(), 1][:, None, :]
@@ -512,7 +561,7 @@ class RefOps:
             v_cache[page, :, offset] = v.to(v_cache.dtype)
 
     def paged_attention(self, q, k_cache, v_cache, block_tables, ctx, nh, nkv, hd, page_size,
-                        scale, window, out, ragged=None, value_dim=None):
+                        scale, window, out, ragged=None, value_dim=None, sinks=None):
         vd = hd if value_dim is None else value_dim  # value rows: the first `vd` entries of v_cache's rows
         groups = nh // nkv
         tables = block_tables.long().cpu()
@@ -530,7 +579,9 @@ class RefOps:
             v = v.repeat_interleave(groups, dim=1)
             qt = q[t].reshape(nh, hd).float()
             scores = torch.einsum("hd,khd->hk", qt, k) * scale
-            probs = scores.softmax(-1)
+            if sinks is not None:
+                scores = torch.cat([scores, sinks[:, None]], dim=1)
+            probs = scores.softmax(-1)[:, : keys.numel()]
             out[t] = torch.einsum("hk,khd->hd", probs, v).reshape(nh * vd).to(out.dtype)
 
     def silu_mul(self, gate_up, out, interleave=0):
