@@ -784,6 +784,93 @@ def livitar_rows(size: str, kinds: dict, peaks: dict, tokens: int, batch: int, c
     return rows
 
 
+# --- the Kolisun design beside the closest models ------------------------------------------------
+
+KOLISUN_SIZES = {
+    # width, (latent: heads, dim, rot_dim, vdim, kv_rank, q_rank), (window attention: heads, kv_heads, dim, vdim,
+    # window), (recurrence: heads, vdim, state, groups, norm groups, taps), dense ff
+    "w1024": (1024, (8, 64, 32, 64, 256, 384), (16, 4, 64, 64, 512), (32, 64, 128, 2, 2, 4), 4096),
+    "w2048": (2048, (16, 128, 64, 128, 512, 768), (16, 4, 128, 128, 1024), (64, 64, 128, 4, 4, 4), 8192),
+}
+
+
+def kolisun_config(size: str) -> dict:
+    width, la, at, ss, ff = KOLISUN_SIZES[size]
+    latent = {"heads": la[0], "dim": la[1], "rot_dim": la[2], "vdim": la[3], "kv_rank": la[4], "q_rank": la[5],
+              "scale": (la[1] + la[2]) ** -0.5,
+              "rot": {"base": 10000.0, "dims": la[2],
+                      "scaling": {"factor": 16.0, "original": 4096, "fast": 24.0, "slow": 2.0}}}
+    left = {"heads": at[0], "kv_heads": at[1], "dim": at[2], "vdim": at[3], "scale": at[2] ** -0.5,
+            "mask": {"size": at[4]},
+            "rot": {"base": 500000.0, "dims": at[2],
+                    "scaling": {"factor": 4.0, "low": 1.5, "high": 5.0, "original": 4096}}}
+    right = {"heads": ss[0], "vdim": ss[1], "state": ss[2], "groups": ss[3], "norm_groups": ss[4], "conv": ss[5]}
+    both = {"left": left, "right": right, "left_scale": 0.8, "right_scale": 1.1}
+    dense = {"kind": "dense", "ff": ff}
+    return {"architecture": "Kolisun", "vocab": DESIGN_VOCAB, "width": width, "max_positions": MAX_CONTEXT,
+            "norm": {"eps": 1e-6},
+            "layers": [{"type": t, "mixer": m, "mlp": dense}
+                       for t, m in (("latent_attention", latent), ("parallel", both)) * 2]}
+
+
+def kolisun_rows(size: str, kinds: dict, peaks: dict, tokens: int, batch: int, ctx: float, decode: bool) -> dict:
+    """Per kind of kernel of the Kolisun model: microseconds per launch and, where the kind has such a
+    figure, what it is of the measured peak: decode launches against the copy rate for the bytes they
+    must read (weights, cached rows, state read and written), prompt launches against the burst bf16
+    rate for their flops (the recurrence in a prompt: four per state entry and token); the norms, the
+    convolution and the gated norm of a prompt against the copy rate."""
+    width, la, at, ss, ff = KOLISUN_SIZES[size]
+    H, dim, rot, vdim, kvr, qr = la
+    row, inner = kvr + rot, ss[0] * ss[1]
+    channels = inner + 2 * ss[3] * ss[2]
+    weights = {  # elements of the matrices a launch reads
+        "linear:latent.in": width * (qr + row), "linear:latent.uq": qr * H * (dim + rot),
+        "linear:mixer.delta": width * H * vdim,
+        "latent.headwise": H * kvr * (dim + vdim) // 2,  # (two launches per layer, averaged)
+        "linear:parallel.in": width * ((at[0] + at[1]) * at[2] + at[1] * at[3] + inner + channels + ss[0]),
+        "linear:parallel.delta": width * (at[0] * at[3] + inner),
+        "linear:ffn.gate_up": 2 * width * ff, "linear:ffn.delta": width * ff, "linear:head": width * DESIGN_VOCAB,
+    }
+    state = inner * ss[2]  # floats of a layer's state per request
+    seen = min(tokens, at[4])  # keys a prompt's query sees through the window, on average
+    seen = (seen * (seen + 1) / 2 + max(tokens - at[4], 0) * at[4]) / tokens
+    flops = {  # per prompt launch
+        "attention.latent": 2.0 * tokens * tokens / 2 * H * (row + kvr),
+        "latent.headwise": 2.0 * tokens * H * kvr * (dim + vdim) / 2,
+        "attention.sink": 2.0 * at[0] * (at[2] + at[3]) * tokens * seen,
+        "recurrent.state_space": 4.0 * tokens * state,
+    }
+    moved = {  # bytes a prompt launch moves
+        "norm": tokens * width * (2 * 4 + 4 + 2) * 8 / 9,
+        "recurrent.conv": tokens * channels * (4 + 2), "recurrent.out": tokens * inner * (4 + 2),
+    }
+    rows = {}
+    for kind, r in kinds.items():
+        us = r["ms"] / r["launches"] * 1e3
+        out = {"us": round(us, 2), "launches": r["launches"]}
+        nbytes = None
+        if decode:
+            if weights.get(kind):
+                nbytes = 2 * weights[kind]
+            elif kind == "attention.latent":
+                nbytes = batch * ctx * row * 2
+            elif kind == "attention.sink":
+                nbytes = batch * min(ctx, at[4]) * at[1] * (at[2] + at[3]) * 2
+            elif kind == "recurrent.state_space":
+                nbytes = batch * state * 4 * 2
+        else:
+            nbytes = moved.get(kind)
+            f = flops.get(kind) or (2.0 * tokens * weights[kind] if weights.get(kind) and kind != "linear:head" else None)
+            if f:
+                out.update(tflops=round(f / (us * 1e-6) / 1e12, 1),
+                           frac=round(f / (us * 1e-6) / 1e12 / peaks["bf16_tflops"], 4))
+        if nbytes:
+            out.update(gbs=round(nbytes / (us * 1e-6) / 1e9, 1),
+                       frac=round(nbytes / (us * 1e-6) / 1e9 / peaks["hbm_gbs"], 4))
+        rows[kind] = out
+    return rows
+
+
 def run_design(args) -> dict:
     """`--design rugedra`: prompt and decode throughput of the Rugedra design at layer sizes of a real
     model's (four layers: latent attention + dense, delta rule + experts, latent attention + experts,
@@ -798,7 +885,9 @@ def run_design(args) -> dict:
     beside its mixer) beside the Vofanex and the Llama model.  `--design livitar`: the Livitar design
     (retention, attention with a logarithmic and with a bucketed bias by distance, retention; every
     layer with experts beside a shared one, four residual streams) beside the Puposun, Vofanex and
-    Llama models."""
+    Llama models.  `--design kolisun`: the Kolisun design (latent attention and windowed attention beside
+    a state-space recurrence in turn, every layer with a dense feed-forward) beside the Rugedra, Livitar,
+    Vofanex and Llama models."""
     import torch
 
     from inference_engine_b200.engine.llm_engine import LLMEngine
@@ -825,6 +914,10 @@ def run_design(args) -> dict:
         elif args.design == "livitar":
             models = [("livitar", livitar_config(size)), ("puposun", puposun_config(size)),
                       ("vofanex", vofanex_config(size)), ("llama", llama_config_like(size))]
+        elif args.design == "kolisun":
+            models = [("kolisun", kolisun_config(size)), ("rugedra", rugedra_config(size)),
+                      ("livitar", livitar_config(size)), ("vofanex", vofanex_config(size)),
+                      ("llama", llama_config_like(size))]
         if args.only:
             models = [m for m in models if m[0] in args.only.split(",")]
         for name, cfg in models:
@@ -839,7 +932,10 @@ def run_design(args) -> dict:
                    "prefill_tokens_per_s": round(PREFILL_LEN / (prefill_ms / 1e3), 1), "prefill_ms": round(prefill_ms, 3),
                    # (the prompt step is launched eagerly: what its kernels take by themselves, without the host)
                    "prefill_kernels_ms": round(sum(r["ms"] for r in kinds_prefill.values()), 3)}
-            if name == "livitar":
+            if name == "kolisun":
+                row["kernels"] = {f"decode_b{batch}": kolisun_rows(size, kinds, peaks, batch, batch, ctx, True),
+                                  f"prefill_{PREFILL_LEN}": kolisun_rows(size, kinds_prefill, peaks, PREFILL_LEN, 1, PREFILL_LEN, False)}
+            elif name == "livitar":
                 row["kernels"] = {f"decode_b{batch}": livitar_rows(size, kinds, peaks, batch, batch, ctx, True),
                                   f"prefill_{PREFILL_LEN}": livitar_rows(size, kinds_prefill, peaks, PREFILL_LEN, 1, PREFILL_LEN, False)}
             elif name == "puposun":
@@ -982,7 +1078,7 @@ def main() -> int:
     ap.add_argument("--warmup", type=int, default=8)
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--design", default=None, choices=["rugedra", "ravapel", "vofanex", "puposun", "livitar"],
+    ap.add_argument("--design", default=None, choices=["rugedra", "ravapel", "vofanex", "puposun", "livitar", "kolisun"],
                     help="instead of the default workload: this design at real layer sizes beside the closest "
                          "model the engine had, prompt and decode throughput and every kind of kernel")
     ap.add_argument("--only", default=None, help="with --design: only these of its models (comma-separated)")

@@ -194,6 +194,117 @@ qk_wide_norm_rope_write_kernel(const float* __restrict__ proj, int ld, const int
         ie_store(v_cache + (first_row + (long long)g * page_size) * vdim + d, e * value_scale);
     }
 }
+
+// The same, four entries at a time (sizes and addresses allow it): a thread holds its pieces of the token's
+// columns in registers; norm weights and biases, which no kernel writes, are asked for before the wait.
+constexpr int WV_THREADS = 512, WV_PIECES = 4;
+
+__device__ __forceinline__ void store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) {
+    __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<unsigned*>(&lo), *reinterpret_cast<unsigned*>(&hi));
+}
+
+template <typename T>
+__global__ void __launch_bounds__(WV_THREADS)
+qk_wide_norm_rope_write4_kernel(const float* __restrict__ proj, int ld, const int* __restrict__ positions,
+                                const float* __restrict__ table, int rot_dims, int table_positions,
+                                const float* __restrict__ bias, int interleaved, const float* __restrict__ q_weight,
+                                const float* __restrict__ k_weight, float eps, float value_scale, T* __restrict__ q_out,
+                                T* __restrict__ k_cache, T* __restrict__ v_cache, const int* __restrict__ slot_mapping,
+                                int heads, int kv_heads, int dim, int vdim, int page_size, int total_pages, int* err) {
+    extern __shared__ __align__(16) float row[];  // halves: the normalised columns, for the pairs' other entries
+    __shared__ float red[2][WV_THREADS / 32];
+    ie_pdl_trigger();
+    const int n = blockIdx.x, tid = threadIdx.x, nq = heads * dim, nqk = (heads + kv_heads) * dim, all = nqk + kv_heads * vdim;
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    float4 w[WV_PIECES], e[WV_PIECES];
+#pragma unroll
+    for (int i = 0; i < WV_PIECES; ++i) {
+        int c = (i * WV_THREADS + tid) * 4;
+        w[i] = c < nq ? *reinterpret_cast<const float4*>(q_weight + c)
+             : c < nqk ? *reinterpret_cast<const float4*>(k_weight + c - nq) : zero;
+        e[i] = c < all && bias != nullptr ? *reinterpret_cast<const float4*>(bias + c) : zero;
+    }
+    ie_pdl_wait();
+    const float* src = proj + (size_t)n * ld;
+    const int pos = positions[n], half = rot_dims / 2;
+    const int slot = slot_mapping != nullptr ? slot_mapping[n] : -1;
+    float sq = 0.f, sk = 0.f;
+#pragma unroll
+    for (int i = 0; i < WV_PIECES; ++i) {
+        int c = (i * WV_THREADS + tid) * 4;
+        if (c >= all) break;
+        float4 x = *reinterpret_cast<const float4*>(src + c);
+        e[i].x += x.x; e[i].y += x.y; e[i].z += x.z; e[i].w += x.w;
+    }
+#pragma unroll
+    for (int i = 0; i < WV_PIECES; ++i) {
+        int c = (i * WV_THREADS + tid) * 4;
+        float s = fmaf(e[i].x, e[i].x, fmaf(e[i].y, e[i].y, fmaf(e[i].z, e[i].z, e[i].w * e[i].w)));
+        if (c < nq) sq += s;
+        else if (c < nqk) sk += s;
+    }
+    sq = warp_sum(sq);
+    sk = warp_sum(sk);
+    if ((tid & 31) == 0) { red[0][tid >> 5] = sq; red[1][tid >> 5] = sk; }
+    __syncthreads();
+    sq = sk = 0.f;
+#pragma unroll
+    for (int i = 0; i < WV_THREADS / 32; ++i) { sq += red[0][i]; sk += red[1][i]; }
+    const float inv_q = 1.0f / sqrtf(sq / (float)nq + eps), inv_k = 1.0f / sqrtf(sk / (float)(nqk - nq) + eps);
+#pragma unroll
+    for (int i = 0; i < WV_PIECES; ++i) {
+        int c = (i * WV_THREADS + tid) * 4;
+        if (c >= nqk) continue;
+        float inv = c < nq ? inv_q : inv_k;
+        e[i].x = (e[i].x * inv) * w[i].x; e[i].y = (e[i].y * inv) * w[i].y;
+        e[i].z = (e[i].z * inv) * w[i].z; e[i].w = (e[i].w * inv) * w[i].w;
+        if (!interleaved && rot_dims > 0) *reinterpret_cast<float4*>(row + c) = e[i];
+    }
+    if (half > 0 && (pos < 0 || pos >= table_positions)) {
+        if (tid == 0) ie_report(err, IE_ERR_POSITION, pos, n);
+        return;
+    }
+    int page = slot / page_size;
+    bool writes = slot_mapping != nullptr;
+    if (writes && (slot < 0 || page >= total_pages)) {
+        if (tid == 0) ie_report(err, IE_ERR_PAGE, slot, n);
+        writes = false;
+    }
+    if (!interleaved && rot_dims > 0) __syncthreads();
+    const float* cs = table + (size_t)max(pos, 0) * rot_dims;  // cos of the angles, then their sin
+    const long long first_row = (long long)page * kv_heads * page_size + (slot - page * page_size);
+#pragma unroll
+    for (int i = 0; i < WV_PIECES; ++i) {
+        int c = (i * WV_THREADS + tid) * 4;
+        if (c >= all || (c >= nq && !writes)) break;
+        float4 x = e[i];
+        if (c >= nqk) {
+            int g = (c - nqk) / vdim, d = c - nqk - g * vdim;
+            x.x *= value_scale; x.y *= value_scale; x.z *= value_scale; x.w *= value_scale;
+            store4(v_cache + (first_row + (long long)g * page_size) * vdim + d, x);
+            continue;
+        }
+        int unit = c / dim, d = c - unit * dim;
+        if (d < rot_dims) {
+            if (interleaved) {
+                float2 co = *reinterpret_cast<const float2*>(cs + (d >> 1)), si = *reinterpret_cast<const float2*>(cs + half + (d >> 1));
+                x = make_float4(x.x * co.x - x.y * si.x, x.y * co.x + x.x * si.x, x.z * co.y - x.w * si.y, x.w * co.y + x.z * si.y);
+            } else {
+                bool second = d >= half;
+                int j = second ? d - half : d;
+                float4 co = *reinterpret_cast<const float4*>(cs + j), si = *reinterpret_cast<const float4*>(cs + half + j);
+                float4 o = *reinterpret_cast<const float4*>(row + (second ? c - half : c + half));
+                float sg = second ? 1.f : -1.f;
+                x = make_float4(x.x * co.x + sg * (o.x * si.x), x.y * co.y + sg * (o.y * si.y),
+                                x.z * co.z + sg * (o.z * si.z), x.w * co.w + sg * (o.w * si.w));
+            }
+        }
+        if (c < nq) store4(q_out + (size_t)n * nq + c, x);
+        else store4(k_cache + (first_row + (long long)(unit - heads) * page_size) * dim + d, x);
+    }
+}
 }  // namespace
 
 IE_API int ie_qk_norm_rope_write(const float* proj, int ld, const int* positions, const float* table, int rot_dims,
@@ -235,6 +346,24 @@ IE_API int ie_qk_wide_norm_rope_write(const float* proj, int ld, const int* posi
     size_t smem = (size_t)(heads + kv_heads) * dim * sizeof(float);
     if (smem > 200 * 1024) return (int)cudaErrorInvalidValue;
     cudaStream_t s = (cudaStream_t)stream;
+    // (which of the two kernels runs depends on the sizes and on how the arrays lie, not on the step)
+    const int all = (heads + kv_heads) * dim + kv_heads * vdim;
+    const uintptr_t bits = reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(table) | reinterpret_cast<uintptr_t>(bias) |
+                           reinterpret_cast<uintptr_t>(q_weight) | reinterpret_cast<uintptr_t>(k_weight) |
+                           reinterpret_cast<uintptr_t>(q_out) | reinterpret_cast<uintptr_t>(k_cache) | reinterpret_cast<uintptr_t>(v_cache);
+    if (dim % 4 == 0 && vdim % 4 == 0 && ld % 4 == 0 && rot_dims % (interleaved ? 4 : 8) == 0 && bits % 16 == 0 &&
+        all <= 4 * WV_THREADS * WV_PIECES && smem <= 40 * 1024) {
+        size_t rows = interleaved ? 0 : smem;
+        if (dtype == IE_BF16)
+            return ie_launch(qk_wide_norm_rope_write4_kernel<__nv_bfloat16>, dim3(num_tokens), dim3(WV_THREADS), rows, s, proj,
+                             ld, positions, table, rot_dims, table_positions, bias, interleaved, q_weight, k_weight, eps,
+                             value_scale, (__nv_bfloat16*)q_out, (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache,
+                             slot_mapping, heads, kv_heads, dim, vdim, page_size, total_pages, err);
+        return ie_launch(qk_wide_norm_rope_write4_kernel<float>, dim3(num_tokens), dim3(WV_THREADS), rows, s, proj, ld,
+                         positions, table, rot_dims, table_positions, bias, interleaved, q_weight, k_weight, eps,
+                         value_scale, (float*)q_out, (float*)k_cache, (float*)v_cache, slot_mapping, heads, kv_heads, dim,
+                         vdim, page_size, total_pages, err);
+    }
 #define IE_WN_LAUNCH(T)                                                                                              \
     do {                                                                                                             \
         static IePerDevice allowed;                                                                                  \

@@ -285,6 +285,25 @@ conv_silu_kernel(const float* __restrict__ x, int x_ld, const float* __restrict_
             tail = state + (size_t)slot * state_stride + tail_at;
         }
         if (!live) continue;
+        if (TAPS > 0 && n == n0 && n1 - n0 == CS_TOKENS && n1 <= cu_q[seq + 1]) {
+            // a whole tile of one request: every input is on its way before the first is used
+            float in[CS_TOKENS + KEEP];
+#pragma unroll
+            for (int i = 0; i < CS_TOKENS; ++i) in[KEEP + i] = x[(size_t)(n0 + i) * x_ld + c];
+#pragma unroll
+            for (int i = 0; i < TAPS - 1; ++i) {
+                int back = TAPS - 1 - i;
+                in[i] = n0 - back >= first ? x[(size_t)(n0 - back) * x_ld + c] : tail[(size_t)(taps - 1 + n0 - first - back) * channels + c];
+            }
+#pragma unroll
+            for (int i = 0; i < CS_TOKENS; ++i) {
+                float acc = b;
+#pragma unroll
+                for (int j = 0; j < TAPS; ++j) acc = fmaf(wt[j], in[KEEP + i - (TAPS - 1) + j], acc);
+                ie_store(out + (size_t)(n0 + i) * out_ld + c, silu_f(acc));
+            }
+            return;
+        }
         const int t = n - first;
         auto earlier = [&](int back) {
             return t - back >= 0 ? x[(size_t)(n - back) * x_ld + c] : tail[(size_t)(taps - 1 + t - back) * channels + c];
@@ -308,32 +327,85 @@ conv_silu_kernel(const float* __restrict__ x, int x_ld, const float* __restrict_
     }
 }
 
-// grid: (tokens, parts).  y: [N, size] 32-bit; with `x` (the convolved values, [N, x_ld]) D[head] x is added, and
+// The slot's kept convolution inputs moved on by the step's tokens: the last taps - 1 of (kept, new).  A thread owns
+// a channel; every value is read before the first is written.
+__device__ __forceinline__ void move_kept_inputs(int seq, int c, const float* __restrict__ raw, int raw_ld,
+                                                 float* __restrict__ state, long long state_stride, long long tail_at,
+                                                 const int* __restrict__ slots, const int* __restrict__ cu_q, int channels,
+                                                 int taps, int num_slots) {
+    const int start = cu_q[seq], len = cu_q[seq + 1] - start, slot = slots[seq];
+    if (c >= channels || len <= 0 || slot < 0 || slot >= num_slots) return;
+    float* tail = state + (size_t)slot * state_stride + tail_at + c;
+    auto kept = [&](int j) {
+        int tt = len - (taps - 1) + j;
+        return tt >= 0 ? raw[(size_t)(start + tt) * raw_ld + c] : tail[(size_t)(taps - 1 + tt) * channels];
+    };
+    constexpr int MOST = 3;
+    if (taps - 1 <= MOST) {
+        float v[MOST];
+#pragma unroll
+        for (int j = 0; j < MOST; ++j)
+            if (j < taps - 1) v[j] = kept(j);
+#pragma unroll
+        for (int j = 0; j < MOST; ++j)
+            if (j < taps - 1) tail[(size_t)j * channels] = v[j];
+        return;
+    }
+    for (int j = 0; j < taps - 1; ++j) tail[(size_t)j * channels] = kept(j);  // (rising: read before it is overwritten)
+}
+
+// grid: tokens * parts, then the blocks that move the kept inputs (256 channels of a request each).  y: [N, size] 32-bit; with `x` (the convolved values, [N, x_ld]) D[head] x is added, and
 // with `z` ([N, z_ld] 32-bit) the sum is multiplied by silu(z); then each of the row's equal parts is divided by
-// its root mean square and multiplied by the weight.  The blocks of a request's last token also move its kept
-// convolution inputs on: channels [part's share] of `raw` ([N, raw_ld], 32-bit).
+// its root mean square and multiplied by the weight.  raw: the convolution's inputs, [N, raw_ld] 32-bit.
+// VEC: y alone (no x, no z), four entries at a time, a part of at most GN_THREADS * 16 entries.
 constexpr int GN_THREADS = 256;
-template <typename T>
+template <typename T, bool VEC>
 __global__ void __launch_bounds__(GN_THREADS)
 gated_group_norm_kernel(const float* __restrict__ y, const float* __restrict__ x, int x_ld, const float* __restrict__ skip,
                         const float* __restrict__ z, int z_ld, const float* __restrict__ weight, float eps,
-                        T* __restrict__ out, int out_ld, int size, int parts, int vdim,
+                        T* __restrict__ out, int out_ld, int num_tokens, int size, int parts, int vdim,
                         const float* __restrict__ raw, int raw_ld, float* __restrict__ state, long long state_stride,
-                        long long tail_at, const int* __restrict__ slots, const int* __restrict__ seq_of_token,
-                        const int* __restrict__ cu_q, int channels, int taps, int num_slots) {
-    extern __shared__ float part_buf[];  // [size / parts]
+                        long long tail_at, const int* __restrict__ slots, const int* __restrict__ cu_q, int channels,
+                        int taps, int num_slots) {
+    extern __shared__ __align__(16) float part_buf[];  // [size / parts]
     __shared__ float red[GN_THREADS / 32];
     ie_pdl_trigger();
-    ie_pdl_wait();
-    const int n = blockIdx.x, part = blockIdx.y, width = size / parts, at = part * width;
+    if ((int)blockIdx.x >= num_tokens * parts) {
+        ie_pdl_wait();
+        int i = blockIdx.x - num_tokens * parts, per = (channels + GN_THREADS - 1) / GN_THREADS;
+        move_kept_inputs(i / per, (i % per) * GN_THREADS + threadIdx.x, raw, raw_ld, state, state_stride, tail_at, slots, cu_q,
+                         channels, taps, num_slots);
+        return;
+    }
+    const int n = blockIdx.x / parts, part = blockIdx.x - n * parts, width = size / parts, at = part * width;
     const float* yr = y + (size_t)n * size + at;
+    constexpr int PIECES = 4;
+    float4 w4[PIECES], y4[PIECES];
     float ss = 0.f;
-    for (int i = threadIdx.x; i < width; i += GN_THREADS) {
-        float v = yr[i];
-        if (x != nullptr) v = fmaf(skip[(at + i) / vdim], x[(size_t)n * x_ld + at + i], v);
-        if (z != nullptr) v *= silu_f(z[(size_t)n * z_ld + at + i]);
-        part_buf[i] = v;
-        ss = fmaf(v, v, ss);
+    if constexpr (VEC) {
+#pragma unroll
+        for (int i = 0; i < PIECES; ++i) {  // (no kernel writes the weight)
+            int c = (i * GN_THREADS + threadIdx.x) * 4;
+            if (c < width) w4[i] = *reinterpret_cast<const float4*>(weight + at + c);
+        }
+        ie_pdl_wait();
+#pragma unroll
+        for (int i = 0; i < PIECES; ++i) {
+            int c = (i * GN_THREADS + threadIdx.x) * 4;
+            y4[i] = c < width ? *reinterpret_cast<const float4*>(yr + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+#pragma unroll
+        for (int i = 0; i < PIECES; ++i)
+            ss = fmaf(y4[i].x, y4[i].x, fmaf(y4[i].y, y4[i].y, fmaf(y4[i].z, y4[i].z, fmaf(y4[i].w, y4[i].w, ss))));
+    } else {
+        ie_pdl_wait();
+        for (int i = threadIdx.x; i < width; i += GN_THREADS) {
+            float v = yr[i];
+            if (x != nullptr) v = fmaf(skip[(at + i) / vdim], x[(size_t)n * x_ld + at + i], v);
+            if (z != nullptr) v *= silu_f(z[(size_t)n * z_ld + at + i]);
+            part_buf[i] = v;
+            ss = fmaf(v, v, ss);
+        }
     }
     ss = warp_sum(ss);
     if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
@@ -342,18 +414,23 @@ gated_group_norm_kernel(const float* __restrict__ y, const float* __restrict__ x
 #pragma unroll
     for (int w = 0; w < GN_THREADS / 32; ++w) total += red[w];
     const float inv = 1.0f / sqrtf(total / (float)width + eps);
-    for (int i = threadIdx.x; i < width; i += GN_THREADS)
-        ie_store(out + (size_t)n * out_ld + at + i, part_buf[i] * inv * weight[at + i]);
-    if (raw == nullptr || taps < 2) return;
-    const int seq = seq_of_token[n], start = cu_q[seq], end = cu_q[seq + 1], slot = slots[seq];
-    if (n != end - 1 || slot < 0 || slot >= num_slots) return;  // (a captured step's padding belongs to no request)
-    float* tail = state + (size_t)slot * state_stride + tail_at;
-    const int len = end - start, share = (channels + parts - 1) / parts;
-    for (int c = part * share + threadIdx.x; c < min(channels, (part + 1) * share); c += GN_THREADS)
-        for (int j = 0; j < taps - 1; ++j) {  // (rising: a kept row is read before it is overwritten)
-            int tt = len - (taps - 1) + j;
-            tail[(size_t)j * channels + c] = tt >= 0 ? raw[(size_t)(start + tt) * raw_ld + c] : tail[(size_t)(taps - 1 + tt) * channels + c];
+    T* dst = out + (size_t)n * out_ld + at;
+    if constexpr (VEC) {
+#pragma unroll
+        for (int i = 0; i < PIECES; ++i) {
+            int c = (i * GN_THREADS + threadIdx.x) * 4;
+            if (c >= width) break;
+            float4 v = make_float4(y4[i].x * inv * w4[i].x, y4[i].y * inv * w4[i].y, y4[i].z * inv * w4[i].z, y4[i].w * inv * w4[i].w);
+            if constexpr (sizeof(T) == 2) {
+                __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+                *reinterpret_cast<uint2*>(dst + c) = make_uint2(*reinterpret_cast<unsigned*>(&lo), *reinterpret_cast<unsigned*>(&hi));
+            } else {
+                *reinterpret_cast<float4*>(dst + c) = v;
+            }
         }
+    } else {
+        for (int i = threadIdx.x; i < width; i += GN_THREADS) ie_store(dst + i, part_buf[i] * inv * weight[at + i]);
+    }
 }
 
 constexpr int GR_THREADS = 128;
@@ -705,25 +782,34 @@ IE_API int ie_conv_silu(const float* x, int x_ld, const float* w, const float* b
 IE_API int ie_gated_group_norm(const float* y, const float* x, int x_ld, const float* skip, const float* z, int z_ld,
                                const float* weight, float eps, void* out, int out_ld, int out_dtype, int num_tokens,
                                int size, int parts, int vdim, const float* raw, int raw_ld, float* state,
-                               long long state_stride, long long tail_at, const int* slots, const int* seq_of_token,
-                               const int* cu_q, int channels, int taps, int num_slots, void* stream) {
+                               long long state_stride, long long tail_at, const int* slots, const int* cu_q, int num_seqs,
+                               int channels, int taps, int num_slots, void* stream) {
     if (num_tokens <= 0) return 0;
     if (parts < 1 || size % parts || vdim < 1 || out_ld < size) return (int)cudaErrorInvalidValue;
     size_t smem = (size_t)(size / parts) * sizeof(float);
     if (smem > 200 * 1024) return (int)cudaErrorInvalidValue;
     cudaStream_t s = (cudaStream_t)stream;
-#define IE_GG_LAUNCH(T)                                                                                              \
+    const int width = size / parts, mine = raw != nullptr && taps > 1 ? num_seqs * ((channels + GN_THREADS - 1) / GN_THREADS) : 0;
+    const bool vec = x == nullptr && z == nullptr && width % 4 == 0 && width <= GN_THREADS * 16 && out_ld % 4 == 0 &&
+                     ((reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(weight)) % 16 == 0) &&
+                     reinterpret_cast<uintptr_t>(out) % (out_dtype == IE_BF16 ? 8 : 16) == 0;
+#define IE_GG_LAUNCH(T, V)                                                                                           \
     do {                                                                                                             \
         static IePerDevice allowed;                                                                                  \
-        if (smem > 40 * 1024) {                                                                                      \
-            cudaError_t e = ie_allow_smem(allowed, gated_group_norm_kernel<T>, 200 * 1024);                          \
+        if (!V && smem > 40 * 1024) {                                                                                \
+            cudaError_t e = ie_allow_smem(allowed, gated_group_norm_kernel<T, V>, 200 * 1024);                       \
             if (e != cudaSuccess) return (int)e;                                                                     \
         }                                                                                                            \
-        return ie_launch(gated_group_norm_kernel<T>, dim3(num_tokens, parts), dim3(GN_THREADS), smem, s, y, x, x_ld, \
-                         skip, z, z_ld, weight, eps, (T*)out, out_ld, size, parts, vdim, raw, raw_ld, state,         \
-                         state_stride, tail_at, slots, seq_of_token, cu_q, channels, taps, num_slots);               \
+        return ie_launch(gated_group_norm_kernel<T, V>, dim3((unsigned)(num_tokens * parts + mine)),                 \
+                         dim3(GN_THREADS), V ? 0 : smem, s, y, x, x_ld, skip, z, z_ld, weight, eps, (T*)out, out_ld, \
+                         num_tokens, size, parts, vdim, raw, raw_ld, state, state_stride, tail_at, slots, cu_q,      \
+                         channels, taps, num_slots);                                                                 \
     } while (0)
-    if (out_dtype == IE_BF16) IE_GG_LAUNCH(__nv_bfloat16);
-    IE_GG_LAUNCH(float);
+    if (out_dtype == IE_BF16) {
+        if (vec) IE_GG_LAUNCH(__nv_bfloat16, true);
+        IE_GG_LAUNCH(__nv_bfloat16, false);
+    }
+    if (vec) IE_GG_LAUNCH(float, true);
+    IE_GG_LAUNCH(float, false);
 #undef IE_GG_LAUNCH
 }

@@ -21,8 +21,32 @@
 
 namespace {
 
+// A row of a 32-bit product that may have come back in parts (of a split inner dimension): added in order.
+struct Row {
+    const float* p;
+    int parts;
+    size_t stride;
+    __device__ __forceinline__ float operator[](int i) const {
+        float v = p[i];
+#pragma unroll 4
+        for (int s = 1; s < parts; ++s) v += p[s * stride + i];
+        return v;
+    }
+    __device__ __forceinline__ float4 four(int i) const {
+        float4 v = *reinterpret_cast<const float4*>(p + i);
+#pragma unroll 4
+        for (int s = 1; s < parts; ++s) {
+            float4 x = *reinterpret_cast<const float4*>(p + s * stride + i);
+            v.x += x.x; v.y += x.y; v.z += x.z; v.w += x.w;
+        }
+        return v;
+    }
+    __device__ __forceinline__ Row at(int i) const { return Row{p + i, parts, stride}; }
+};
+
 // entry d of a rotated part `src`, turned by the angles at `cs` (null: not turned)
-__device__ __forceinline__ float turned(const float* src, int d, const float* cs, int rot_dims, int interleaved) {
+template <typename Src>
+__device__ __forceinline__ float turned(const Src& src, int d, const float* cs, int rot_dims, int interleaved) {
     float v = src[d];
     if (cs == nullptr || d >= rot_dims) return v;
     int half = rot_dims / 2;
@@ -33,35 +57,33 @@ __device__ __forceinline__ float turned(const float* src, int d, const float* cs
     return fmaf(v, c, -src[interleaved ? d + 1 : d + half] * s);
 }
 
-__device__ __forceinline__ float rms_factor(const float* x, int size, float eps, float* red) {
-    float ss = 0.f;
-    for (int i = threadIdx.x; i < size; i += blockDim.x) ss = fmaf(x[i], x[i], ss);
-    ss = warp_sum(ss);
-    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
-    __syncthreads();
-    return 1.0f / sqrtf((red[0] + red[1] + red[2] + red[3]) / (float)size + eps);
-}
-
 // What a call asks for is what has a pointer: queries (q), gates (gate_pre), the cached row (dkv and
-// slot_mapping), the queries' latent (cq).  Each input is a row `*_ld` numbers long per token.
+// slot_mapping), the queries' latent (cq).  Each input is a row `*_ld` numbers long per token, in `parts` parts
+// `part_stride` apart.
 struct LatentIn {
     const float* q; int q_ld;
     const float* gate_pre; int gate_ld;
     const float* dkv; int dkv_ld;
     const float* cq; int cq_ld, q_rank;
+    int parts; size_t part_stride;
     const float* norm_w;
     const float* cq_norm_w;
     float eps;
+    bool fours;  // sizes and addresses of cq and dkv allow pieces of four
+    __device__ Row row(const float* p, int ld, int n) const { return Row{p + (size_t)n * ld, parts, part_stride}; }
 };
 
+constexpr int LP_THREADS = 256;
+
 template <typename T>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(LP_THREADS)
 latent_prep_kernel(LatentIn in, const int* __restrict__ positions,
                    const float* __restrict__ table, int rot_dims, int table_rows, int interleaved,
                    T* __restrict__ q_plain, T* __restrict__ q_abs, float* __restrict__ gate, T* __restrict__ cq_out,
                    T* __restrict__ cache, const int* __restrict__ slot_mapping, int heads, int dim, int rot_dim,
                    int rank, int total_slots, int* err) {
-    __shared__ float red[4], red_cq[4];
+    extern __shared__ __align__(16) float rows[];  // the queries' latent, then the cached row, as they come
+    __shared__ float red[2][LP_THREADS / 32];
     ie_pdl_trigger();
     ie_pdl_wait();
     int n = blockIdx.x, tid = threadIdx.x;
@@ -76,37 +98,63 @@ latent_prep_kernel(LatentIn in, const int* __restrict__ positions,
 
     if (in.q != nullptr) {
         // queries: unrotated parts as they are, rotated parts behind the latent part of the query rows
-        const float* row = in.q + (size_t)n * in.q_ld;
-        for (int i = tid; i < heads * dim; i += blockDim.x) {
+        const Row row = in.row(in.q, in.q_ld, n);
+        for (int i = tid; i < heads * dim; i += LP_THREADS) {
             int h = i / dim, d = i - h * dim;
             ie_store(q_plain + (size_t)n * heads * dim + i, row[h * hq + d]);
         }
-        for (int i = tid; i < heads * rot_dim; i += blockDim.x) {
+        for (int i = tid; i < heads * rot_dim; i += LP_THREADS) {
             int h = i / rot_dim, d = i - h * rot_dim;
-            ie_store(q_abs + ((size_t)n * heads + h) * krow + rank + d, turned(row + h * hq + dim, d, cs, rot_dims, interleaved));
+            ie_store(q_abs + ((size_t)n * heads + h) * krow + rank + d, turned(row.at(h * hq + dim), d, cs, rot_dims, interleaved));
         }
     }
     if (in.gate_pre != nullptr) {
-        const float* g = in.gate_pre + (size_t)n * in.gate_ld;
-        for (int h = tid; h < heads; h += blockDim.x) gate[(size_t)n * heads + h] = 1.0f / (1.0f + expf(-g[h]));
+        const Row g = in.row(in.gate_pre, in.gate_ld, n);
+        for (int h = tid; h < heads; h += LP_THREADS) gate[(size_t)n * heads + h] = 1.0f / (1.0f + expf(-g[h]));
     }
-    if (in.cq != nullptr) {
-        const float* src = in.cq + (size_t)n * in.cq_ld;
-        float inv = rms_factor(src, in.q_rank, in.eps, red_cq);
-        for (int i = tid; i < in.q_rank; i += blockDim.x)
-            ie_store(cq_out + (size_t)n * in.q_rank + i, src[i] * inv * in.cq_norm_w[i]);
-    }
-    if (in.dkv == nullptr || slot_mapping == nullptr) return;  // a run that borrows another layer's cache writes none
-    int slot = slot_mapping[n];
-    if (slot < 0 || slot >= total_slots) {
+    int slot = in.dkv != nullptr && slot_mapping != nullptr ? slot_mapping[n] : -1;
+    bool cached = in.dkv != nullptr && slot_mapping != nullptr;  // (a run that borrows another layer's cache writes none)
+    if (cached && (slot < 0 || slot >= total_slots)) {
         if (tid == 0) ie_report(err, IE_ERR_PAGE, slot, n);
-        return;
+        cached = false;
     }
-    const float* dkv = in.dkv + (size_t)n * in.dkv_ld;
-    float inv = rms_factor(dkv, rank, in.eps, red);
-    T* dst = cache + (size_t)slot * krow;
-    for (int i = tid; i < rank; i += blockDim.x) ie_store(dst + i, dkv[i] * inv * in.norm_w[i]);
-    for (int d = tid; d < rot_dim; d += blockDim.x) ie_store(dst + rank + d, turned(dkv + rank, d, cs, rot_dims, interleaved));
+    const int n_cq = in.cq != nullptr ? in.q_rank : 0, n_row = cached ? krow : 0;
+    if (n_cq + n_row == 0) return;
+    const Row cq = in.row(in.cq, in.cq_ld, n), dkv = in.row(in.dkv, in.dkv_ld, n);
+    float ss_q = 0.f, ss_c = 0.f;
+    if (in.fours) {
+#pragma unroll 2
+        for (int i = tid * 4; i < n_cq + n_row; i += LP_THREADS * 4) {
+            float4 v = i < n_cq ? cq.four(i) : dkv.four(i - n_cq);
+            *reinterpret_cast<float4*>(rows + i) = v;
+            float s = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, v.w * v.w)));
+            if (i < n_cq) ss_q += s;
+            else if (i - n_cq < rank) ss_c += s;
+        }
+    } else {
+        for (int i = tid; i < n_cq + n_row; i += LP_THREADS) {
+            float v = i < n_cq ? cq[i] : dkv[i - n_cq];
+            rows[i] = v;
+            if (i < n_cq) ss_q = fmaf(v, v, ss_q);
+            else if (i - n_cq < rank) ss_c = fmaf(v, v, ss_c);
+        }
+    }
+    ss_q = warp_sum(ss_q);
+    ss_c = warp_sum(ss_c);
+    if ((tid & 31) == 0) { red[0][tid >> 5] = ss_q; red[1][tid >> 5] = ss_c; }
+    __syncthreads();
+    ss_q = ss_c = 0.f;
+#pragma unroll
+    for (int w = 0; w < LP_THREADS / 32; ++w) { ss_q += red[0][w]; ss_c += red[1][w]; }
+    const float inv_q = n_cq > 0 ? 1.0f / sqrtf(ss_q / (float)n_cq + in.eps) : 0.f;
+    const float inv_c = 1.0f / sqrtf(ss_c / (float)rank + in.eps);
+    T* dst = cache + (size_t)max(slot, 0) * krow;
+    const float* part = rows + n_cq + rank;
+    for (int i = tid; i < n_cq + n_row; i += LP_THREADS) {
+        if (i < n_cq) ie_store(cq_out + (size_t)n * n_cq + i, rows[i] * inv_q * in.cq_norm_w[i]);
+        else if (i - n_cq < rank) ie_store(dst + i - n_cq, rows[i] * inv_c * in.norm_w[i - n_cq]);
+        else ie_store(dst + i - n_cq, turned(part, i - n_cq - rank, cs, rot_dims, interleaved));
+    }
 }
 
 // out[n, h, o] = scale[n, h] * sum_k x[n, h, k] * W[h, o, k], k ascending per output.
@@ -174,7 +222,7 @@ __global__ void scale_head_rows_kernel(__nv_bfloat16* __restrict__ out, long lon
 
 // The same products on the tensor cores (bfloat16 weights, K a multiple of 16): W's rows are the
 // instruction's 16 rows, tokens its columns.  XT float: x is the queries' 32-bit product (rounded to bfloat16
-// here), and the blocks of a head's first outputs also turn the rotated part that follows x in its row
+// here; in `x_parts` parts x_stride apart), and a head's last block turns the rotated part that follows x in its row
 // (`rot`).  A block of four warps takes either 64 outputs, a warp each sixteen (SPLIT false), or sixteen
 // outputs with K cut among its warps, whose sums are added in order (SPLIT true: long K, few outputs).
 // grid: (output blocks, heads, blocks of 8 * NT tokens).
@@ -196,7 +244,7 @@ template <typename XT, int NT, bool SPLIT>
 __global__ void __launch_bounds__(128)
 headwise_mma_kernel(const XT* __restrict__ x, long long x_ld, long long x_hs, const __nv_bfloat16* __restrict__ w,
                     __nv_bfloat16* __restrict__ out, long long o_ld, long long o_hs, const float* __restrict__ scale,
-                    RotatedPart rot, int N, int heads, int O, int K) {
+                    RotatedPart rot, int x_parts, long long x_stride, bool fours, int N, int heads, int O, int K) {
     extern __shared__ __align__(16) unsigned char raw[];
     __nv_bfloat16* xs = reinterpret_cast<__nv_bfloat16*>(raw);  // [8 * NT][K + 8]
     float* sums = reinterpret_cast<float*>(xs + 8 * NT * (K + 8));  // SPLIT: [4][16][8 * NT]
@@ -207,17 +255,7 @@ headwise_mma_kernel(const XT* __restrict__ x, long long x_ld, long long x_hs, co
     const int steps = K / 16, k_begin = SPLIT ? warp * steps / 4 : 0, k_end = SPLIT ? (warp + 1) * steps / 4 : steps;
     ie_pdl_wait();
     const int cnt = min(8 * NT, N - n0);
-    for (int i = tid; i < 8 * NT * (K / 4); i += 128) {
-        int r = i / (K / 4), c = (i - r * (K / 4)) * 4;
-        uint2 v = make_uint2(0u, 0u);
-        if (r < cnt) {
-            const XT* p = x + (size_t)(n0 + r) * x_ld + (size_t)h * x_hs + c;
-            __nv_bfloat162 lo = __floats2bfloat162_rn(ie_load(p), ie_load(p + 1)), hi = __floats2bfloat162_rn(ie_load(p + 2), ie_load(p + 3));
-            v = make_uint2(*reinterpret_cast<unsigned*>(&lo), *reinterpret_cast<unsigned*>(&hi));
-        }
-        *reinterpret_cast<uint2*>(xs + r * ld + c) = v;
-    }
-    if (rot.rot_dim > 0 && blockIdx.x == 0) {
+    if (rot.rot_dim > 0 && blockIdx.x + 1 == gridDim.x) {
         for (int i = tid; i < cnt * rot.rot_dim; i += 128) {
             int r = i / rot.rot_dim, d = i - r * rot.rot_dim, pos = rot.positions[n0 + r];
             bool turn = rot.table != nullptr && rot.rot_dims > 0;
@@ -228,9 +266,34 @@ headwise_mma_kernel(const XT* __restrict__ x, long long x_ld, long long x_hs, co
             const XT* p = x + (size_t)(n0 + r) * x_ld + (size_t)h * x_hs + rot.at;
             float v = 0.f;
             if constexpr (sizeof(XT) == 4)
-                v = turned(p, d, turn ? rot.table + (size_t)pos * rot.rot_dims : nullptr, rot.rot_dims, rot.interleaved);
+                v = turned(Row{p, x_parts, (size_t)x_stride}, d, turn ? rot.table + (size_t)pos * rot.rot_dims : nullptr, rot.rot_dims, rot.interleaved);
             out[(size_t)(n0 + r) * o_ld + (size_t)h * o_hs + rot.dst_at + d] = __float2bfloat16_rn(v);
         }
+        return;
+    }
+    for (int i = tid; i < 8 * NT * (K / 4); i += 128) {
+        int r = i / (K / 4), c = (i - r * (K / 4)) * 4;
+        uint2 v = make_uint2(0u, 0u);
+        if (r < cnt) {
+            const XT* p = x + (size_t)(n0 + r) * x_ld + (size_t)h * x_hs + c;
+            if constexpr (sizeof(XT) == 4) {
+                float4 f;
+                if (fours) {
+                    f = Row{p, x_parts, (size_t)x_stride}.four(0);
+                } else {
+                    const Row all{p, x_parts, (size_t)x_stride};
+                    f = make_float4(all[0], all[1], all[2], all[3]);
+                }
+                __nv_bfloat162 lo = __floats2bfloat162_rn(f.x, f.y), hi = __floats2bfloat162_rn(f.z, f.w);
+                v = make_uint2(*reinterpret_cast<unsigned*>(&lo), *reinterpret_cast<unsigned*>(&hi));
+            } else if (fours) {
+                v = *reinterpret_cast<const uint2*>(p);
+            } else {
+                __nv_bfloat162 lo = __halves2bfloat162(p[0], p[1]), hi = __halves2bfloat162(p[2], p[3]);
+                v = make_uint2(*reinterpret_cast<unsigned*>(&lo), *reinterpret_cast<unsigned*>(&hi));
+            }
+        }
+        *reinterpret_cast<uint2*>(xs + r * ld + c) = v;
     }
     __syncthreads();
     float c[NT][4];
@@ -284,20 +347,23 @@ headwise_mma_kernel(const XT* __restrict__ x, long long x_ld, long long x_hs, co
 
 template <typename XT, int NT, bool SPLIT>
 int launch_headwise_mma(const void* x, long long x_ld, long long x_hs, const void* w, void* out, long long o_ld,
-                        long long o_hs, const float* scale, RotatedPart rot, int N, int heads, int O, int K, cudaStream_t s) {
+                        long long o_hs, const float* scale, RotatedPart rot, int x_parts, long long x_stride, int N,
+                        int heads, int O, int K, cudaStream_t s) {
     size_t smem = (size_t)8 * NT * (K + 8) * 2 + (SPLIT ? (size_t)4 * 16 * 8 * NT * 4 : 0);
     static IePerDevice allowed;
     cudaError_t e = ie_allow_smem(allowed, headwise_mma_kernel<XT, NT, SPLIT>, 96 * 1024);
     if (e != cudaSuccess) return (int)e;
-    dim3 grid(SPLIT ? (O + 15) / 16 : (O + 63) / 64, heads, (N + 8 * NT - 1) / (8 * NT));
+    const bool fours = x_ld % 4 == 0 && x_hs % 4 == 0 && x_stride % 4 == 0 && reinterpret_cast<uintptr_t>(x) % (4 * sizeof(XT)) == 0;
+    dim3 grid((SPLIT ? (O + 15) / 16 : (O + 63) / 64) + (rot.rot_dim > 0 ? 1 : 0), heads, (N + 8 * NT - 1) / (8 * NT));
     return ie_launch(headwise_mma_kernel<XT, NT, SPLIT>, grid, dim3(128), smem, s, (const XT*)x, x_ld, x_hs,
-                     (const __nv_bfloat16*)w, (__nv_bfloat16*)out, o_ld, o_hs, scale, rot, N, heads, O, K);
+                     (const __nv_bfloat16*)w, (__nv_bfloat16*)out, o_ld, o_hs, scale, rot, x_parts, x_stride, fours, N, heads, O, K);
 }
 
 template <typename XT>
 int pick_headwise_mma(const void* x, long long x_ld, long long x_hs, const void* w, void* out, long long o_ld,
-                      long long o_hs, const float* scale, RotatedPart rot, int N, int heads, int O, int K, cudaStream_t s) {
-#define IE_HM_ARGS x, x_ld, x_hs, w, out, o_ld, o_hs, scale, rot, N, heads, O, K, s
+                      long long o_hs, const float* scale, RotatedPart rot, int x_parts, long long x_stride, int N,
+                        int heads, int O, int K, cudaStream_t s) {
+#define IE_HM_ARGS x, x_ld, x_hs, w, out, o_ld, o_hs, scale, rot, x_parts, x_stride, N, heads, O, K, s
     // (the cut must not change with the number of tokens: a token's sums depend on the sizes alone)
     bool split = K >= 256;
     if (N <= 8) return split ? launch_headwise_mma<XT, 1, true>(IE_HM_ARGS) : launch_headwise_mma<XT, 1, false>(IE_HM_ARGS);
@@ -314,7 +380,7 @@ IE_API int ie_scale_head_rows(void* out, long long o_ld, long long o_hs, const f
 }
 
 IE_API int ie_latent_prep(const float* q, int q_ld, const float* gate_pre, int gate_ld, const float* dkv, int dkv_ld,
-                          const float* cq, int cq_ld, int q_rank, const float* norm_w, const float* cq_norm_w, float eps,
+                          const float* cq, int cq_ld, int q_rank, int parts, long long part_stride, const float* norm_w, const float* cq_norm_w, float eps,
                           const int* positions, const float* table, int rot_dims, int table_rows, int interleaved,
                           void* q_plain, void* q_abs, float* gate, void* cq_out, void* cache, int dtype,
                           const int* slot_mapping, int num_tokens, int heads, int dim, int rot_dim, int rank,
@@ -322,13 +388,18 @@ IE_API int ie_latent_prep(const float* q, int q_ld, const float* gate_pre, int g
     if (num_tokens <= 0) return 0;
     if (rot_dims < 0 || rot_dims % 2 || rot_dims > rot_dim) return (int)cudaErrorInvalidValue;
     cudaStream_t s = (cudaStream_t)stream;
-    LatentIn in{q, q_ld, gate_pre, gate_ld, dkv, dkv_ld, cq, cq_ld, q_rank, norm_w, cq_norm_w, eps};
+    if (parts < 1) return (int)cudaErrorInvalidValue;
+    LatentIn in{q, q_ld, gate_pre, gate_ld, dkv, dkv_ld, cq, cq_ld, q_rank, parts, (size_t)part_stride, norm_w, cq_norm_w, eps, false};
+    in.fours = q_rank % 4 == 0 && rank % 4 == 0 && rot_dim % 4 == 0 && cq_ld % 4 == 0 && dkv_ld % 4 == 0 && part_stride % 4 == 0 &&
+               ((reinterpret_cast<uintptr_t>(cq) | reinterpret_cast<uintptr_t>(dkv)) % 16 == 0);
+    size_t smem = ((cq ? q_rank : 0) + (dkv ? rank + rot_dim : 0)) * sizeof(float);
+    if (smem > 40 * 1024) return (int)cudaErrorInvalidValue;
     if (dtype == IE_BF16)
-        return ie_launch(latent_prep_kernel<__nv_bfloat16>, dim3(num_tokens), dim3(128), 0, s, in, positions, table,
+        return ie_launch(latent_prep_kernel<__nv_bfloat16>, dim3(num_tokens), dim3(LP_THREADS), smem, s, in, positions, table,
                          rot_dims, table_rows, interleaved, (__nv_bfloat16*)q_plain, (__nv_bfloat16*)q_abs, gate,
                          (__nv_bfloat16*)cq_out, (__nv_bfloat16*)cache, slot_mapping, heads, dim, rot_dim, rank,
                          total_slots, err);
-    return ie_launch(latent_prep_kernel<float>, dim3(num_tokens), dim3(128), 0, s, in, positions, table, rot_dims,
+    return ie_launch(latent_prep_kernel<float>, dim3(num_tokens), dim3(LP_THREADS), smem, s, in, positions, table, rot_dims,
                      table_rows, interleaved, (float*)q_plain, (float*)q_abs, gate, (float*)cq_out, (float*)cache,
                      slot_mapping, heads, dim, rot_dim, rank, total_slots, err);
 }
@@ -339,16 +410,16 @@ IE_API int ie_headwise_mma_ok(int K) { return K % 16 == 0 && K >= 16 && K <= 102
 // x: bfloat16, or 32-bit (x_f32) with a rotated part of rot_dim entries that starts `rot_at` entries behind x.
 IE_API int ie_headwise_mma(const void* x, int x_f32, long long x_ld, long long x_hs, const void* w, void* out,
                            long long o_ld, long long o_hs, const float* scale, int N, int heads, int O, int K,
-                           const int* positions, const float* table, int rot_dims, int table_rows, int interleaved,
-                           int rot_dim, int rot_at, int rot_dst, int* err, void* stream) {
+                           int x_parts, long long x_stride, const int* positions, const float* table, int rot_dims,
+                           int table_rows, int interleaved, int rot_dim, int rot_at, int rot_dst, int* err, void* stream) {
     if (N <= 0 || heads <= 0 || O <= 0) return 0;
-    if (!ie_headwise_mma_ok(K) || (rot_dim > 0 && (!x_f32 || positions == nullptr)) || rot_dims < 0 || rot_dims % 2 ||
+    if (!ie_headwise_mma_ok(K) || x_parts < 1 || (rot_dim > 0 && (!x_f32 || positions == nullptr)) || rot_dims < 0 || rot_dims % 2 ||
         rot_dims > rot_dim || reinterpret_cast<uintptr_t>(w) % 8)
         return (int)cudaErrorInvalidValue;
     RotatedPart rot{positions, table, rot_dims, table_rows, interleaved, rot_dim, rot_at, rot_dst, err};
     cudaStream_t s = (cudaStream_t)stream;
-    if (x_f32) return pick_headwise_mma<float>(x, x_ld, x_hs, w, out, o_ld, o_hs, scale, rot, N, heads, O, K, s);
-    return pick_headwise_mma<__nv_bfloat16>(x, x_ld, x_hs, w, out, o_ld, o_hs, scale, rot, N, heads, O, K, s);
+    if (x_f32) return pick_headwise_mma<float>(x, x_ld, x_hs, w, out, o_ld, o_hs, scale, rot, x_parts, x_stride, N, heads, O, K, s);
+    return pick_headwise_mma<__nv_bfloat16>(x, x_ld, x_hs, w, out, o_ld, o_hs, scale, rot, x_parts, x_stride, N, heads, O, K, s);
 }
 
 IE_API int ie_headwise_linear(const void* x, long long x_ld, long long x_hs, const void* w, void* out,

@@ -23,6 +23,7 @@
 
 namespace {
 
+constexpr float LM_LOG2E = 1.4426950408889634f;  // scores, maxima and the parts' maxima are in units of log2 e
 constexpr int LM_MAX_DV = 512;  // value rows of up to this many entries (64 8-column slices dealt over the warps)
 
 __device__ __forceinline__ void cp_async16(void* dst, const void* src, int src_bytes) {
@@ -67,11 +68,11 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
     constexpr int LM_ROWS = 16 * MT, LM_KEYS = KEYS, LM_THREADS = LM_WARPS * 32;
     constexpr int LM_MAX_NT = LM_MAX_DV / 8 / LM_WARPS;  // 8-column slices of the output per warp
     constexpr int N_TILES = KEYS / 8;            // 8-key slices of a key tile
-    constexpr int WPN = LM_WARPS / N_TILES;      // warps that share a slice, each with MT / WPN row tiles
-    constexpr int MPW = MT / WPN;
+    constexpr int WPM = LM_WARPS / MT;           // warps that share sixteen rows, each with NPW slices of keys
+    constexpr int NPW = N_TILES / WPM;
     constexpr int TPR = LM_THREADS / LM_ROWS;    // softmax threads per row
     constexpr int KPT = KEYS / TPR;              // ... and keys per thread
-    static_assert(LM_WARPS % N_TILES == 0 && MT % WPN == 0 && MPW >= 1 && KPT % 4 == 0 && TPR <= 32, "shape");
+    static_assert(LM_WARPS % MT == 0 && N_TILES % WPM == 0 && (NPW == 1 || NPW == 2) && KPT % 4 == 0 && TPR <= 32, "shape");
     ie_pdl_trigger();
     ie_pdl_wait();
     // (the blocks of a request's last rows see the most keys: they start first)
@@ -143,7 +144,7 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
     }
     if (tid < LM_ROWS) {  // (cut contexts: the merge adds the sink's term)
         bool with_sink = sinks != nullptr && splits == 1 && tid < rows_here;
-        sm.m[tid] = with_sink ? sinks[(row0 + tid) % heads] : -INFINITY;
+        sm.m[tid] = with_sink ? sinks[(row0 + tid) % heads] * LM_LOG2E : -INFINITY;
         sm.l[tid] = with_sink ? 1.f : 0.f;
     }
 
@@ -160,53 +161,56 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
         __syncthreads();
         if (t + 1 < t_end) load_keys(t + 1, buf ^ 1);
         const __nv_bfloat16* ks = sm.k + (size_t)buf * LM_KEYS * ld;
-        // scores: this warp's eight keys against its row tiles
+        // scores: this warp's keys (eight, or sixteen with NPW 2) against its sixteen rows, even and odd steps of
+        // k in sums of their own
         {
-            int ns = warp % N_TILES, m_first = (warp / N_TILES) * MPW;
-            float c[MPW][4];
+            const int ns = (warp % WPM) * NPW, m_tile = warp / WPM;
+            float c[NPW][2][4];
 #pragma unroll
-            for (int i = 0; i < MPW; ++i) c[i][0] = c[i][1] = c[i][2] = c[i][3] = 0.f;
-            // fragments by ldmatrix: A (16 x 16 of Q) one x4; B (8 keys x 32 of k) one x4 for two steps
-            unsigned qa = (unsigned)__cvta_generic_to_shared(sm.q + (m_first * 16 + (lane & 15)) * ld + (lane >> 4) * 8);
-            unsigned kb = (unsigned)__cvta_generic_to_shared(ks + (ns * 8 + (lane & 7)) * ld + (lane >> 3) * 8);
+            for (int i = 0; i < NPW; ++i)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) c[i][0][e] = c[i][1][e] = 0.f;
+            // fragments by ldmatrix: A (16 x 16 of Q) one x4; B one x4: 8 keys x 32 of k, or 16 keys x 16
+            unsigned qa = (unsigned)__cvta_generic_to_shared(sm.q + (m_tile * 16 + (lane & 15)) * ld + (lane >> 4) * 8);
+            const int brow = NPW == 1 ? (lane & 7) : (lane & 7) + ((lane >> 4) << 3), bcol = NPW == 1 ? (lane >> 3) * 8 : ((lane >> 3) & 1) * 8;
+            unsigned kb = (unsigned)__cvta_generic_to_shared(ks + (ns * 8 + brow) * ld + bcol);
             int kk = 0;
+#pragma unroll 2
             for (; kk + 32 <= dkp; kk += 32) {
-                unsigned b[4];
-                asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-                             : "=r"(b[0]), "=r"(b[1]), "=r"(b[2]), "=r"(b[3]) : "r"(kb + kk * 2));
-                // (all fragments of the 32 columns first, then the products: a load's latency is paid
-                // once per 32 columns, not once per product)
-                unsigned a[MPW][2][4];
+                unsigned a[2][4], b[NPW][4];
 #pragma unroll
-                for (int i = 0; i < MPW; ++i)
+                for (int h = 0; h < 2; ++h)
+                    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+                                 : "=r"(a[h][0]), "=r"(a[h][1]), "=r"(a[h][2]), "=r"(a[h][3]) : "r"(qa + (kk + h * 16) * 2));
 #pragma unroll
-                    for (int h = 0; h < 2; ++h)
-                        asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-                                     : "=r"(a[i][h][0]), "=r"(a[i][h][1]), "=r"(a[i][h][2]), "=r"(a[i][h][3])
-                                     : "r"(qa + (i * 16 * ld + kk + h * 16) * 2));
+                for (int i = 0; i < NPW; ++i)
+                    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+                                 : "=r"(b[i][0]), "=r"(b[i][1]), "=r"(b[i][2]), "=r"(b[i][3]) : "r"(kb + (kk + i * 16) * 2));
 #pragma unroll
                 for (int h = 0; h < 2; ++h)
 #pragma unroll
-                    for (int i = 0; i < MPW; ++i) mma_bf16(c[i], a[i][h], b + 2 * h);
+                    for (int i = 0; i < NPW; ++i) mma_bf16(c[i][h], a[h], NPW == 1 ? b[0] + 2 * h : b[h % NPW] + 2 * i);
             }
             if (kk < dkp) {  // a last step of 16
-                unsigned b[2];
-                unsigned kb2 = (unsigned)__cvta_generic_to_shared(ks + (ns * 8 + (lane & 7)) * ld + ((lane >> 3) & 1) * 8);
-                asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];"
-                             : "=r"(b[0]), "=r"(b[1]) : "r"(kb2 + kk * 2));
-#pragma unroll
-                for (int i = 0; i < MPW; ++i) {
-                    unsigned a[4];
+                unsigned a[4], b[4];
+                asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+                             : "=r"(a[0]), "=r"(a[1]), "=r"(a[2]), "=r"(a[3]) : "r"(qa + kk * 2));
+                if (NPW == 1) {
+                    unsigned kb2 = (unsigned)__cvta_generic_to_shared(ks + (ns * 8 + (lane & 7)) * ld + ((lane >> 3) & 1) * 8);
+                    asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];" : "=r"(b[0]), "=r"(b[1]) : "r"(kb2 + kk * 2));
+                } else {
                     asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-                                 : "=r"(a[0]), "=r"(a[1]), "=r"(a[2]), "=r"(a[3]) : "r"(qa + (i * 16 * ld + kk) * 2));
-                    mma_bf16(c[i], a, b);
+                                 : "=r"(b[0]), "=r"(b[1]), "=r"(b[2]), "=r"(b[3]) : "r"(kb + kk * 2));
                 }
-            }
 #pragma unroll
-            for (int i = 0; i < MPW; ++i) {
-                float* s0 = sm.s + ((m_first + i) * 16 + g) * (LM_KEYS + 4) + ns * 8 + 2 * t4;
-                s0[0] = c[i][0] * scale; s0[1] = c[i][1] * scale;
-                s0[8 * (LM_KEYS + 4)] = c[i][2] * scale; s0[8 * (LM_KEYS + 4) + 1] = c[i][3] * scale;
+                for (int i = 0; i < NPW; ++i) mma_bf16(c[i][0], a, b + 2 * i);
+            }
+            const float sl2 = scale * LM_LOG2E;
+#pragma unroll
+            for (int i = 0; i < NPW; ++i) {
+                float* s0 = sm.s + (m_tile * 16 + g) * (LM_KEYS + 4) + (ns + i) * 8 + 2 * t4;
+                *reinterpret_cast<float2*>(s0) = make_float2((c[i][0][0] + c[i][1][0]) * sl2, (c[i][0][1] + c[i][1][1]) * sl2);
+                *reinterpret_cast<float2*>(s0 + 8 * (LM_KEYS + 4)) = make_float2((c[i][0][2] + c[i][1][2]) * sl2, (c[i][0][3] + c[i][1][3]) * sl2);
             }
         }
         __syncthreads();
@@ -231,7 +235,7 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
             __align__(8) __nv_bfloat16 pr[KPT];
 #pragma unroll
             for (int i = 0; i < KPT; ++i) {
-                float pv = (v[i] == -INFINITY) ? 0.f : expf(v[i] - m_new);
+                float pv = (v[i] == -INFINITY) ? 0.f : exp2f(v[i] - m_new);
                 pb[i] = __float2bfloat16_rn(pv);
                 pr[i] = __float2bfloat16_rn(pv - __bfloat162float(pb[i]));
                 sum += pv;
@@ -244,7 +248,7 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
                 *reinterpret_cast<uint2*>(sm.p + (LM_ROWS + r) * (LM_KEYS + 8) + j * KPT + i) = *reinterpret_cast<uint2*>(pr + i);
             }
             if (j == 0) {
-                float a = (m_old == -INFINITY) ? 0.f : expf(m_old - m_new);
+                float a = (m_old == -INFINITY) ? 0.f : exp2f(m_old - m_new);
                 if (m_new == -INFINITY) a = 1.f;
                 sm.alpha[r] = a;
                 sm.m[r] = m_new;
@@ -334,6 +338,7 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
     }
 }
 
+constexpr int LM_MAX_SPLITS = 32;
 // One block per (token, head) row: the ranges' parts added in order.
 __global__ void __launch_bounds__(128)
 latent_attention_merge_kernel(const float* __restrict__ scratch, __nv_bfloat16* __restrict__ out, int dv, int splits,
@@ -342,22 +347,39 @@ latent_attention_merge_kernel(const float* __restrict__ scratch, __nv_bfloat16* 
     ie_pdl_wait();
     size_t row = blockIdx.x;
     const float* base = scratch + row * splits * (dv + 2);
-    float sink = sinks != nullptr ? sinks[row % heads] : -INFINITY;
+    // the ranges' maxima and sums first, all at once (a range per thread), then the rows
+    __shared__ float s_m[LM_MAX_SPLITS], s_l[LM_MAX_SPLITS];
+    if ((int)threadIdx.x < splits) {
+        s_m[threadIdx.x] = base[(size_t)threadIdx.x * (dv + 2)];
+        s_l[threadIdx.x] = base[(size_t)threadIdx.x * (dv + 2) + 1];
+    }
+    const float sink = sinks != nullptr ? sinks[row % heads] * LM_LOG2E : -INFINITY;
+    __syncthreads();
     float m = sink;
-    for (int s = 0; s < splits; ++s) m = fmaxf(m, base[(size_t)s * (dv + 2)]);
-    float l = sinks != nullptr ? expf(sink - m) : 0.f;
+    for (int s = 0; s < splits; ++s) m = fmaxf(m, s_m[s]);
+    float l = sinks != nullptr ? exp2f(sink - m) : 0.f;
+    constexpr int PER = LM_MAX_DV / 128;
+    float o[PER];
+#pragma unroll
+    for (int i = 0; i < PER; ++i) o[i] = 0.f;
+#pragma unroll 4
     for (int s = 0; s < splits; ++s) {
-        float ms = base[(size_t)s * (dv + 2)];
-        if (ms != -INFINITY) l += base[(size_t)s * (dv + 2) + 1] * expf(ms - m);
+        const float* part = base + (size_t)s * (dv + 2) + 2;
+        const bool empty = s_m[s] == -INFINITY;  // (an empty range: its sums count for nothing)
+        const float w = empty ? 0.f : exp2f(s_m[s] - m);
+        l = fmaf(s_l[s], w, l);
+#pragma unroll
+        for (int i = 0; i < PER; ++i) {
+            int c = i * 128 + threadIdx.x;
+            float v = c < dv && !empty ? part[c] : 0.f;
+            o[i] = fmaf(v, w, o[i]);
+        }
     }
     float inv = l > 0.f ? 1.0f / l : 0.f;
-    for (int c = threadIdx.x; c < dv; c += blockDim.x) {
-        float o = 0.f;
-        for (int s = 0; s < splits; ++s) {
-            float ms = base[(size_t)s * (dv + 2)];
-            if (ms != -INFINITY) o = fmaf(base[(size_t)s * (dv + 2) + 2 + c], expf(ms - m), o);
-        }
-        out[row * dv + c] = __float2bfloat16_rn(o * inv);
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+        int c = i * 128 + threadIdx.x;
+        if (c < dv) out[row * dv + c] = __float2bfloat16_rn(o[i] * inv);
     }
 }
 
@@ -380,7 +402,7 @@ IE_API int ie_latent_attention_mma(const void* q, const void* cache, const int* 
                                    int num_seqs, int max_tiles, int rows, int heads, int dk, int dv, int page_size,
                                    int total_pages, float scale, const float* sinks, int splits, int* err, void* stream) {
     if (num_seqs <= 0 || max_tiles <= 0) return 0;
-    if (!ie_latent_attention_mma_ok(dk, dv) || splits < 1 || (splits > 1 && scratch == nullptr)) return (int)cudaErrorInvalidValue;
+    if (!ie_latent_attention_mma_ok(dk, dv) || splits < 1 || splits > LM_MAX_SPLITS || (splits > 1 && scratch == nullptr)) return (int)cudaErrorInvalidValue;
     if (rows != 16 && rows != 64) return (int)cudaErrorInvalidValue;
     cudaStream_t s = (cudaStream_t)stream;
     int rc;

@@ -934,7 +934,7 @@ class CudaOps:
             max_tiles = -(-longest * nh // rows)
             blocks = max_tiles * ctx.num_seqs
             table_tokens = block_tables.shape[1] * page_size
-            splits = max(1, min(self.sm_count // blocks, table_tokens // 128, 16))
+            splits = max(1, min(self.sm_count // blocks, table_tokens // 64, 32))
             scratch = None
             if splits > 1:
                 scratch = self._scratch(ctx, "attn.latent_partial", ctx.num_tokens * nh * splits * (value_dim + 2), q.device)
@@ -956,11 +956,11 @@ class CudaOps:
 
     _PART_SIGNATURES = {
         "latent": {
-            "ie_latent_prep": "P I P I P I P I I P P F P P I I I P P P P P I P I I I I I I P P",
+            "ie_latent_prep": "P I P I P I P I I I L P P F P P I I I P P P P P I P I I I I I I P P",
             "ie_headwise_linear": "P L L P P L L P I I I I I P",
             "ie_scale_head_rows": "P L L P I I I P",
             "ie_headwise_mma_ok": "I",
-            "ie_headwise_mma": "P I L L P P L L P I I I I P P I I I I I I P P",
+            "ie_headwise_mma": "P I L L P P L L P I I I I I L P P I I I I I I P P",
             "ie_latent_attention_mma_ok": "I I",
             "ie_latent_attention_mma": "P P P I P P P P I I I I I I I I I F P I P P",
             "ie_latent_attention_rows": "I",
@@ -983,7 +983,7 @@ class CudaOps:
             "ie_mlstm_gates": "P P I P P F P L L P P P I I I P",
             "ie_gated_recurrence": "P I P I P I P I P I P L P P P I I I I I I F I P",
             "ie_conv_silu": "P I P P P L L P P P P I I I I I I P P P P I P P",
-            "ie_gated_group_norm": "P P I P P I P F P I I I I I I P I P L L P P P I I I P",
+            "ie_gated_group_norm": "P P I P P I P F P I I I I I I P I P L L P P I I I I P",
             "ie_rotate_heads": "P I P P I I I I I P P",
             "ie_recurrence_readout": "P I P P I F P I I P I L I I P",
             "ie_lowrank_decay": "P I P P F P I I I P",
@@ -1020,21 +1020,26 @@ class CudaOps:
         32-bit views ``[N, columns]`` of products of the mixer's input.  ``q`` (``heads * (dim + rot_dim)`` columns):
         unrotated parts to ``q_plain``, rotated ones behind the latent parts of ``q_abs``; ``gate_pre`` (``heads``):
         sigmoids to ``gate``; ``dkv`` (``rank + rot_dim``): the row of ``cache`` (``[pages, 1, page_size, rank +
-        rot_dim]``), unless ``slot_mapping`` is None; ``cq``: the queries' own latent, normalised, to ``cq_out``."""
+        rot_dim]``), unless ``slot_mapping`` is None; ``cq``: the queries' own latent, normalised, to ``cq_out``.  The inputs of a call may all be parts ``[S, N,
+        columns]`` of one product (they are added in order)."""
         if table is not None and table.shape[2] * 2 != rot_dims:
             raise KernelError("rotary table does not match the rotated dims")
         n = positions.shape[0]
         for t, columns in ((q, heads * (dim + rot_dim)), (gate_pre, heads), (dkv, rank + rot_dim),
                            (cq, None if cq_out is None else cq_out.shape[1])):
-            if t is not None and (t.dtype != self.torch.float32 or t.stride(1) != 1 or tuple(t.shape) != (n, columns)):
+            if t is not None and (t.dtype != self.torch.float32 or t.stride(-1) != 1 or tuple(t.shape[-2:]) != (n, columns)):
                 raise KernelError("latent_prep reads 32-bit columns of the sizes' widths")
+        given = {self._partials(t) for t in (q, gate_pre, dkv, cq) if t is not None}
+        if len(given) != 1:
+            raise KernelError("latent_prep: the inputs of a call are columns of one product")
+        (parts, stride), = given
         if dkv is not None and cache.shape[-1] != rank + rot_dim:
             raise KernelError("latent_prep: the cache rows do not fit the sizes")
         out = next(t for t in (cq_out, q_abs, cache) if t is not None)
-        ld = lambda t: 0 if t is None else t.stride(0)  # noqa: E731
+        ld = lambda t: 0 if t is None else t.stride(-2)  # noqa: E731
         self._check(self._part_lib("latent").ie_latent_prep(
             self._ptr(q), ld(q), self._ptr(gate_pre), ld(gate_pre), self._ptr(dkv), ld(dkv), self._ptr(cq), ld(cq),
-            0 if cq is None else cq.shape[1], self._ptr(norm_w), self._ptr(cq_norm_w), eps, positions.data_ptr(),
+            0 if cq is None else cq.shape[-1], parts, stride, self._ptr(norm_w), self._ptr(cq_norm_w), eps, positions.data_ptr(),
             self._ptr(table), rot_dims, 0 if table is None else table.shape[0], 1 if interleaved else 0,
             self._ptr(q_plain), self._ptr(q_abs), self._ptr(gate), self._ptr(cq_out), self._ptr(cache), _dtype_code(out),
             self._ptr(slot_mapping), n, heads, dim, rot_dim, rank, 0 if cache is None else cache.shape[0] * page_size,
@@ -1044,10 +1049,10 @@ class CudaOps:
 
     def latent_queries(self, q, w, q_abs, positions, table, rot_dims, *, heads, dim, rot_dim, rank, page_size,
                        interleaved: bool = True, ws) -> None:
-        """From the queries' 32-bit product ``q`` (``[N, heads * (dim + rot_dim)]``) the rows the attention reads,
+        """From the queries' 32-bit product ``q`` (``[N, heads * (dim + rot_dim)]``, or parts of it ``[S, N, ...]``) the rows the attention reads,
         ``q_abs`` ``[N, heads * (rank + rot_dim)]``: per head ``w[head] @ (unrotated part)`` (``w``: ``[heads, rank,
         dim]``), then the rotated part turned by its position.  bfloat16 steps of few tokens: one launch."""
-        n = q.shape[0]
+        n = q.shape[-2]
         rows = q_abs.view(n, heads, rank + rot_dim)
         if (q_abs.dtype == self.torch.bfloat16 and 0 < n < self.HEADWISE_LIBRARY_ROWS and self.headwise_mma
                 and self._part_lib("latent").ie_headwise_mma_ok(dim)):
@@ -1060,14 +1065,14 @@ class CudaOps:
     @_kind("latent.headwise")
     def _latent_queries_mma(self, q, w, rows, positions, table, rot_dims, dim, rot_dim, rank, interleaved) -> None:
         n, heads, _ = rows.shape
-        if (q.dtype != self.torch.float32 or q.stride(1) != 1 or q.shape[1] != heads * (dim + rot_dim)
+        if (q.dtype != self.torch.float32 or q.stride(-1) != 1 or q.shape[-1] != heads * (dim + rot_dim)
                 or w.shape != (heads, rank, dim) or not w.is_contiguous() or w.dtype != rows.dtype):
             raise KernelError("latent_queries: shapes, strides or dtypes do not fit")
         if table is not None and table.shape[2] * 2 != rot_dims:
             raise KernelError("rotary table does not match the rotated dims")
         self._check(self._part_lib("latent").ie_headwise_mma(
-            q.data_ptr(), 1, q.stride(0), dim + rot_dim, w.data_ptr(), rows.data_ptr(), rows.stride(0), rows.stride(1),
-            None, n, heads, rank, dim, positions.data_ptr(), self._ptr(table), rot_dims,
+            q.data_ptr(), 1, q.stride(-2), dim + rot_dim, w.data_ptr(), rows.data_ptr(), rows.stride(0), rows.stride(1),
+            None, n, heads, rank, dim, *self._partials(q), positions.data_ptr(), self._ptr(table), rot_dims,
             0 if table is None else table.shape[0], 1 if interleaved else 0, rot_dim, dim, rank, self._err_ptr,
             self._stream()), "headwise_mma")
 
@@ -1094,7 +1099,7 @@ class CudaOps:
         if x.dtype == self.torch.bfloat16 and self.headwise_mma and lib.ie_headwise_mma_ok(k):
             self._check(lib.ie_headwise_mma(
                 x.data_ptr(), 0, x.stride(0), x.stride(1), w.data_ptr(), out.data_ptr(), out.stride(0), out.stride(1),
-                self._ptr(row_scale), n, heads, o, k, None, None, 0, 0, 0, 0, 0, 0, self._err_ptr, self._stream()),
+                self._ptr(row_scale), n, heads, o, k, 1, 0, None, None, 0, 0, 0, 0, 0, 0, self._err_ptr, self._stream()),
                 "headwise_mma")
             return
         self._check(lib.ie_headwise_linear(
@@ -1548,8 +1553,8 @@ class CudaOps:
             y.data_ptr(), self._ptr(x_skip), 0 if x_skip is None else x_skip.stride(0), skip.data_ptr(), self._ptr(z),
             0 if z is None else z.stride(0), norm_w.data_ptr(), eps, out.data_ptr(), out.stride(0), _dtype_code(out),
             y.shape[0], y.shape[1], parts, vdim, raw.data_ptr(), raw.stride(0), state.data_ptr(), state.stride(0), tail_at,
-            slots.data_ptr(), ctx.seq_of_token.data_ptr(), ctx.cu_q.data_ptr(), channels, taps, state.shape[0],
-            self._stream()), "gated_group_norm")
+            slots.data_ptr(), ctx.cu_q.data_ptr(), ctx.num_seqs, channels, taps, state.shape[0], self._stream()),
+            "gated_group_norm")
 
     @_kind("recurrent.gates")
     def lowrank_decay(self, y, w2, bias, tau: float, decay) -> None:

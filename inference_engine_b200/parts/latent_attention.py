@@ -111,22 +111,22 @@ class LatentAttention(Mixer):
         rot_dims = self.position.rotary_dim if self.position is not None else 0
         sizes = dict(heads=H, dim=self.dim, rot_dim=self.rot_dim, rank=self.kv_rank, page_size=group.page_size,
                      interleaved=self.interleaved)
-        proj = ops.linear(x, self.w_in, ws=ws, tag="latent.in", out_dtype=torch.float32)
+        proj = ops.linear(x, self.w_in, ws=ws, tag="latent.in", out_dtype=torch.float32, allow_split=True)
         at = self.q_size if self.q_rank is None else self.q_rank  # where the latent's columns start
         gate = cq = None
         extra = {}
         if "gate" in self.names:
             gate = ws.buffer("latent.gate", n, H, torch.float32)
-            extra.update(gate_pre=proj[:, at + self.row: at + self.row + H], gate=gate)
+            extra.update(gate_pre=proj[..., at + self.row: at + self.row + H], gate=gate)
         if self.q_rank is not None:
             cq = ws.buffer("latent.cq", n, self.q_rank, self.dtype)
-            extra.update(cq=proj[:, : self.q_rank], cq_norm_w=self.q_norm, cq_out=cq)
-        ops.latent_prep(ctx.positions, table, rot_dims, **sizes, eps=self.eps, dkv=proj[:, at: at + self.row],
+            extra.update(cq=proj[..., : self.q_rank], cq_norm_w=self.q_norm, cq_out=cq)
+        ops.latent_prep(ctx.positions, table, rot_dims, **sizes, eps=self.eps, dkv=proj[..., at: at + self.row],
                         norm_w=self.latent_norm, cache=cache,
                         slot_mapping=group.slot_mapping if binding.writes else None, **extra)
-        q = proj[:, : self.q_size]
+        q = proj[..., : self.q_size]
         if cq is not None:
-            q = ops.linear(cq, self.w_uq, ws=ws, tag="latent.uq", out_dtype=torch.float32)
+            q = ops.linear(cq, self.w_uq, ws=ws, tag="latent.uq", out_dtype=torch.float32, allow_split=True)
         q_abs = ws.buffer("latent.q", n, H * self.row, self.dtype)
         ops.latent_queries(q, self.w_uk_t, q_abs, ctx.positions, table, rot_dims, **sizes, ws=ws)
         mixed = ws.buffer("latent.mixed", n, H * self.kv_rank, self.dtype)
