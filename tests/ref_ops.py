@@ -78,6 +78,8 @@ class RefOps:
 
         n = positions.shape[0]
         row = rank + rot_dim
+        # (the parts of a split product)
+        q, gate_pre, dkv, cq = (t.sum(0) if t is not None and t.dim() == 3 else t for t in (q, gate_pre, dkv, cq))
         if q is not None:
             q = q.reshape(n, heads, dim + rot_dim).float()
             q_plain.copy_(q[..., :dim].reshape(n, heads * dim).to(q_plain.dtype))
@@ -95,7 +97,7 @@ class RefOps:
 
     def latent_queries(self, q, w, q_abs, positions, table, rot_dims, *, heads, dim, rot_dim, rank, page_size,
                        interleaved=True, ws):
-        n = q.shape[0]
+        n = q.shape[-2]
         plain = torch.empty(n, heads * dim, dtype=q_abs.dtype)
         self.latent_prep(positions, table, rot_dims, heads=heads, dim=dim, rot_dim=rot_dim, rank=rank,
                          page_size=page_size, interleaved=interleaved, q=q, q_plain=plain, q_abs=q_abs)
@@ -353,7 +355,7 @@ class RefOps:
             acc = conv_b + sum(seen[j: j + count] * conv_w[:, j] for j in range(taps))
             conv[start: start + count] = torch.nn.functional.silu(acc)
             tail.copy_(seen[seen.shape[0] - (taps - 1):].clone())
-        if out.dtype == torch.bfloat16:
+        if out.dtype == torch.bfloat16 and max(dim, vdim) <= 128:  # (the fused kernels' sizes)
             conv = conv.to(out.dtype).float()
         dt = torch.nn.functional.softplus(proj[:, inner + channels: inner + channels + heads].float() + dt_bias)
         gates = torch.stack([torch.exp(-torch.exp(A_log) * dt), dt, torch.zeros_like(dt)], dim=-1)
