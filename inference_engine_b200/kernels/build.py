@@ -184,6 +184,23 @@ def build_retention(dim: int, vdim: int) -> Path:
     return build_library(f"ie_b200_retention_d{d}_v{dv}", ["retention.cu"], [f"-DRT_D={d}", f"-DRT_DV={dv}"])
 
 
+def latent_attention_fits(dk: int, dv: int) -> bool:
+    """Whether the tensor-core attention over shared latent rows takes key rows of ``dk`` and value rows of ``dv``
+    entries (its tiles of queries and keys must fit a block's shared memory)."""
+    ld = -(-dk // 16) * 16 + 8
+    most = max((rows + 2 * keys) * ld * 2 + rows * (keys + 4) * 4 + 2 * rows * (keys + 8) * 2 + 3 * rows * 4
+               for rows, keys in ((16, 64), (64, 32)))
+    return dk % 8 == 0 and dv % 8 == 0 and 8 <= dv <= min(dk, 512) and most <= 220 * 1024
+
+
+def build_latent_attention(dk: int, dv: int) -> Path:
+    """The tensor-core attention over shared latent rows for one pair of row sizes (compiled on first use for
+    the sizes the loaded model has)."""
+    if not latent_attention_fits(dk, dv):
+        raise BuildError(f"the tensor-core latent attention does not take rows of {dk} and {dv} entries")
+    return build_library(f"ie_b200_latentattn_k{dk}_v{dv}", ["latent_attention_mma.cu"], [f"-DLM_DK={dk}", f"-DLM_DV={dv}"])
+
+
 def build_state_space(state: int, vdim: int) -> Path:
     """The bfloat16 path's state-space kernels for one pair of state and value sizes, each rounded up to a
     multiple of 16 (compiled on first use for the sizes the loaded model has)."""
@@ -196,8 +213,8 @@ def build_state_space(state: int, vdim: int) -> Path:
 # Kernels only some mixers and feed-forwards need, each a library of its own that is built the
 # first time a model with such a part runs: name -> sources.
 PART_LIBRARIES = {
-    # the latent attention's input stage and per-head products, and its tensor-core attention
-    "latent": ["latent_attention.cu", "latent_attention_mma.cu"],
+    # the latent attention's input stage and per-head products
+    "latent": ["latent_attention.cu"],
     "delta": ["delta_rule.cu"],  # the gated delta rule: convolutions, the recurrence, the read-out norm
     "routed": ["routed_experts.cu"],  # routing and the grouped products of the routed feed-forward
     # recurrent mixers with a decaying matrix state (gated-write linear attention, exponential-gate
@@ -225,7 +242,7 @@ def build_all(prune: bool = True) -> list[Path]:
         libs += list(pool.map(build_part_library, PART_LIBRARIES))
         libs += [build_sigmoid_attention(64, 64), build_sink_attention(64, 64),
                  build_sink_attention(64, 64, "log"), build_sink_attention(64, 64, "table"),
-                 build_retention(64, 64), build_state_space(64, 64)]
+                 build_retention(64, 64), build_state_space(64, 64), build_latent_attention(320, 256)]
     if prune:
         keep = {lib.name for lib in libs}
         for old in build_dir().glob("libie_b200_*.so"):

@@ -17,8 +17,9 @@ import functools
 import os
 from ctypes import c_float, c_int, c_void_p
 
-from .build import (ATTENTION_HEAD_DIMS, build_attention, build_core, build_part_library,
-                    build_retention, build_sigmoid_attention, build_sink_attention, build_state_space)
+from .build import (ATTENTION_HEAD_DIMS, build_attention, build_core, build_latent_attention, build_part_library,
+                    build_retention, build_sigmoid_attention, build_sink_attention, build_state_space,
+                    latent_attention_fits)
 
 _ERRORS = {
     1: "a token id outside the vocabulary",
@@ -138,6 +139,7 @@ class CudaOps:
         self._part_libs: dict[str, object] = {}
         self._sigattn_libs: dict[tuple[int, int], object] = {}
         self._retention_libs: dict[tuple[int, int], object] = {}
+        self._latentattn_libs: dict[tuple[int, int], object] = {}
         self._state_space_libs: dict[tuple[int, int], object] = {}
         self.state_space_fused = os.environ.get("IE_B200_STATE_SPACE", "1") != "0"  # the state-space kernels of the bfloat16 path
         self.retention_fused = os.environ.get("IE_B200_RETENTION", "1") != "0"  # the retention kernels of the bfloat16 path
@@ -912,6 +914,20 @@ class CudaOps:
             k_cache.shape[0], scale, window, 0, None, None, None, 0, 0.0, 0, *self._NO_BIAS, nh * hd, self._err_ptr,
             self._stream()), "paged_attention")
 
+    def _latent_attention_lib(self, dk: int, dv: int):
+        lib = self._latentattn_libs.get((dk, dv))
+        if lib is None:
+            path = build_latent_attention(dk, dv)
+            try:
+                lib = ctypes.CDLL(str(path))
+            except OSError as exc:
+                raise KernelError(f"the kernel library {path} could not be loaded: {exc}") from exc
+            P, I, F = c_void_p, c_int, c_float
+            lib.ie_latent_attention_mma.argtypes = [P, P, P, I, P, P, P, P, I, I, I, I, I, I, I, F, P, I, P, P]
+            lib.ie_latent_attention_mma.restype = c_int
+            self._latentattn_libs[(dk, dv)] = lib
+        return lib
+
     @_kind("attention.latent")
     def latent_paged_attention(self, q, k_cache, v_cache, block_tables, ctx, nh, nkv, hd, value_dim,
                                page_size, scale, window, out, sinks=None) -> None:
@@ -923,11 +939,11 @@ class CudaOps:
         if not 0 < value_dim <= 512:
             raise KernelError(f"value rows of {value_dim} entries are not supported (1 to 512)")
         if (q.dtype == self.torch.bfloat16 and nkv == 1 and window == 0 and v_cache is k_cache
-                and self.latent_mma and self._part_lib("latent").ie_latent_attention_mma_ok(hd, value_dim)):
+                and self.latent_mma and latent_attention_fits(hd, value_dim) and page_size & (page_size - 1) == 0):
             # one shared row per token, values inside the key rows: the tensor-core kernel; a context is
             # cut into ranges of key tiles while the blocks are few (from the batch and the tables'
             # width alone, so that a captured launch stays valid)
-            lib = self._part_lib("latent")
+            lib = self._latent_attention_lib(hd, value_dim)
             bounds = getattr(ctx, "bounds", None)
             longest = bounds[0] if bounds is not None else ctx.max_q_len
             rows = lib.ie_latent_attention_rows(longest * nh)
@@ -941,7 +957,7 @@ class CudaOps:
             self._check(lib.ie_latent_attention_mma(
                 q.data_ptr(), k_cache.data_ptr(), block_tables.data_ptr(), block_tables.shape[1], ctx.cu_q.data_ptr(),
                 ctx.ctx_lens.data_ptr(), out.data_ptr(), self._ptr(scratch), ctx.num_tokens, ctx.num_seqs, max_tiles,
-                rows, nh, hd, value_dim, page_size, k_cache.shape[0], scale, self._ptr(sinks), splits, self._err_ptr,
+                rows, nh, page_size, k_cache.shape[0], scale, self._ptr(sinks), splits, self._err_ptr,
                 self._stream()),
                 "latent_attention_mma")
             return
@@ -961,9 +977,6 @@ class CudaOps:
             "ie_scale_head_rows": "P L L P I I I P",
             "ie_headwise_mma_ok": "I",
             "ie_headwise_mma": "P I L L P P L L P I I I I I L P P I I I I I I P P",
-            "ie_latent_attention_mma_ok": "I I",
-            "ie_latent_attention_mma": "P P P I P P P P I I I I I I I I I F P I P P",
-            "ie_latent_attention_rows": "I",
         },
         "delta": {
             "ie_delta_prep": "P I P P P P P L P P P P P P P P I I I I I I I I P P",

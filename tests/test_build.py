@@ -43,3 +43,25 @@ def test_part_libraries_export_what_is_declared():
     d, dv = ctypes.c_int(), ctypes.c_int()
     lib.ie_sigmoid_attention_dims(ctypes.byref(d), ctypes.byref(dv))
     assert (d.value, dv.value) == (32, 48) and hasattr(lib, "ie_sigmoid_attention_mma")
+
+
+@pytest.mark.skipif(shutil.which("nvcc") is None, reason="no CUDA compiler")
+def test_libraries_built_for_a_models_sizes():
+    """The state-space recurrence and the latent attention, each for one pair of sizes."""
+    from inference_engine_b200.kernels.build import (BuildError, build_latent_attention, build_state_space,
+                                                     latent_attention_fits)
+
+    a, b = ctypes.c_int(), ctypes.c_int()
+    lib = ctypes.CDLL(str(build_state_space(20, 33)))
+    assert lib.ie_state_space_dims(ctypes.byref(a), ctypes.byref(b)) == 64 and (a.value, b.value) == (32, 48)
+    assert hasattr(lib, "ie_state_space_step") and hasattr(lib, "ie_state_space_chunks")
+    with pytest.raises(BuildError, match="128"):
+        build_state_space(16, 129)
+    lib = ctypes.CDLL(str(build_latent_attention(40, 24)))
+    assert lib.ie_latent_attention_dims(ctypes.byref(a), ctypes.byref(b)) == 1 and (a.value, b.value) == (40, 24)
+    assert hasattr(lib, "ie_latent_attention_mma") and hasattr(lib, "ie_latent_attention_rows")
+    for dk, dv, fits in ((576, 512, True), (640, 512, True), (28, 24, False), (40, 20, False), (24, 32, False), (1024, 520, False),
+                         (1024, 512, False)):
+        assert latent_attention_fits(dk, dv) == fits, (dk, dv)
+    with pytest.raises(BuildError, match="28"):
+        build_latent_attention(28, 20)
