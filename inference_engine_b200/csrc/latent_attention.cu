@@ -34,7 +34,7 @@ struct Row {
     }
     __device__ __forceinline__ float4 four(int i) const {
         float4 v = *reinterpret_cast<const float4*>(p + i);
-#pragma unroll 4
+#pragma unroll 8
         for (int s = 1; s < parts; ++s) {
             float4 x = *reinterpret_cast<const float4*>(p + s * stride + i);
             v.x += x.x; v.y += x.y; v.z += x.z; v.w += x.w;
@@ -253,6 +253,19 @@ headwise_mma_kernel(const XT* __restrict__ x, long long x_ld, long long x_hs, co
     const int g = lane >> 2, t4 = lane & 3, ld = K + 8;
     const int o0 = SPLIT ? blockIdx.x * 16 : (blockIdx.x * 4 + warp) * 16;
     const int steps = K / 16, k_begin = SPLIT ? warp * steps / 4 : 0, k_end = SPLIT ? (warp + 1) * steps / 4 : steps;
+    // A thread's four consecutive entries of a row are the instruction's columns 2 t4, 2 t4 + 1 and 2 t4 + 8, 2 t4 + 9:
+    // the same renaming of k for both operands.  The first steps' weights, which no kernel writes, are asked for
+    // before the wait.
+    const __nv_bfloat16* wa = w + ((size_t)h * O + (o0 + g < O ? o0 + g : 0)) * K + t4 * 4;
+    const __nv_bfloat16* wb = w + ((size_t)h * O + (o0 + g + 8 < O ? o0 + g + 8 : 0)) * K + t4 * 4;
+    constexpr int EARLY = 8;
+    uint2 ra[EARLY], rb[EARLY];
+#pragma unroll
+    for (int i = 0; i < EARLY; ++i)
+        if (k_begin + i < k_end) {
+            ra[i] = *reinterpret_cast<const uint2*>(wa + (k_begin + i) * 16);
+            rb[i] = *reinterpret_cast<const uint2*>(wb + (k_begin + i) * 16);
+        }
     ie_pdl_wait();
     const int cnt = min(8 * NT, N - n0);
     if (rot.rot_dim > 0 && blockIdx.x + 1 == gridDim.x) {
@@ -300,21 +313,20 @@ headwise_mma_kernel(const XT* __restrict__ x, long long x_ld, long long x_hs, co
 #pragma unroll
     for (int t = 0; t < NT; ++t) c[t][0] = c[t][1] = c[t][2] = c[t][3] = 0.f;
     if (o0 < O) {
-        // a thread's four consecutive entries of a row are the instruction's columns 2 t4, 2 t4 + 1 and 2 t4 + 8,
-        // 2 t4 + 9: the same renaming of k for both operands
-        const bool in_a = o0 + g < O, in_b = o0 + g + 8 < O;
-        const __nv_bfloat16* wa = w + ((size_t)h * O + (in_a ? o0 + g : 0)) * K + t4 * 4;
-        const __nv_bfloat16* wb = w + ((size_t)h * O + (in_b ? o0 + g + 8 : 0)) * K + t4 * 4;
-#pragma unroll 8
-        for (int kk = k_begin; kk < k_end; ++kk) {
-            uint2 ra = *reinterpret_cast<const uint2*>(wa + kk * 16), rb = *reinterpret_cast<const uint2*>(wb + kk * 16);
-            unsigned a[4] = {ra.x, rb.x, ra.y, rb.y};
+        auto step = [&](int kk, uint2 pa, uint2 pb) {
+            unsigned a[4] = {pa.x, pb.x, pa.y, pb.y};
 #pragma unroll
             for (int t = 0; t < NT; ++t) {
                 uint2 b = *reinterpret_cast<const uint2*>(xs + (t * 8 + g) * ld + kk * 16 + t4 * 4);
                 mma_m16n8k16(c[t], a, b.x, b.y);
             }
-        }
+        };
+#pragma unroll
+        for (int i = 0; i < EARLY; ++i)
+            if (k_begin + i < k_end) step(k_begin + i, ra[i], rb[i]);
+#pragma unroll 8
+        for (int kk = k_begin + EARLY; kk < k_end; ++kk)
+            step(kk, *reinterpret_cast<const uint2*>(wa + kk * 16), *reinterpret_cast<const uint2*>(wb + kk * 16));
     }
     if constexpr (SPLIT) {
 #pragma unroll
