@@ -88,8 +88,8 @@ WIDE = config(128, 211, [
     (latent(6, 32, 32, 48, 96, 64, base=30000.0, scaling=yarn(6.0, 128, 16.0, 1.5)), dense(192)),
     (parallel(attention(8, 2, 48, 32, 70, rot=32, base=9000.0, scaling=llama3(6.0, 1.0, 3.0, 256)),
               recurrence(6, 64, 128, groups=2, norm_groups=3, conv=4), 0.8, 1.2), dense(160)),
-    (latent(4, 64, 16, 32, 64, 48), None),
-    (parallel(attention(4, 4, 32, 64, 200, rot=32), recurrence(4, 48, 32, groups=1, norm_groups=2, conv=3), 1.1, 0.7), dense(96)),
+    (latent(4, 48, 16, 32, 80, 56), None),
+    (parallel(attention(4, 4, 32, 64, 200, rot=32), recurrence(4, 32, 48, groups=1, norm_groups=2, conv=3), 1.1, 0.7), dense(96)),
 ])
 
 CONFIGS = {"mixed": MIXED, "odd": ODD, "parallel_only": PARALLEL_ONLY, "latent_only": LATENT_ONLY}

@@ -52,8 +52,8 @@ def test_libraries_built_for_a_models_sizes():
                                                      latent_attention_fits)
 
     a, b = ctypes.c_int(), ctypes.c_int()
-    lib = ctypes.CDLL(str(build_state_space(20, 33)))
-    assert lib.ie_state_space_dims(ctypes.byref(a), ctypes.byref(b)) == 64 and (a.value, b.value) == (32, 48)
+    lib = ctypes.CDLL(str(build_state_space(20, 17)))
+    assert lib.ie_state_space_dims(ctypes.byref(a), ctypes.byref(b)) == 64 and (a.value, b.value) == (32, 32)
     assert hasattr(lib, "ie_state_space_step") and hasattr(lib, "ie_state_space_chunks")
     with pytest.raises(BuildError, match="128"):
         build_state_space(16, 129)

@@ -480,7 +480,7 @@ def test_window_edges(device, window):
 
 
 @pytest.mark.gpu
-@pytest.mark.parametrize("d,dv,heads,kv", [(96, 96, 4, 2), (48, 32, 8, 2), (64, 128, 3, 3), (128, 16, 4, 1)])
+@pytest.mark.parametrize("d,dv,heads,kv", [(112, 80, 6, 3), (48, 32, 8, 2), (64, 128, 3, 3), (128, 16, 4, 1)])
 @pytest.mark.parametrize("window", [1, 33, 64, 100, 257])
 def test_window_edges_on_the_tensor_cores(d, dv, heads, kv, window):
     """The same in bfloat16: portions that start and end inside tiles of 64, single tokens whose window's keys are cut
@@ -645,7 +645,7 @@ def test_latent_attention_with_a_sink(device):
 
 
 @pytest.mark.gpu
-@pytest.mark.parametrize("dk,dv,H", [(80, 64, 6), (576, 512, 16), (40, 24, 3), (128, 96, 20), (48, 48, 1), (296, 256, 7)])
+@pytest.mark.parametrize("dk,dv,H", [(88, 72, 5), (576, 512, 16), (40, 24, 3), (128, 96, 20), (48, 48, 1), (296, 256, 7)])
 def test_latent_attention_with_a_sink_on_the_tensor_cores(dk, dv, H):
     """bfloat16: 64 rows per block for portions, sixteen for steps of few tokens whose context is cut into ranges that a
     second kernel merges with the sink's term; a second request of one token in every step."""
@@ -686,14 +686,14 @@ def test_far_keys_of_the_latent_attention(dtype):
     from inference_engine_b200.kernels import get_ops
 
     ops, g = get_ops("cuda"), torch.Generator().manual_seed(9)
-    T, H, dk, dv, ps, scale, td = 4500, 4, 80, 64, 16, 0.5, getattr(torch, dtype)
+    T, H, dk, dv, ps, scale, td = 4500, 4, 88, 72, 16, 0.5, getattr(torch, dtype)
     bf = lambda x: x.to(torch.bfloat16).float()  # noqa: E731
     rows, q = bf(torch.randn(T, dk, generator=g) * 0.3), torch.randn(T, H, dk, generator=g) * 0.3
     far = {T - 1: 3, T - 2: 1100, 4099: 4035, 4031: 64, 2500: 0, 70: 63, 3000: 15, 3001: 16}
     for i, (t, target) in enumerate(far.items()):  # (an entry of its own for every probe)
-        q[:, :, 66 + i], rows[:, 66 + i] = 0.0, 0.0
-        rows[target, 66 + i] = 3.0
-        q[t, :, 66 + i] = 10.0
+        q[:, :, 76 + i], rows[:, 76 + i] = 0.0, 0.0
+        rows[target, 76 + i] = 3.0
+        q[t, :, 76 + i] = 10.0
     q, rows, sinks = bf(q), bf(rows), torch.tensor([-1.0, 12.0, 14.0, 10.0])
     order = torch.randperm(-(-T // ps), generator=g).tolist()
     tables = torch.tensor([order], dtype=torch.int32, device="cuda")
@@ -750,7 +750,7 @@ def _space_plain(s, rows, state, weight, parts, eps, rounded):
 
 STEPS = [([1, 1, 3], [5, 0, 9]), ([8, 2], [0, 600]), ([150, 1, 64, 63, 65], [0, 100, 7, 3, 64]), ([300], [11]),
          ([2, 9], [64, 0]), ([65], [0]), ([1], [0]), ([16, 17, 2], [3, 0, 0])]
-SPACES = [(6, 64, 128, 2, 4, 3), (4, 48, 32, 1, 3, 2), (3, 20, 12, 3, 2, 1), (5, 7, 9, 5, 6, 7), (2, 128, 128, 1, 4, 2), (4, 16, 16, 2, 1, 4),
+SPACES = [(6, 64, 128, 2, 4, 3), (4, 40, 48, 1, 3, 2), (3, 20, 12, 3, 2, 1), (5, 7, 9, 5, 6, 7), (2, 128, 128, 1, 4, 2), (4, 16, 16, 2, 1, 4),
           (1, 1, 1, 1, 2, 1), (8, 13, 20, 4, 4, 2), (2, 40, 144, 2, 4, 1), (2, 136, 24, 1, 3, 2)]
 
 
